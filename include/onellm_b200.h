@@ -27,7 +27,9 @@ extern "C" {
 
 #define ONELLM_API __attribute__((visibility("default")))
 
-enum onellm_dtype { ONELLM_F32 = 0, ONELLM_F16 = 1 };
+/* BF16 is the 16-bit type of the designs opened with onellm_model_open; the kernel entry points below take F32 and F16
+ * unless they say otherwise. */
+enum onellm_dtype { ONELLM_F32 = 0, ONELLM_F16 = 1, ONELLM_BF16 = 2 };
 
 enum onellm_status {
     ONELLM_OK = 0,
@@ -488,6 +490,17 @@ ONELLM_API int onellm_llama_create(const onellm_llama_config* cfg, onellm_llama*
 ONELLM_API int onellm_llama_config_from_ini(const char* path, onellm_llama_config* cfg, int* top_k);
 ONELLM_API int onellm_llama_create_from_ini(const char* path, int max_batch, int max_seq_len, int tp_rank, int tp_size,
                                             onellm_llama** out);
+/* A model folder of any registered design: config.json, whose "architecture" names the design, and
+ * model.safetensors.  dtype is the element type of matrix products and activations (ONELLM_BF16 or ONELLM_F32: then
+ * everything is true 32-bit); max_seq_len <= 0: what the configuration allows.  The handle is used with the
+ * onellm_llama_* calls below (prefill, extend, decode_step, generate, set_sampling, get_logits, ...), whatever the design.
+ * Designs: "Finuvik".  onellm_model_create builds the same model from the text of a configuration, without weights
+ * (onellm_llama_init_random fills them).  onellm_model_design: the name of a handle's design ("llama" for
+ * onellm_llama_create).  Unknown design, malformed file, missing or wrongly shaped tensor: ONELLM_ERR_IO. */
+ONELLM_API int onellm_model_open(const char* folder, int dtype, int max_batch, int max_seq_len, onellm_llama** out);
+ONELLM_API int onellm_model_create(const char* config_json, int dtype, int max_batch, int max_seq_len, onellm_llama** out);
+ONELLM_API const char* onellm_model_design(const onellm_llama* m);
+ONELLM_API int onellm_model_limits(const onellm_llama* m, int* vocab_size, int* max_seq_len, int* max_batch);
 ONELLM_API void onellm_llama_destroy(onellm_llama* m);
 ONELLM_API size_t onellm_llama_device_bytes(const onellm_llama* m);
 ONELLM_API void* onellm_llama_stream(onellm_llama* m);
@@ -506,6 +519,7 @@ ONELLM_API int onellm_llama_init_random(onellm_llama* m, uint64_t seed, float st
 ONELLM_API int onellm_nccl_unique_id(void* id128);
 ONELLM_API int onellm_llama_init_comm(onellm_llama* m, const void* id128);
 
+/* top_k 0: a step computes logits only and samples nothing. */
 ONELLM_API int onellm_llama_set_sampling(onellm_llama* m, int top_k, float temperature, int literal_walk);
 ONELLM_API int onellm_llama_set_graphs(onellm_llama* m, int enabled);
 /* Tensor parallel over peer memory instead of NCCL for the decode step (batch * hidden small): every rank
@@ -558,6 +572,11 @@ ONELLM_API int onellm_llama_generate(onellm_llama* m, const int* host_prompt, in
                                      int n_new, int* host_out);
 /* Logits of the last step as float [batch, vocab_size] on the host. */
 ONELLM_API int onellm_llama_get_logits(onellm_llama* m, float* host_logits);
+/* Logits of single tokens of a context pass: the next prefill / prefill_ragged / extend call also computes the logits
+ * of the given token rows (0 = its first token, packed in sequence order); onellm_llama_get_row_logits then copies
+ * them out as float [n_rows, vocab_size], in the order they were asked for. */
+ONELLM_API int onellm_llama_want_logits(onellm_llama* m, const int* rows, int n_rows);
+ONELLM_API int onellm_llama_get_row_logits(onellm_llama* m, float* host_logits, int n_rows);
 ONELLM_API int onellm_llama_get_state(onellm_llama* m, int* cur_len, long* kernel_launches, int* host_seqlen,
                                       unsigned char* host_finished);
 ONELLM_API int onellm_llama_kv_cache(onellm_llama* m, int layer, void** k_cache, void** v_cache);

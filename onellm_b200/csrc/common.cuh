@@ -1,11 +1,13 @@
 // Shared helpers for the sm_100a kernels and their C-ABI entry points.
 #pragma once
+#include <cuda_bf16.h>
 #include <cuda_fp16.h>
 #include <cuda_runtime.h>
 #include <stdint.h>
 #include <stdio.h>
 
 #include <mutex>
+#include <type_traits>
 
 #include "onellm_b200.h"
 
@@ -151,6 +153,65 @@ struct Vec16<__half> {
     }
 };
 
+template <>
+struct Vec16<__nv_bfloat16> {
+    static constexpr int N = 8;
+    __device__ static __forceinline__ void unpack(const uint4& r, float (&f)[8])
+    {
+        const uint32_t w[4] = {r.x, r.y, r.z, r.w};
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+            f[2 * i] = __uint_as_float(w[i] << 16);
+            f[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+        }
+    }
+    __device__ static __forceinline__ uint4 pack(const float (&f)[8])
+    {
+        uint32_t w[4];
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+            const __nv_bfloat162 h = __floats2bfloat162_rn(f[2 * i], f[2 * i + 1]);
+            w[i] = *reinterpret_cast<const uint32_t*>(&h);
+        }
+        return make_uint4(w[0], w[1], w[2], w[3]);
+    }
+    __device__ static __forceinline__ void load(const __nv_bfloat16* p, float (&f)[8])
+    {
+        unpack(*reinterpret_cast<const uint4*>(p), f);
+    }
+};
+
+// Two adjacent 16-bit elements <-> floats, and single elements, for kernels written over the element type.
+template <typename T>
+__device__ __forceinline__ uint32_t pack2(float lo, float hi)
+{
+    if constexpr (sizeof(T) == 2 && std::is_same<T, __half>::value) {
+        const __half2 h = __floats2half2_rn(lo, hi);
+        return *reinterpret_cast<const uint32_t*>(&h);
+    } else {
+        const __nv_bfloat162 h = __floats2bfloat162_rn(lo, hi);
+        return *reinterpret_cast<const uint32_t*>(&h);
+    }
+}
+template <typename T>
+__device__ __forceinline__ float2 unpack2(uint32_t w)
+{
+    if constexpr (std::is_same<T, __half>::value)
+        return __half22float2(*reinterpret_cast<const __half2*>(&w));
+    else
+        return make_float2(__uint_as_float(w << 16), __uint_as_float(w & 0xffff0000u));
+}
+__device__ __forceinline__ float to_float(float v) { return v; }
+__device__ __forceinline__ float to_float(__half v) { return __half2float(v); }
+__device__ __forceinline__ float to_float(__nv_bfloat16 v) { return __bfloat162float(v); }
+template <typename T>
+__device__ __forceinline__ T from_float(float v)
+{
+    if constexpr (std::is_same<T, float>::value) return v;
+    else if constexpr (std::is_same<T, __half>::value) return __float2half_rn(v);
+    else return __float2bfloat16_rn(v);
+}
+
 __device__ __forceinline__ uint4 ld_nc_16(const void* p)
 {
     uint4 r;
@@ -234,6 +295,22 @@ __device__ __forceinline__ void mma_f16(float (&c)[4], uint32_t a0, uint32_t a1,
         : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
         : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
+// The same product on bfloat16 operands, and the element-type dispatch of the two.
+__device__ __forceinline__ void mma_bf16(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0,
+                                         uint32_t b1)
+{
+    asm volatile(
+        "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, "
+        "{%0,%1,%2,%3};"
+        : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+        : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+template <typename T>
+__device__ __forceinline__ void mma_16b(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1)
+{
+    if constexpr (std::is_same<T, __half>::value) mma_f16(c, a0, a1, a2, a3, b0, b1);
+    else mma_bf16(c, a0, a1, a2, a3, b0, b1);
+}
 __device__ __forceinline__ uint32_t pack_h2(float lo, float hi)
 {
     const __half2 h = __floats2half2_rn(lo, hi);
@@ -283,6 +360,11 @@ struct TpEpilogue {
     int rank, world;
 };
 
+// element size of the types every entry point of the C interface takes (bfloat16 is known to a subset of them)
 inline size_t dtype_size(int dtype) { return dtype == ONELLM_F16 ? 2 : (dtype == ONELLM_F32 ? 4 : 0); }
+
+// Gate function of a gated projection, act(x.W) * (x.W2)
+enum GateAct { GATE_SILU = 0, GATE_RELU = 1 };
+__device__ __forceinline__ float gate_act(float g, int act) { return act == GATE_RELU ? fmaxf(g, 0.f) : g / (1.0f + __expf(-g)); }
 
 }  // namespace onellm

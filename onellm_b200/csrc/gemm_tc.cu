@@ -51,19 +51,25 @@ constexpr int kTcSmemBytes = kTcStages * kTcStageBytes + 1024 /* alignment slack
 //   ss_out:  [M, ceil(N / tile columns)]: the sum of squares of the stored (rounded) values of each row inside this
 //            tile's columns -- the row_ss of the projection that reads y next.  Every entry is written by exactly
 //            one block, so the sums do not depend on the order the blocks run in.
+//   act:     gate function of MODE 2
+//   ldy:     row stride of y (and of resid); 0: N
+//   f32:     y and resid are float instead of the element type (no ss_out then)
 struct TcEpilogue {
     const float* row_ss;
     int ss_parts;
     float eps;
-    const __half* resid;
-    const __half* bias;
+    const void* resid;
+    const void* bias;
     float* ss_out;
+    int act;
+    long ldy;
+    int f32;
 };
 
-template <int MODE>
+template <typename T, int MODE>
 __global__ void __launch_bounds__(kTcThreads)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
-               const __grid_constant__ CUtensorMap map_b2, __half* y, int M, int N, int K, const TcEpilogue epi)
+               const __grid_constant__ CUtensorMap map_b2, T* y, int M, int N, int K, const TcEpilogue epi)
 {
     constexpr bool W_NK = MODE == 1;
     constexpr bool DUAL = MODE == 2;
@@ -144,8 +150,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
             }
         }
     } else if (warp == 1 && lane == 0) {
-        // instruction descriptor: D = f32, A = B = f16, A K-major, B MN-major unless W_NK, N = 256, M = 128
-        const uint32_t idesc = (1u << 4) | ((W_NK ? 0u : 1u) << 16) | ((uint32_t)(kTcBN >> 3) << 17) | ((uint32_t)(kTcBM >> 4) << 24);
+        // instruction descriptor: D = f32, A and B of type T, A K-major, B MN-major unless W_NK, N = 256, M = 128
+        const uint32_t idesc = (1u << 4) | umma_operand_bits<T>() | ((W_NK ? 0u : 1u) << 16) | ((uint32_t)(kTcBN >> 3) << 17) | ((uint32_t)(kTcBM >> 4) << 24);
         int it = 0, lt = 0;
         bool ok = true;
         for (int t = blockIdx.x; t < n_tiles && ok; t += gridDim.x, lt++) {
@@ -178,6 +184,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
     } else if (warp >= 2) {
         // epilogue: warp w may touch TMEM lanes 32 * (w % 4) .. + 31, which are the tile rows of the same numbers
         const int q = warp & 3;
+        const size_t ldy = epi.ldy ? (size_t)epi.ldy : (size_t)N;
         int lt = 0;
         bool ok = true;
         for (int t = blockIdx.x; t < n_tiles && ok; t += gridDim.x, lt++) {
@@ -206,7 +213,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
 #pragma unroll
                     for (int i = 0; i < 32; i++) {
                         const float g = __uint_as_float(r[i]) * inv;
-                        r[i] = __float_as_uint(g / (1.0f + __expf(-g)) * (__uint_as_float(u[i]) * inv));
+                        r[i] = __float_as_uint(gate_act(g, epi.act) * (__uint_as_float(u[i]) * inv));
                     }
                 } else {
                     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
@@ -216,28 +223,40 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                     }
                 }
                 if (row < M) {
-                    __half* dst = y + (size_t)row * N + n0 + c0;
+                    const size_t at = (size_t)row * ldy + n0 + c0;
 #pragma unroll
                     for (int j = 0; j < 4; j++) {
                         if (n0 + c0 + 8 * j < N) {  // N is a multiple of 8
                             float v[8];
 #pragma unroll
                             for (int e = 0; e < 8; e++) v[e] = __uint_as_float(r[8 * j + e]);
-                            if (epi.resid) {
-                                float a[8];
-                                Vec16<__half>::load(epi.resid + (size_t)row * N + n0 + c0 + 8 * j, a);
+                            float a[8];
+                            if (epi.bias) {
+                                Vec16<T>::load(static_cast<const T*>(epi.bias) + n0 + c0 + 8 * j, a);
 #pragma unroll
                                 for (int e = 0; e < 8; e++) v[e] += a[e];
-                                if (epi.bias) {
-                                    Vec16<__half>::load(epi.bias + n0 + c0 + 8 * j, a);
-#pragma unroll
-                                    for (int e = 0; e < 8; e++) v[e] += a[e];
-                                }
                             }
-                            const uint4 packed = Vec16<__half>::pack(v);
-                            *reinterpret_cast<uint4*>(dst + 8 * j) = packed;
+                            if (epi.f32) {
+                                float4* dst = reinterpret_cast<float4*>(reinterpret_cast<float*>(y) + at + 8 * j);
+                                if (epi.resid) {
+                                    const float4* rs = reinterpret_cast<const float4*>(static_cast<const float*>(epi.resid) + at + 8 * j);
+                                    const float4 r0 = rs[0], r1 = rs[1];
+                                    v[0] += r0.x; v[1] += r0.y; v[2] += r0.z; v[3] += r0.w;
+                                    v[4] += r1.x; v[5] += r1.y; v[6] += r1.z; v[7] += r1.w;
+                                }
+                                dst[0] = make_float4(v[0], v[1], v[2], v[3]);
+                                dst[1] = make_float4(v[4], v[5], v[6], v[7]);
+                                continue;
+                            }
+                            if (epi.resid) {
+                                Vec16<T>::load(static_cast<const T*>(epi.resid) + at + 8 * j, a);
+#pragma unroll
+                                for (int e = 0; e < 8; e++) v[e] += a[e];
+                            }
+                            const uint4 packed = Vec16<T>::pack(v);
+                            *reinterpret_cast<uint4*>(y + at + 8 * j) = packed;
                             if (epi.ss_out) {
-                                Vec16<__half>::unpack(packed, v);  // what the next projection will read
+                                Vec16<T>::unpack(packed, v);  // what the next projection will read
 #pragma unroll
                                 for (int e = 0; e < 8; e++) sq = fmaf(v[e], v[e], sq);
                             }
@@ -278,7 +297,7 @@ static EncodeTiledFn encode_tiled()
     return fn;
 }
 
-// 2-D fp16 tensor map: `inner` contiguous elements, `outer` rows of `inner` elements; box {64, box_outer}; 128-byte swizzle
+// 2-D tensor map of 16-bit elements: `inner` contiguous elements, `outer` rows of `inner` elements; box {64, box_outer}; 128-byte swizzle
 int make_map(CUtensorMap* map, const void* base, uint64_t inner, uint64_t outer, uint32_t box_outer)
 {
     EncodeTiledFn enc = encode_tiled();
@@ -297,7 +316,8 @@ int make_map(CUtensorMap* map, const void* base, uint64_t inner, uint64_t outer,
 int gemm_f16_skinny(const __half* x, const __half* W, __half* y, int M, int N, int K, int w_layout, cudaStream_t st);
 
 // mode 0: W [K,N]; 1: W [N,K]; 2: W and W2 [K,N], y = silu(x.W) * (x.W2)
-static int gemm_tc_launch(const __half* x, const __half* W, const __half* W2, __half* y, int M, int N, int K, int mode, cudaStream_t st,
+template <typename T>
+static int gemm_tc_launch(const T* x, const T* W, const T* W2, T* y, int M, int N, int K, int mode, cudaStream_t st,
                           const TcEpilogue& epi = TcEpilogue{})
 {
     ONELLM_REQUIRE(K % 8 == 0 && N % 8 == 0, ONELLM_ERR_UNSUPPORTED, "gemm: M > 64 needs K %% 8 == 0 and N %% 8 == 0 (K=%d N=%d)",
@@ -314,7 +334,7 @@ static int gemm_tc_launch(const __half* x, const __half* W, const __half* W2, __
     }
     static DeviceOnce smem_attr[3];
     {
-        const void* fn = mode == 0 ? (const void*)gemm_tc_kernel<0> : mode == 1 ? (const void*)gemm_tc_kernel<1> : (const void*)gemm_tc_kernel<2>;
+        const void* fn = mode == 0 ? (const void*)gemm_tc_kernel<T, 0> : mode == 1 ? (const void*)gemm_tc_kernel<T, 1> : (const void*)gemm_tc_kernel<T, 2>;
         ONELLM_CUDA(smem_attr[mode].run([fn] { return cudaFuncSetAttribute(fn, cudaFuncAttributeMaxDynamicSharedMemorySize, kTcSmemBytes); }));
     }
     const int out_n = mode == 2 ? kTcBN / 2 : kTcBN;
@@ -322,23 +342,23 @@ static int gemm_tc_launch(const __half* x, const __half* W, const __half* W2, __
     ONELLM_REQUIRE(tiles <= 0x7fffffffL, ONELLM_ERR_UNSUPPORTED, "gemm: too many tiles");
     const dim3 grid((unsigned)std::min<long>(tiles, num_sms()));  // persistent: one block per SM (shared memory allows no more)
     if (mode == 0)
-        ONELLM_CUDA(launch_pdl(gemm_tc_kernel<0>, grid, dim3(kTcThreads), kTcSmemBytes, st, map_a, map_b, map_b2, y, M, N, K, epi));
+        ONELLM_CUDA(launch_pdl(gemm_tc_kernel<T, 0>, grid, dim3(kTcThreads), kTcSmemBytes, st, map_a, map_b, map_b2, y, M, N, K, epi));
     else if (mode == 1)
-        ONELLM_CUDA(launch_pdl(gemm_tc_kernel<1>, grid, dim3(kTcThreads), kTcSmemBytes, st, map_a, map_b, map_b2, y, M, N, K, epi));
+        ONELLM_CUDA(launch_pdl(gemm_tc_kernel<T, 1>, grid, dim3(kTcThreads), kTcSmemBytes, st, map_a, map_b, map_b2, y, M, N, K, epi));
     else
-        ONELLM_CUDA(launch_pdl(gemm_tc_kernel<2>, grid, dim3(kTcThreads), kTcSmemBytes, st, map_a, map_b, map_b2, y, M, N, K, epi));
+        ONELLM_CUDA(launch_pdl(gemm_tc_kernel<T, 2>, grid, dim3(kTcThreads), kTcSmemBytes, st, map_a, map_b, map_b2, y, M, N, K, epi));
     return ONELLM_OK;
 }
 
 int gemm_f16_large(const __half* x, const __half* W, __half* y, int M, int N, int K, int w_layout, cudaStream_t st)
 {
-    return gemm_tc_launch(x, W, nullptr, y, M, N, K, w_layout == ONELLM_W_NK ? 1 : 0, st);
+    return gemm_tc_launch<__half>(x, W, nullptr, y, M, N, K, w_layout == ONELLM_W_NK ? 1 : 0, st);
 }
 
 // Gate and up projections with SwiGLU in the epilogue, M > 64.
 int gemm_swiglu_f16_large(const __half* x, const __half* Wg, const __half* Wu, __half* out, int M, int I, int K, cudaStream_t st)
 {
-    return gemm_tc_launch(x, Wg, Wu, out, M, I, K, 2, st);
+    return gemm_tc_launch<__half>(x, Wg, Wu, out, M, I, K, 2, st);
 }
 
 // Column tiles of a projection with N outputs (two weights: gate and up share a tile): the second extent of the
@@ -353,8 +373,27 @@ int gemm_rows_parts(int N, bool dual)
 int gemm_rows_f16(const __half* x, const __half* W, const __half* W2, __half* y, int M, int N, int K, const float* row_ss, int ss_parts,
                   float eps, const __half* resid, const __half* bias, float* ss_out, cudaStream_t st)
 {
-    const TcEpilogue epi = {row_ss, ss_parts, eps, resid, resid ? bias : nullptr, ss_out};
-    return gemm_tc_launch(x, W, W2, y, M, N, K, W2 ? 2 : 0, st, epi);
+    TcEpilogue epi = {};
+    epi.row_ss = row_ss;
+    epi.ss_parts = ss_parts;
+    epi.eps = eps;
+    epi.resid = resid;
+    epi.bias = resid ? bias : nullptr;
+    epi.ss_out = ss_out;
+    return gemm_tc_launch<__half>(x, W, W2, y, M, N, K, W2 ? 2 : 0, st, epi);
+}
+
+// The bfloat16 form (more than 64 tokens) for the model classes: W and W2 [K,N] (W2: gate form, act(x.W) * (x.W2)); y in
+// bfloat16 or, with f32, in float with an optional float residual; ldy is the row stride of y and resid.
+int gemm_bf16_large(const __nv_bfloat16* x, const __nv_bfloat16* W, const __nv_bfloat16* W2, void* y, long ldy, int M, int N, int K, int act,
+                    int f32, const float* resid, cudaStream_t st)
+{
+    TcEpilogue epi = {};
+    epi.resid = resid;
+    epi.act = act;
+    epi.ldy = ldy;
+    epi.f32 = f32;
+    return gemm_tc_launch<__nv_bfloat16>(x, W, W2, static_cast<__nv_bfloat16*>(y), M, N, K, W2 ? 2 : 0, st, epi);
 }
 
 int attn_tc_timeout_flag();  // context_attn_tc.cu

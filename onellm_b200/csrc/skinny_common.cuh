@@ -20,13 +20,19 @@ constexpr int kRedLd = kBN + 1;   // row stride of the partial tile in shared me
 //          of squares is taken from the activations as they pass through the ring (no extra reads).
 //   resid: y = resid + bias + result (bias may be NULL); resid may be y itself (each element is read
 //          and written by the same thread).
+//   act:   gate function of the two-weight form.
+//   ldy:   row stride of y (and of resid); 0: N.
+//   f32:   y and resid are float instead of the element type (a residual stream or logits kept in 32 bits).
 struct EpilogueArgs {
-    const __half* resid;  // [M, N] or NULL
-    const __half* bias;   // [N] or NULL
+    const void* resid;  // [M, N] or NULL
+    const void* bias;   // [N] or NULL
     float rms_eps;
     int rms;
     int early_dependents;  // release the next kernel before the main loop (it then shares the SM with this one)
     TpEpilogue tp;         // tensor parallel: y = resid + bias + sum over ranks of this projection (see common.cuh)
+    int act;
+    long ldy;
+    int f32;
 };
 
 // `red` holds this block's partial tile as [NW][MP][kRedLd] floats followed by MP partial sums of squares (used
@@ -34,8 +40,8 @@ struct EpilogueArgs {
 // same tile.  Sums them in rank order and finishes the tile; every thread of the block (NT of them) calls it.
 // WIDE (tcgen05 kernel, no tensor-parallel exchange): the second half of `red` is not a second weight but the next
 // 128 output columns of the same weight (a block owns 256 columns and reads its activations once for both).
-template <int MP, bool DUAL, bool FUSED, int NT, bool WIDE = false>
-__device__ __forceinline__ void splitk_epilogue(float* red, cg::cluster_group& cluster, __half* y, int M, int N, int K, int n0,
+template <typename T, int MP, bool DUAL, bool FUSED, int NT, bool WIDE = false>
+__device__ __forceinline__ void splitk_epilogue(float* red, cg::cluster_group& cluster, T* y, int M, int N, int K, int n0,
                                                 const EpilogueArgs& ep)
 {
     static_assert(!(DUAL && WIDE), "two weights or two column tiles, not both");
@@ -93,8 +99,8 @@ __device__ __forceinline__ void splitk_epilogue(float* red, cg::cluster_group& c
             s1.x *= inv;
             s1.y *= inv;
         }
-        v0 = DUAL ? (s0.x / (1.0f + __expf(-s0.x))) * s1.x : s0.x;
-        v1 = DUAL ? (s0.y / (1.0f + __expf(-s0.y))) * s1.y : s0.y;
+        v0 = DUAL ? gate_act(s0.x, ep.act) * s1.x : s0.x;
+        v1 = DUAL ? gate_act(s0.y, ep.act) * s1.y : s0.y;
         w0 = s1.x;  // WIDE: the same pair 128 columns further
         w1 = s1.y;
         return true;
@@ -122,26 +128,37 @@ __device__ __forceinline__ void splitk_epilogue(float* red, cg::cluster_group& c
         for (int r = 0; r < 8; r++)
             if (r < ep.tp.world) {
                 const uint32_t w = r == ep.tp.rank ? word : await(ep.tp.mine + (size_t)r * ep.tp.slot_words + idx / 2);
-                const float2 f = __half22float2(*reinterpret_cast<const __half2*>(&w));
+                const float2 f = unpack2<T>(w);
                 v0 += f.x;
                 v1 += f.y;
             }
     };
-    // residual and bias, then the store; returns what was stored
-    auto finish = [&](size_t idx, int c, float v0, float v1) {
+    // residual and bias, then the store; returns what was stored (16-bit outputs)
+    const size_t ldy = ep.ldy ? (size_t)ep.ldy : (size_t)N;
+    auto finish = [&](int tok, int c, float v0, float v1) {
+        const size_t at = (size_t)tok * ldy + n0 + c;
+        if (!FUSED && ep.bias) {
+            const float2 bb = unpack2<T>(*reinterpret_cast<const uint32_t*>(static_cast<const T*>(ep.bias) + n0 + c));
+            v0 += bb.x;
+            v1 += bb.y;
+        }
+        if (!FUSED && ep.f32) {
+            if (ep.resid) {
+                const float2 rr = *reinterpret_cast<const float2*>(static_cast<const float*>(ep.resid) + at);
+                v0 += rr.x;
+                v1 += rr.y;
+            }
+            *reinterpret_cast<float2*>(reinterpret_cast<float*>(y) + at) = make_float2(v0, v1);
+            return 0u;
+        }
         if (!FUSED && ep.resid) {
-            const float2 rr = __half22float2(*reinterpret_cast<const __half2*>(ep.resid + idx));
+            const float2 rr = unpack2<T>(*reinterpret_cast<const uint32_t*>(static_cast<const T*>(ep.resid) + at));
             v0 += rr.x;
             v1 += rr.y;
-            if (ep.bias) {
-                const float2 bb = __half22float2(*reinterpret_cast<const __half2*>(ep.bias + n0 + c));
-                v0 += bb.x;
-                v1 += bb.y;
-            }
         }
-        const __half2 out = __floats2half2_rn(v0, v1);
-        *reinterpret_cast<__half2*>(y + idx) = out;
-        return *reinterpret_cast<const uint32_t*>(&out);
+        const uint32_t out = pack2<T>(v0, v1);
+        *reinterpret_cast<uint32_t*>(y + at) = out;
+        return out;
     };
 
     if (tp && ep.tp.two_shot) {
@@ -157,8 +174,7 @@ __device__ __forceinline__ void splitk_epilogue(float* red, cg::cluster_group& c
             float v0, v1, w0, w1;
             if (!partial(e, v0, v1, w0, w1)) continue;
             const int tok = e / kBN, c = e % kBN;
-            const __half2 own = __floats2half2_rn(v0, v1);
-            mine[it] = *reinterpret_cast<const uint32_t*>(&own);
+            mine[it] = pack2<T>(v0, v1);
             valid |= 1u << it;
             const int owner = tok % ep.tp.world;
             if (owner != ep.tp.rank) send(ep.tp.push[owner] + ((size_t)tok * N + n0 + c) / 2, mine[it]);
@@ -170,7 +186,7 @@ __device__ __forceinline__ void splitk_epilogue(float* red, cg::cluster_group& c
             const size_t idx = (size_t)tok * N + n0 + c;
             float v0, v1;
             gather(idx, mine[it], v0, v1);
-            const uint32_t w = finish(idx, c, v0, v1);
+            const uint32_t w = finish(tok, c, v0, v1);
 #pragma unroll
             for (int r = 0; r < 8; r++)
                 if (r < ep.tp.world && r != ep.tp.rank) send(ep.tp.final_push[r] + idx / 2, w);
@@ -189,17 +205,16 @@ __device__ __forceinline__ void splitk_epilogue(float* red, cg::cluster_group& c
         if (!partial(e, v0, v1, w0, w1)) continue;
         const int tok = e / kBN, c = e % kBN;
         const size_t idx = (size_t)tok * N + n0 + c;
-        if (WIDE && n0 + kBN + c < N) (void)finish(idx + kBN, c + kBN, w0, w1);
+        if (WIDE && n0 + kBN + c < N) (void)finish(tok, c + kBN, w0, w1);
         if (tp) {
             // one-shot: this rank's value of the two elements to every peer, then theirs
-            const __half2 own = __floats2half2_rn(v0, v1);
-            const uint32_t word = *reinterpret_cast<const uint32_t*>(&own);
+            const uint32_t word = pack2<T>(v0, v1);
 #pragma unroll
             for (int r = 0; r < 8; r++)
                 if (r < ep.tp.world && r != ep.tp.rank) send(ep.tp.push[r] + idx / 2, word);
             gather(idx, word, v0, v1);
         }
-        (void)finish(idx, c, v0, v1);
+        (void)finish(tok, c, v0, v1);
     }
 }
 

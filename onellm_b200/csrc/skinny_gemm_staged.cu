@@ -41,14 +41,6 @@ __device__ __forceinline__ void ldmatrix_x4_trans(uint32_t (&r)[4], uint32_t add
                  : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
                  : "r"(addr));
 }
-__device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1)
-{
-    asm volatile(
-        "mma.sync.aligned.m16n8k16.row.col.f32.f16.f16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, "
-        "{%0,%1,%2,%3};"
-        : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-        : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
 
 // y[M,N] = x[M,K] . W0                    (DUAL = false)
 // y[M,N] = silu(x.W0) * (x.W1)            (DUAL = true)
@@ -59,19 +51,20 @@ __device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], 
 // the projection, as src/layers/decoder/self_decoder.cpp:50-73 sequences them), keeps xn in shared
 // memory for the whole kernel and, in the blocks of column tile 0, stores r as the new residual.
 // `x` may be NULL (r = residual: the plain RMSNorm in front of layer 0).
+template <typename T>
 struct FusedNormArgs {
-    const __half* residual;  // [M, K]
-    const __half* bias;      // [K] or NULL
-    const __half* gamma;     // [K]
-    __half* residual_out;    // [M, K], must not alias residual (other blocks still read it); NULL when x is NULL
+    const T* residual;  // [M, K]
+    const T* bias;      // [K] or NULL
+    const T* gamma;     // [K]
+    T* residual_out;    // [M, K], must not alias residual (other blocks still read it); NULL when x is NULL
     float eps;
 };
 
-template <int MB, bool DUAL, bool FUSED>
+template <typename T, int MB, bool DUAL, bool FUSED>
 __global__ void __launch_bounds__(kStThreads)
-skinny_kn_staged_kernel(const __half* __restrict__ x, const __half* __restrict__ W0, const __half* __restrict__ W1,
-                        __half* y, int M, int N, int K, int stages_per_block, int nst,
-                        const FusedNormArgs fn, const EpilogueArgs ep)
+skinny_kn_staged_kernel(const T* __restrict__ x, const T* __restrict__ W0, const T* __restrict__ W1,
+                        T* y, int M, int N, int K, int stages_per_block, int nst,
+                        const FusedNormArgs<T> fn, const EpilogueArgs ep)
 {
     constexpr int NW = DUAL ? 2 : 1;
     constexpr int MP = 8 * MB;
@@ -91,7 +84,7 @@ skinny_kn_staged_kernel(const __half* __restrict__ x, const __half* __restrict__
     // Copy assignments, fixed for the whole kernel: chunk c = tid + 256*i is row c/16 of the stage,
     // 16-byte column c%16.  Source pointers advance by 32 rows per stage; destinations are offsets
     // inside a stage (XOR-swizzled by the row).
-    const __half* wsrc[NW][CPT];
+    const T* wsrc[NW][CPT];
     uint32_t wdst[CPT];
     int wrow[CPT];
     bool wcol_ok[CPT];
@@ -111,7 +104,7 @@ skinny_kn_staged_kernel(const __half* __restrict__ x, const __half* __restrict__
     // activations: thread tid < 4*MP copies 16 bytes of row tid/4
     const bool x_thread = !FUSED && tid < MP * 4;
     const int x_part = tid & 3;
-    const __half* xsrc = FUSED ? x : x + (size_t)min(tid >> 2, M - 1) * K + k_begin + x_part * 8;
+    const T* xsrc = FUSED ? x : x + (size_t)min(tid >> 2, M - 1) * K + k_begin + x_part * 8;
     const uint32_t xdst = NW * kStageBytes + (tid >> 2) * kXRowBytes + x_part * 16;
 
     int w_issued = 0, x_issued = 0;  // stages whose copies have been issued
@@ -164,14 +157,14 @@ skinny_kn_staged_kernel(const __half* __restrict__ x, const __half* __restrict__
     // FUSED: normalised activations of this block's K range, [MP][xn_ld] halfs behind the ring
     const int kc = stages_per_block * kKC;               // K range of a block (multiple of 32)
     const int xn_ld = kc + 8;                            // row stride in halfs: an odd number of 16-byte units
-    __half* xn = reinterpret_cast<__half*>(smem + (size_t)nst * STAGE);
+    T* xn = reinterpret_cast<T*>(smem + (size_t)nst * STAGE);
     if (FUSED) {
         __shared__ float inv_rms[MP];
         // one warp per token row: r = x + residual + bias over the whole row, sum of squares by shuffles
         for (int m = warp; m < MP; m += kStThreads / 32) {
             const int mr = min(m, M - 1);
-            const __half* xr = x ? x + (size_t)mr * K : nullptr;
-            const __half* rr = fn.residual + (size_t)mr * K;
+            const T* xr = x ? x + (size_t)mr * K : nullptr;
+            const T* rr = fn.residual + (size_t)mr * K;
             float ss = 0.f;
             // loads are issued eight vectors at a time before any of them is used: the row comes
             // from L2 and a load-use-load chain would cost one L2 round trip per vector
@@ -193,9 +186,9 @@ skinny_kn_staged_kernel(const __half* __restrict__ x, const __half* __restrict__
                     const int i = i0 + 32 * j;
                     if (i >= nv) break;
                     float v[8], a[8], c[8];
-                    Vec16<__half>::unpack(rv[j], v);
-                    Vec16<__half>::unpack(xv[j], a);
-                    Vec16<__half>::unpack(bv[j], c);
+                    Vec16<T>::unpack(rv[j], v);
+                    Vec16<T>::unpack(xv[j], a);
+                    Vec16<T>::unpack(bv[j], c);
 #pragma unroll
                     for (int e = 0; e < 8; e++) {
                         v[e] = v[e] + a[e] + c[e];
@@ -203,7 +196,7 @@ skinny_kn_staged_kernel(const __half* __restrict__ x, const __half* __restrict__
                     }
                     const int k = i * 8;
                     if (k >= k_begin && k < k_end) {
-                        const uint4 packed = Vec16<__half>::pack(v);
+                        const uint4 packed = Vec16<T>::pack(v);
                         *reinterpret_cast<uint4*>(xn + (size_t)m * xn_ld + (k - k_begin)) = packed;
                         if (blockIdx.x == 0 && fn.residual_out && m < M)
                             *reinterpret_cast<uint4*>(fn.residual_out + (size_t)m * K + k) = packed;
@@ -218,12 +211,12 @@ skinny_kn_staged_kernel(const __half* __restrict__ x, const __half* __restrict__
         for (int idx = tid; idx < MP * nvec; idx += kStThreads) {
             const int m = idx / nvec, i = idx % nvec;
             float v[8], gmm[8];
-            Vec16<__half>::load(xn + (size_t)m * xn_ld + i * 8, v);
-            Vec16<__half>::load(fn.gamma + k_begin + i * 8, gmm);
+            Vec16<T>::load(xn + (size_t)m * xn_ld + i * 8, v);
+            Vec16<T>::load(fn.gamma + k_begin + i * 8, gmm);
             const float inv = inv_rms[m];
 #pragma unroll
             for (int e = 0; e < 8; e++) v[e] = gmm[e] * v[e] * inv;
-            *reinterpret_cast<uint4*>(xn + (size_t)m * xn_ld + i * 8) = Vec16<__half>::pack(v);
+            *reinterpret_cast<uint4*>(xn + (size_t)m * xn_ld + i * 8) = Vec16<T>::pack(v);
         }
         // visibility to the other warps: the barrier at the top of the main loop
     } else {
@@ -284,8 +277,8 @@ skinny_kn_staged_kernel(const __half* __restrict__ x, const __half* __restrict__
                 // lane (g, t) holds x[token 8*mb + g][k = 2t, 2t+1, 2t+8, 2t+9] of this 16-row step
 #pragma unroll
                 for (int mb = 0; mb < MB; mb++) {
-                    const float2 a = __half22float2(*reinterpret_cast<const __half2*>(&xb[mb][0]));
-                    const float2 b = __half22float2(*reinterpret_cast<const __half2*>(&xb[mb][1]));
+                    const float2 a = unpack2<T>(xb[mb][0]);
+                    const float2 b = unpack2<T>(xb[mb][1]);
                     ssq[mb] = fmaf(a.x, a.x, fmaf(a.y, a.y, fmaf(b.x, b.x, fmaf(b.y, b.y, ssq[mb]))));
                 }
             }
@@ -296,7 +289,7 @@ skinny_kn_staged_kernel(const __half* __restrict__ x, const __half* __restrict__
                 // ldmatrix order is (n 0-7, k 0-7), (n 8-15, k 0-7), (n 0-7, k 8-15), (n 8-15, k 8-15)
                 // = a0, a1, a2, a3 of the mma "row" operand
 #pragma unroll
-                for (int mb = 0; mb < MB; mb++) mma16816(acc[w][mb], a, xb[mb][0], xb[mb][1]);
+                for (int mb = 0; mb < MB; mb++) mma_16b<T>(acc[w][mb], a[0], a[1], a[2], a[3], xb[mb][0], xb[mb][1]);
             }
         }
     }
@@ -326,7 +319,7 @@ skinny_kn_staged_kernel(const __half* __restrict__ x, const __half* __restrict__
             if (t == 0) red_ss[8 * mb + g] = v;
         }
     }
-    splitk_epilogue<MP, DUAL, FUSED, kStThreads>(red, cluster, y, M, N, K, n0, ep);
+    splitk_epilogue<T, MP, DUAL, FUSED, kStThreads>(red, cluster, y, M, N, K, n0, ep);
     cluster.sync();  // peers may still be reading this block's tile
 }
 
@@ -398,10 +391,10 @@ static std::map<std::tuple<int, int, bool>, std::pair<int, int>>& plan_overrides
 }
 static std::mutex g_override_mu;
 
-template <int MB, bool DUAL, bool FUSED>
+template <typename T, int MB, bool DUAL, bool FUSED>
 static StagedPlan plan_staged(int N, int K, bool tp)
 {
-    auto kern = skinny_kn_staged_kernel<MB, DUAL, FUSED>;
+    auto kern = skinny_kn_staged_kernel<T, MB, DUAL, FUSED>;
     constexpr int NW = DUAL ? 2 : 1;
     constexpr size_t stage = (size_t)NW * kStageBytes + (FUSED ? 0 : 8 * MB * kXRowBytes);
     constexpr size_t red = ((size_t)NW * 8 * MB * kRedLd + 8 * MB) * sizeof(float);
@@ -423,7 +416,7 @@ static StagedPlan plan_staged(int N, int K, bool tp)
             plan.ks = std::max(1, std::min(ov->second.first, std::min(8, total_stages)));
             plan.nst = std::max(3, std::min(ov->second.second, 12));  // the prologue holds at most 11 stages of activations in registers
             plan.per_block = (total_stages + plan.ks - 1) / plan.ks;
-            const size_t xn = FUSED ? (size_t)8 * MB * (plan.per_block * kKC + 8) * sizeof(__half) : 0;
+            const size_t xn = FUSED ? (size_t)8 * MB * (plan.per_block * kKC + 8) * sizeof(T) : 0;
             plan.smem = std::max(stage * plan.nst, red) + xn;
             if (plan.smem > smem_cap) plan.status = cudaErrorInvalidConfiguration;
             return plan;
@@ -463,7 +456,7 @@ static StagedPlan plan_staged(int N, int K, bool tp)
         const int per = (total_stages + ks - 1) / ks;
         if (ks > 1 && per < 4) break;
         const long total = (long)col_blocks * ks;
-        const size_t xn_b = FUSED ? (size_t)8 * MB * (per * kKC + 8) * sizeof(__half) : 0;
+        const size_t xn_b = FUSED ? (size_t)8 * MB * (per * kKC + 8) * sizeof(T) : 0;
         for (int nst = std::min(12, std::max(3, per + 1)); nst >= 3; nst--) {
             const size_t smem = std::max(stage * nst, red) + xn_b;
             if (smem > smem_cap) continue;
@@ -488,7 +481,7 @@ static StagedPlan plan_staged(int N, int K, bool tp)
     plan.ks = best_ks;
     plan.nst = best_nst;
     plan.per_block = (total_stages + best_ks - 1) / best_ks;
-    const size_t xn_final = FUSED ? (size_t)8 * MB * (plan.per_block * kKC + 8) * sizeof(__half) : 0;
+    const size_t xn_final = FUSED ? (size_t)8 * MB * (plan.per_block * kKC + 8) * sizeof(T) : 0;
     plan.smem = std::max(stage * best_nst, red) + xn_final;
     if (plan.status == cudaSuccess && plan.smem > smem_cap) plan.status = cudaErrorInvalidConfiguration;
     if (plan.status == cudaSuccess && tp && (long)col_blocks * best_ks > kTpMaxBlocks) plan.status = cudaErrorInvalidConfiguration;
@@ -496,12 +489,12 @@ static StagedPlan plan_staged(int N, int K, bool tp)
     return plan;
 }
 
-template <int MB, bool DUAL, bool FUSED>
-static cudaError_t launch_staged(const __half* x, const __half* W0, const __half* W1, __half* y, int M, int N, int K,
-                                 const FusedNormArgs& fn, const EpilogueArgs& ep, cudaStream_t st)
+template <typename T, int MB, bool DUAL, bool FUSED>
+static cudaError_t launch_staged(const T* x, const T* W0, const T* W1, T* y, int M, int N, int K, const FusedNormArgs<T>& fn,
+                                 const EpilogueArgs& ep, cudaStream_t st)
 {
-    auto kern = skinny_kn_staged_kernel<MB, DUAL, FUSED>;
-    const StagedPlan plan = plan_staged<MB, DUAL, FUSED>(N, K, ep.tp.world > 1);
+    auto kern = skinny_kn_staged_kernel<T, MB, DUAL, FUSED>;
+    const StagedPlan plan = plan_staged<T, MB, DUAL, FUSED>(N, K, ep.tp.world > 1);
     if (plan.status != cudaSuccess) return plan.status;
     cudaLaunchConfig_t cfg = {};
     cudaLaunchAttribute attr[2];
@@ -524,7 +517,7 @@ static cudaError_t launch_staged(const __half* x, const __half* W0, const __half
 template <int MB>
 static StagedPlan plan_for(bool dual, int N, int K)
 {
-    return dual ? plan_staged<MB, true, false>(N, K, false) : plan_staged<MB, false, false>(N, K, false);
+    return dual ? plan_staged<__half, MB, true, false>(N, K, false) : plan_staged<__half, MB, false, false>(N, K, false);
 }
 
 // The plan a projection of M tokens would be launched with (K split, ring depth, thread blocks).
@@ -569,33 +562,49 @@ void staged_plan_override(int N, int K, bool dual, int ks, int nst)
 }
 
 // skinny_gemm_tc.cu
-bool skinny_tc_takes(int M, int N, int K);
-cudaError_t skinny_tc_dispatch(const __half* x, const __half* W0, const __half* W1, __half* y, int M, int N, int K, const EpilogueArgs& ep,
-                               cudaStream_t st);
+template <typename T>
+cudaError_t skinny_tc_dispatch(const T* x, const T* W0, const T* W1, T* y, int M, int N, int K, const EpilogueArgs& ep, cudaStream_t st);
+extern template cudaError_t skinny_tc_dispatch<__half>(const __half*, const __half*, const __half*, __half*, int, int, int,
+                                                       const EpilogueArgs&, cudaStream_t);
+extern template cudaError_t skinny_tc_dispatch<__nv_bfloat16>(const __nv_bfloat16*, const __nv_bfloat16*, const __nv_bfloat16*,
+                                                              __nv_bfloat16*, int, int, int, const EpilogueArgs&, cudaStream_t);
 
-// One pass of at most 64 tokens.  Called from skinny_gemm.cu.
+// One pass of at most 64 tokens (W1: the second weight of the gated form or NULL), whatever the epilogue.
+template <typename T>
+cudaError_t skinny_kn_project(const T* x, const T* W0, const T* W1, T* y, int M, int N, int K, const EpilogueArgs& ep, cudaStream_t st)
+{
+    const FusedNormArgs<T> none = {nullptr, nullptr, nullptr, nullptr, 0.f};
+    // more than a few 8-token rows: the tcgen05 kernel (skinny_gemm_tc.cu)
+    if (skinny_tc_takes(M, N, K)) return skinny_tc_dispatch<T>(x, W0, W1, y, M, N, K, ep, st);
+    if (W1) {
+        if (M <= 8) return launch_staged<T, 1, true, false>(x, W0, W1, y, M, N, K, none, ep, st);
+        if (M <= 16) return launch_staged<T, 2, true, false>(x, W0, W1, y, M, N, K, none, ep, st);
+        if (M <= 32) return launch_staged<T, 4, true, false>(x, W0, W1, y, M, N, K, none, ep, st);
+        return launch_staged<T, 8, true, false>(x, W0, W1, y, M, N, K, none, ep, st);
+    }
+    if (M <= 8) return launch_staged<T, 1, false, false>(x, W0, nullptr, y, M, N, K, none, ep, st);
+    if (M <= 16) return launch_staged<T, 2, false, false>(x, W0, nullptr, y, M, N, K, none, ep, st);
+    if (M <= 32) return launch_staged<T, 4, false, false>(x, W0, nullptr, y, M, N, K, none, ep, st);
+    return launch_staged<T, 8, false, false>(x, W0, nullptr, y, M, N, K, none, ep, st);
+}
+template cudaError_t skinny_kn_project<__nv_bfloat16>(const __nv_bfloat16*, const __nv_bfloat16*, const __nv_bfloat16*, __nv_bfloat16*, int,
+                                                      int, int, const EpilogueArgs&, cudaStream_t);
+
+// The fp16 form with the options of the C interface.  Called from skinny_gemm.cu.
 cudaError_t skinny_kn_staged_dispatch(const __half* x, const __half* W0, const __half* W1, __half* y, int M, int N,
                                       int K, bool dual, cudaStream_t st, const __half* resid, const __half* bias,
                                       float rms_eps, const TpEpilogue* tp)
 {
-    const FusedNormArgs none = {nullptr, nullptr, nullptr, nullptr, 0.f};
-    if (skinny_tc_takes(M, N, K)) {  // more than a few 8-token rows: the tcgen05 kernel (skinny_gemm_tc.cu)
-        const EpilogueArgs ep_tc = {resid, resid ? bias : nullptr, rms_eps, rms_eps >= 0.f ? 1 : 0, 1, tp ? *tp : TpEpilogue{}};
-        return skinny_tc_dispatch(x, W0, dual ? W1 : nullptr, y, M, N, K, ep_tc, st);
-    }
     // the next kernel is released as soon as this one's first weight copies are out: its blocks cannot
     // become resident before blocks of this kernel retire (shared memory), but its launch latency is hidden
-    const EpilogueArgs ep = {resid, resid ? bias : nullptr, rms_eps, rms_eps >= 0.f ? 1 : 0, 1, tp ? *tp : TpEpilogue{}};
-    if (dual) {
-        if (M <= 8) return launch_staged<1, true, false>(x, W0, W1, y, M, N, K, none, ep, st);
-        if (M <= 16) return launch_staged<2, true, false>(x, W0, W1, y, M, N, K, none, ep, st);
-        if (M <= 32) return launch_staged<4, true, false>(x, W0, W1, y, M, N, K, none, ep, st);
-        return launch_staged<8, true, false>(x, W0, W1, y, M, N, K, none, ep, st);
-    }
-    if (M <= 8) return launch_staged<1, false, false>(x, W0, nullptr, y, M, N, K, none, ep, st);
-    if (M <= 16) return launch_staged<2, false, false>(x, W0, nullptr, y, M, N, K, none, ep, st);
-    if (M <= 32) return launch_staged<4, false, false>(x, W0, nullptr, y, M, N, K, none, ep, st);
-    return launch_staged<8, false, false>(x, W0, nullptr, y, M, N, K, none, ep, st);
+    EpilogueArgs ep = {};
+    ep.resid = resid;
+    ep.bias = resid ? bias : nullptr;
+    ep.rms_eps = rms_eps;
+    ep.rms = rms_eps >= 0.f ? 1 : 0;
+    ep.early_dependents = 1;
+    if (tp) ep.tp = *tp;
+    return skinny_kn_project<__half>(x, W0, dual ? W1 : nullptr, y, M, N, K, ep, st);
 }
 
 }  // namespace onellm
@@ -620,19 +629,19 @@ extern "C" int onellm_add_residual_rmsnorm_gemm(int dtype, const void* x, const 
                        (!bias || aligned16(bias)) && (!Wu || aligned16(Wu)) && (!residual_out || aligned16(residual_out)),
                    ONELLM_ERR_ARG, "add_residual_rmsnorm_gemm: pointers must be 16-byte aligned");
     if (M == 0) return ONELLM_OK;
-    const FusedNormArgs fn = {(const __half*)residual, (const __half*)bias, (const __half*)gamma,
+    const FusedNormArgs<__half> fn = {(const __half*)residual, (const __half*)bias, (const __half*)gamma,
                               x ? (__half*)residual_out : nullptr, eps};
     cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
     const __half *xh = (const __half*)x, *w0 = (const __half*)W, *w1 = (const __half*)Wu;
     __half* yh = (__half*)y;
-    const EpilogueArgs no_ep = {nullptr, nullptr, 0.f, 0, 0, TpEpilogue{}};
+    const EpilogueArgs no_ep = {};
     cudaError_t e;
     if (Wu)
-        e = M <= 8 ? launch_staged<1, true, true>(xh, w0, w1, yh, M, N, K, fn, no_ep, st)
-                   : launch_staged<2, true, true>(xh, w0, w1, yh, M, N, K, fn, no_ep, st);
+        e = M <= 8 ? launch_staged<__half, 1, true, true>(xh, w0, w1, yh, M, N, K, fn, no_ep, st)
+                   : launch_staged<__half, 2, true, true>(xh, w0, w1, yh, M, N, K, fn, no_ep, st);
     else
-        e = M <= 8 ? launch_staged<1, false, true>(xh, w0, nullptr, yh, M, N, K, fn, no_ep, st)
-                   : launch_staged<2, false, true>(xh, w0, nullptr, yh, M, N, K, fn, no_ep, st);
+        e = M <= 8 ? launch_staged<__half, 1, false, true>(xh, w0, nullptr, yh, M, N, K, fn, no_ep, st)
+                   : launch_staged<__half, 2, false, true>(xh, w0, nullptr, yh, M, N, K, fn, no_ep, st);
     ONELLM_REQUIRE(e == cudaSuccess, ONELLM_ERR_CUDA, "add_residual_rmsnorm_gemm: %s", cudaGetErrorString(e));
     return ONELLM_OK;
 }

@@ -38,10 +38,10 @@ constexpr int kSkBarBytes = 256;
 
 // WIDE: one weight, 256 output columns per block (the second 128 where DUAL has its second weight): the activation
 // tile of a stage, a third of a narrow block's ring, then serves twice the weight bytes.
-template <bool DUAL, bool WIDE>
+template <typename T, bool DUAL, bool WIDE>
 __global__ void __launch_bounds__(kSkThreads)
 skinny_tc_kernel(const __grid_constant__ CUtensorMap map_w0, const __grid_constant__ CUtensorMap map_w1,
-                 const __grid_constant__ CUtensorMap map_x, __half* y, int M, int N, int K, int stages_per_block, int nst,
+                 const __grid_constant__ CUtensorMap map_x, T* y, int M, int N, int K, int stages_per_block, int nst,
                  const EpilogueArgs ep)
 {
     constexpr int NW = (DUAL || WIDE) ? 2 : 1;
@@ -118,8 +118,8 @@ skinny_tc_kernel(const __grid_constant__ CUtensorMap map_w0, const __grid_consta
     } else if (warp == 1) {
         pdl_wait();
         if (lane == 0) {
-            // D f32, A and B f16, A (weights) MN-major, B (activations) K-major, N = 64 tokens, M = 128 weight columns
-            const uint32_t idesc = (1u << 4) | (1u << 15) | ((uint32_t)(kSkTok >> 3) << 17) | ((uint32_t)(kBN >> 4) << 24);
+            // D f32, A and B of type T, A (weights) MN-major, B (activations) K-major, N = 64 tokens, M = 128 weight columns
+            const uint32_t idesc = (1u << 4) | umma_operand_bits<T>() | (1u << 15) | ((uint32_t)(kSkTok >> 3) << 17) | ((uint32_t)(kBN >> 4) << 24);
             bool ok = true;
             for (int it = 0; it < n_stages && ok; it++) {
                 const int s = it % nst;
@@ -158,7 +158,7 @@ skinny_tc_kernel(const __grid_constant__ CUtensorMap map_w0, const __grid_consta
 #pragma unroll
                 for (int i = 0; i < 4; i++) {
                     float v[8];
-                    Vec16<__half>::load(reinterpret_cast<const __half*>(xt + ((t >> 3) + 16 * i) * 128 + (t & 7) * 16), v);
+                    Vec16<T>::load(reinterpret_cast<const T*>(xt + ((t >> 3) + 16 * i) * 128 + (t & 7) * 16), v);
 #pragma unroll
                     for (int e = 0; e < 8; e++) ss[i] = fmaf(v[e], v[e], ss[i]);
                 }
@@ -205,7 +205,7 @@ skinny_tc_kernel(const __grid_constant__ CUtensorMap map_w0, const __grid_consta
     if (warp == 1) {
         asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem_base), "r"(kCols) : "memory");
     }
-    splitk_epilogue<kSkTok, DUAL, false, kSkThreads, WIDE>(reinterpret_cast<float*>(smem), cluster, y, M, N, K, n0, ep);
+    splitk_epilogue<T, kSkTok, DUAL, false, kSkThreads, WIDE>(reinterpret_cast<float*>(smem), cluster, y, M, N, K, n0, ep);
     cluster.sync();  // peers may still be reading this block's tile
 }
 
@@ -233,10 +233,10 @@ static const TunedTc kTunedTc[] = {
     {1920, 5120, false, 8, 6}, {5120, 640, false, 5, 3},  {1728, 5120, true, 8, 4}, {5120, 1728, false, 4, 4},  // 8 ways
 };
 
-template <bool DUAL, bool WIDE>
+template <typename T, bool DUAL, bool WIDE>
 static TcPlan plan_tc(int N, int K, bool tp)
 {
-    auto kern = skinny_tc_kernel<DUAL, WIDE>;
+    auto kern = skinny_tc_kernel<T, DUAL, WIDE>;
     constexpr int NW = (DUAL || WIDE) ? 2 : 1;
     constexpr int kTileCols = WIDE ? 2 * kBN : kBN;
     constexpr size_t stage = (size_t)NW * kSkWTile + kSkXTile;
@@ -369,19 +369,18 @@ static TcPlan plan_tc(int N, int K, bool tp)
     return plan;
 }
 
-template <bool DUAL, bool WIDE>
-static cudaError_t launch_tc(const __half* x, const __half* W0, const __half* W1, __half* y, int M, int N, int K, const EpilogueArgs& ep,
-                             cudaStream_t st)
+template <typename T, bool DUAL, bool WIDE>
+static cudaError_t launch_tc(const T* x, const T* W0, const T* W1, T* y, int M, int N, int K, const EpilogueArgs& ep, cudaStream_t st)
 {
     constexpr int kTileCols = WIDE ? 2 * kBN : kBN;
-    const TcPlan plan = plan_tc<DUAL, WIDE>(N, K, ep.tp.world > 1);
+    const TcPlan plan = plan_tc<T, DUAL, WIDE>(N, K, ep.tp.world > 1);
     if (plan.status != cudaSuccess) return plan.status;
     CUtensorMap map_w0, map_w1, map_x;
     if (make_map(&map_w0, W0, (uint64_t)N, (uint64_t)K, kSkBK) != ONELLM_OK) return cudaErrorInvalidValue;
     map_w1 = map_w0;
     if (DUAL && make_map(&map_w1, W1, (uint64_t)N, (uint64_t)K, kSkBK) != ONELLM_OK) return cudaErrorInvalidValue;
     if (make_map(&map_x, x, (uint64_t)K, (uint64_t)M, kSkTok) != ONELLM_OK) return cudaErrorInvalidValue;
-    (void)prefer_max_shared((const void*)skinny_tc_kernel<DUAL, WIDE>);
+    (void)prefer_max_shared((const void*)skinny_tc_kernel<T, DUAL, WIDE>);
     cudaLaunchConfig_t cfg = {};
     cudaLaunchAttribute attr[2];
     attr[0].id = cudaLaunchAttributeClusterDimension;
@@ -397,12 +396,12 @@ static cudaError_t launch_tc(const __half* x, const __half* W0, const __half* W1
     cfg.attrs = attr;
     cfg.numAttrs = 2;
     note_launch();
-    return cudaLaunchKernelEx(&cfg, skinny_tc_kernel<DUAL, WIDE>, map_w0, map_w1, map_x, y, M, N, K, plan.per_block, plan.nst, ep);
+    return cudaLaunchKernelEx(&cfg, skinny_tc_kernel<T, DUAL, WIDE>, map_w0, map_w1, map_x, y, M, N, K, plan.per_block, plan.nst, ep);
 }
 
 cudaError_t skinny_tc_plan_query(int N, int K, bool dual, int* ks, int* nst)
 {
-    const TcPlan p = dual ? plan_tc<true, false>(N, K, false) : plan_tc<false, false>(N, K, false);
+    const TcPlan p = dual ? plan_tc<__half, true, false>(N, K, false) : plan_tc<__half, false, false>(N, K, false);
     *ks = p.ks;
     *nst = p.nst;
     return p.status;
@@ -411,10 +410,10 @@ cudaError_t skinny_tc_plan_query(int N, int K, bool dual, int* ks, int* nst)
 // True when a projection of M tokens goes to this kernel rather than to the mma.sync one.
 bool skinny_tc_takes(int M, int N, int K) { return M >= g_tc_min_tokens && M <= kSkTok && K % 8 == 0 && N % 8 == 0; }
 
-cudaError_t skinny_tc_dispatch(const __half* x, const __half* W0, const __half* W1, __half* y, int M, int N, int K, const EpilogueArgs& ep,
-                               cudaStream_t st)
+template <typename T>
+cudaError_t skinny_tc_dispatch(const T* x, const T* W0, const T* W1, T* y, int M, int N, int K, const EpilogueArgs& ep, cudaStream_t st)
 {
-    if (W1) return launch_tc<true, false>(x, W0, W1, y, M, N, K, ep, st);
+    if (W1) return launch_tc<T, true, false>(x, W0, W1, y, M, N, K, ep, st);
     // 256-column blocks for a single weight: not with the tensor-parallel exchange in the epilogue, not where a plan of
     // the narrow kernel was tuned or is forced, and not where the narrow tiles outnumber the SMs (the LM head, which
     // runs as one wave of two narrow blocks per SM)
@@ -423,8 +422,12 @@ cudaError_t skinny_tc_dispatch(const __half* x, const __half* W0, const __half* 
     if (wide && plan_override_lookup(N, K, false, &oks, &onst)) wide = false;
     for (const TunedTc& t : kTunedTc)
         if (wide && g_tc_wide < 2 && t.N == N && t.K == K && !t.dual) wide = false;  // 2: sweeps compare against the tuned plans
-    return wide ? launch_tc<false, true>(x, W0, nullptr, y, M, N, K, ep, st) : launch_tc<false, false>(x, W0, nullptr, y, M, N, K, ep, st);
+    return wide ? launch_tc<T, false, true>(x, W0, nullptr, y, M, N, K, ep, st) : launch_tc<T, false, false>(x, W0, nullptr, y, M, N, K, ep, st);
 }
+template cudaError_t skinny_tc_dispatch<__half>(const __half*, const __half*, const __half*, __half*, int, int, int, const EpilogueArgs&,
+                                                cudaStream_t);
+template cudaError_t skinny_tc_dispatch<__nv_bfloat16>(const __nv_bfloat16*, const __nv_bfloat16*, const __nv_bfloat16*, __nv_bfloat16*,
+                                                       int, int, int, const EpilogueArgs&, cudaStream_t);
 
 int skinny_tc_flag() { return tc_flag_read_clear(); }
 

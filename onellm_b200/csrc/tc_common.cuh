@@ -57,6 +57,12 @@ __device__ __forceinline__ void umma_f16(uint32_t tmem_d, uint64_t adesc, uint64
         "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accumulate)
         : "memory");
 }
+// operand-type fields of a kind::f16 instruction descriptor (A and B always have the same type): 0 = f16, 1 = bf16
+template <typename T>
+__host__ __device__ constexpr uint32_t umma_operand_bits()
+{
+    return std::is_same<T, __nv_bfloat16>::value ? (1u << 7) | (1u << 10) : 0u;
+}
 __device__ __forceinline__ void umma_commit(uint32_t bar)
 {
     asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(bar) : "memory");
@@ -101,7 +107,7 @@ static inline int tc_flag_read_clear()
     return v;
 }
 
-// 2-D fp16 tensor map: `inner` contiguous elements, `outer` rows of `inner` elements; box {64, box_outer}; 128-byte swizzle
+// 2-D tensor map of 16-bit elements: `inner` contiguous elements, `outer` rows of `inner` elements; box {64, box_outer}; 128-byte swizzle
 // (defined in gemm_tc.cu)
 int make_map(CUtensorMap* map, const void* base, uint64_t inner, uint64_t outer, uint32_t box_outer);
 
