@@ -1,4 +1,4 @@
-"""onellm_b200: sm_100a kernels and a LLaMA decode engine behind oneLLM's kernel interface.
+"""onellm_b200: sm_100a kernels and a decoder engine behind oneLLM's kernel interface.
 
 This module is a thin ctypes binding of ``libonellm_b200.so`` (see ``include/onellm_b200.h``)
 for the tests and the benchmark.  It does no arithmetic itself and has no fallback: if the
@@ -13,7 +13,7 @@ import os
 _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(_HERE, "libonellm_b200.so")
 
-F32, F16 = 0, 1
+F32, F16, BF16 = 0, 1, 2
 W_KN, W_NK = 0, 1
 
 _lib = None
@@ -44,12 +44,11 @@ def lib() -> C.CDLL:
             raise OnellmError(-100, f"{LIB_PATH} is missing: run `python -m onellm_b200.build` "
                                     "(there is no CPU fallback)")
         l = C.CDLL(LIB_PATH)
-        l.onellm_last_error.restype = C.c_char_p
-        l.onellm_decode_attn_workspace_bytes.restype = C.c_size_t
-        l.onellm_decode_attn_static_scratch_bytes.restype = C.c_size_t
-        l.onellm_llama_device_bytes.restype = C.c_size_t
-        l.onellm_llama_stream.restype = C.c_void_p
-        l.onellm_llama_destroy.restype = None
+        for name, restype in (("onellm_last_error", C.c_char_p), ("onellm_decode_attn_workspace_bytes", C.c_size_t),
+                              ("onellm_decode_attn_static_scratch_bytes", C.c_size_t), ("onellm_llama_device_bytes", C.c_size_t),
+                              ("onellm_llama_stream", C.c_void_p), ("onellm_llama_destroy", None), ("onellm_model_design", C.c_char_p)):
+            if hasattr(l, name):  # a library built for one design has its entry points only
+                getattr(l, name).restype = restype
         _lib = l
     return _lib
 
@@ -348,27 +347,21 @@ def llama_config_from_ini(path, max_batch=1, max_seq_len=0, tp_rank=0, tp_size=1
     return cfg, top_k.value
 
 
-class Llama:
-    """Host-side handle of the C++ model (weights, KV cache, generation loop)."""
+class Engine:
+    """Host-side handle of a C++ model (weights, KV cache and other sequence state, generation loop), whatever its
+    design; made by Llama(...) or open_model(...)."""
 
-    @classmethod
-    def from_ini(cls, path, max_batch, max_seq_len, tp_rank=0, tp_size=1):
-        """The model described by the reference converter's config.ini (sampling set to the file's top_k)."""
-        self = cls.__new__(cls)
-        self.cfg, _ = llama_config_from_ini(path, max_batch, max_seq_len, tp_rank, tp_size)
-        self._h = C.c_void_p(0)
-        _check(lib().onellm_llama_create_from_ini(str(path).encode(), C.c_int(max_batch), C.c_int(max_seq_len), C.c_int(tp_rank),
-                                                  C.c_int(tp_size), C.byref(self._h)))
-        return self
+    _h = C.c_void_p(0)
 
-    def __init__(self, *, num_layers, hidden, head_num, kv_head_num, head_size, inter_size, vocab_size,
-                 max_seq_len, max_batch, rope_base=10000.0, rot_dim=0, rms_eps=1e-5, bos_id=1, eos_id=2,
-                 attn_bias=False, tp_rank=0, tp_size=1):
-        self.cfg = LlamaConfig(num_layers, hidden, head_num, kv_head_num, head_size, inter_size, vocab_size,
-                               max_seq_len, max_batch, rope_base, rot_dim, rms_eps, bos_id, eos_id,
-                               1 if attn_bias else 0, tp_rank, tp_size)
-        self._h = C.c_void_p(0)
-        _check(lib().onellm_llama_create(C.byref(self.cfg), C.byref(self._h)))
+    @property
+    def design(self):
+        return lib().onellm_model_design(self._h).decode()
+
+    def limits(self):
+        """(vocab_size, max_seq_len, max_batch)"""
+        v, s, b = C.c_int(0), C.c_int(0), C.c_int(0)
+        _check(lib().onellm_model_limits(self._h, C.byref(v), C.byref(s), C.byref(b)))
+        return v.value, s.value, b.value
 
     def close(self):
         if self._h:
@@ -389,33 +382,14 @@ class Llama:
     def stream(self):
         return int(lib().onellm_llama_stream(self._h) or 0)
 
-    def load_weights(self, prefix: str):
-        _check(lib().onellm_llama_load_weights(self._h, prefix.encode()))
-
     def init_random(self, seed: int, std: float = 0.02):
         _check(lib().onellm_llama_init_random(self._h, C.c_uint64(seed), C.c_float(std)))
-
-    def init_comm(self, unique_id: bytes):
-        _check(lib().onellm_llama_init_comm(self._h, C.c_char_p(unique_id)))
-
-    def p2p_handle(self) -> bytes:
-        buf = C.create_string_buffer(64)
-        _check(lib().onellm_llama_p2p_handle(self._h, buf))
-        return buf.raw
-
-    def p2p_connect(self, handles):
-        """handles: the 64-byte handles of all ranks, in rank order."""
-        blob = b"".join(handles)
-        _check(lib().onellm_llama_p2p_connect(self._h, C.c_char_p(blob)))
-
-    def p2p_error(self) -> int:
-        return int(lib().onellm_llama_p2p_error(self._h))
 
     def last_draws(self):
         """(u, step, table_in_use): the uniform draws of the last sampling launch (numpy float32 [max_batch]), the step
         counter that seeded them and whether the engine's skip-ahead table is in use."""
         import numpy as np
-        u = np.zeros(self.cfg.max_batch, np.float32)
+        u = np.zeros(self.limits()[2], np.float32)
         step, used = C.c_int(0), C.c_int(0)
         _check(lib().onellm_llama_last_draws(self._h, u.ctypes.data_as(C.c_void_p), C.byref(step), C.byref(used)))
         return u, step.value, bool(used.value)
@@ -423,9 +397,6 @@ class Llama:
     def set_sampling(self, top_k=1, temperature=1.0, literal_walk=False):
         _check(lib().onellm_llama_set_sampling(self._h, C.c_int(top_k), C.c_float(temperature),
                                                C.c_int(1 if literal_walk else 0)))
-
-    def set_tp_exchange(self, peer_memory: bool):
-        _check(lib().onellm_llama_set_tp_exchange(self._h, C.c_int(1 if peer_memory else 0)))
 
     def set_graphs(self, enabled: bool):
         _check(lib().onellm_llama_set_graphs(self._h, C.c_int(1 if enabled else 0)))
@@ -491,8 +462,21 @@ class Llama:
 
     def logits(self, batch):
         import numpy as np
-        out = np.zeros((batch, self.cfg.vocab_size), np.float32)
+        out = np.zeros((batch, self.limits()[0]), np.float32)
         _check(lib().onellm_llama_get_logits(self._h, out.ctypes.data_as(C.c_void_p)))
+        return out
+
+    def want_logits(self, rows):
+        """The next prefill / extend also computes the logits of these token rows (packed order of that call)."""
+        import numpy as np
+        rows = np.ascontiguousarray(rows, np.int32)
+        _check(lib().onellm_llama_want_logits(self._h, rows.ctypes.data_as(C.c_void_p), C.c_int(len(rows))))
+
+    def row_logits(self, n_rows):
+        """Logits of the rows asked for with want_logits, float32 [n_rows, vocab]."""
+        import numpy as np
+        out = np.zeros((n_rows, self.limits()[0]), np.float32)
+        _check(lib().onellm_llama_get_row_logits(self._h, out.ctypes.data_as(C.c_void_p), C.c_int(n_rows)))
         return out
 
     def state(self):
@@ -501,7 +485,70 @@ class Llama:
         _check(lib().onellm_llama_get_state(self._h, C.byref(cur), C.byref(launches), None, None))
         return cur.value, launches.value
 
+class Llama(Engine):
+    """The LLaMA design from a shape (weights from the reference's .bin files or random)."""
+
+    @classmethod
+    def from_ini(cls, path, max_batch, max_seq_len, tp_rank=0, tp_size=1):
+        """The model described by the reference converter's config.ini (sampling set to the file's top_k)."""
+        self = cls.__new__(cls)
+        self.cfg, _ = llama_config_from_ini(path, max_batch, max_seq_len, tp_rank, tp_size)
+        self._h = C.c_void_p(0)
+        _check(lib().onellm_llama_create_from_ini(str(path).encode(), C.c_int(max_batch), C.c_int(max_seq_len), C.c_int(tp_rank),
+                                                  C.c_int(tp_size), C.byref(self._h)))
+        return self
+
+    def __init__(self, *, num_layers, hidden, head_num, kv_head_num, head_size, inter_size, vocab_size,
+                 max_seq_len, max_batch, rope_base=10000.0, rot_dim=0, rms_eps=1e-5, bos_id=1, eos_id=2,
+                 attn_bias=False, tp_rank=0, tp_size=1):
+        self.cfg = LlamaConfig(num_layers, hidden, head_num, kv_head_num, head_size, inter_size, vocab_size,
+                               max_seq_len, max_batch, rope_base, rot_dim, rms_eps, bos_id, eos_id,
+                               1 if attn_bias else 0, tp_rank, tp_size)
+        self._h = C.c_void_p(0)
+        _check(lib().onellm_llama_create(C.byref(self.cfg), C.byref(self._h)))
+
+    def load_weights(self, prefix: str):
+        _check(lib().onellm_llama_load_weights(self._h, prefix.encode()))
+
+    def init_comm(self, unique_id: bytes):
+        _check(lib().onellm_llama_init_comm(self._h, C.c_char_p(unique_id)))
+
+    def p2p_handle(self) -> bytes:
+        buf = C.create_string_buffer(64)
+        _check(lib().onellm_llama_p2p_handle(self._h, buf))
+        return buf.raw
+
+    def p2p_connect(self, handles):
+        """handles: the 64-byte handles of all ranks, in rank order."""
+        blob = b"".join(handles)
+        _check(lib().onellm_llama_p2p_connect(self._h, C.c_char_p(blob)))
+
+    def p2p_error(self) -> int:
+        return int(lib().onellm_llama_p2p_error(self._h))
+
+    def set_tp_exchange(self, peer_memory: bool):
+        _check(lib().onellm_llama_set_tp_exchange(self._h, C.c_int(1 if peer_memory else 0)))
+
     def kv_cache_ptrs(self, layer):
         k, v = C.c_void_p(0), C.c_void_p(0)
         _check(lib().onellm_llama_kv_cache(self._h, C.c_int(layer), C.byref(k), C.byref(v)))
         return k.value, v.value
+
+
+class Model(Engine):
+    """A model of any registered design, from a folder (config.json, model.safetensors) or from a configuration."""
+
+    def __init__(self, source, dtype=BF16, max_batch=1, max_seq_len=0):
+        self._h = C.c_void_p(0)
+        if isinstance(source, dict):
+            import json
+            _check(lib().onellm_model_create(json.dumps(source).encode(), C.c_int(dtype), C.c_int(max_batch), C.c_int(max_seq_len),
+                                             C.byref(self._h)))
+        else:
+            _check(lib().onellm_model_open(str(source).encode(), C.c_int(dtype), C.c_int(max_batch), C.c_int(max_seq_len),
+                                           C.byref(self._h)))
+
+
+def open_model(folder, dtype=BF16, max_batch=1, max_seq_len=0) -> Model:
+    """The model in a folder; its config.json names the design.  max_seq_len 0: what the configuration allows."""
+    return Model(folder, dtype, max_batch, max_seq_len)

@@ -19,6 +19,12 @@ void set_error(const char* fmt, ...);
 void note_launch(int n = 1);
 long launches_noted();
 
+// Every file with kernels that have bounded waits registers the reader of its time-out flag (see tc_common.cuh);
+// onellm_gemm_timeout_flag asks them all.
+struct TimeoutFlag {
+    explicit TimeoutFlag(int (*read_and_clear)());
+};
+
 #define ONELLM_REQUIRE(cond, code, ...)          \
     do {                                         \
         if (!(cond)) {                           \

@@ -338,7 +338,7 @@ context_attn_tc_kernel(const __half* __restrict__ q, long q_ld, const __grid_con
     }
 }
 
-int attn_tc_timeout_flag() { return tc_flag_read_clear(); }
+static const TimeoutFlag timeout_flag(tc_flag_read_clear);
 
 // Context attention on tensor-core tiles; the caller has checked fp16, D = 128 and the standard cache order.
 int context_attn_tc_launch(const __half* q, long q_ld, const __half* k_cache, const __half* v_cache, int S_max, long cache_rows,

@@ -2,7 +2,7 @@
 //
 // Replace silu_and_mul_kernel (src/kernels/activation_kernel.cu:10-21) and embeddingFunctor
 // (src/kernels/input_embedding.cu:7-20) of the reference with 16-byte vectorised versions.
-#include "common.cuh"
+#include "mixers.h"
 
 namespace onellm {
 
@@ -115,3 +115,59 @@ extern "C" int onellm_embedding(int dtype, const int* ids, void* out, const void
     return embedding_launch(dtype, ids, out, nullptr, table, n_tokens, hidden, vocab, bad_id_flag, true,
                             reinterpret_cast<cudaStream_t>(stream));
 }
+
+namespace onellm {
+// Token embedding plus a learned position vector into a float residual stream:
+//     out[t] = table[id] + pos_table[position],   both tables [.., ld] of element type T
+// The position of token t: hist[b] + its index in sequence b (context pass: cu, hist), or step - 1 + off[t] (decode
+// step: one token per sequence).  Ids outside [0, vocab) raise bad[0], positions outside [0, max_pos) bad[1]; both give a
+// zero row.
+template <typename T>
+__global__ void __launch_bounds__(256)
+embedding_pos_kernel(const int* __restrict__ ids, float* __restrict__ out, const T* __restrict__ table, const T* __restrict__ pos_table, int ld,
+                     int vocab, int max_pos, const TokenPositions tp, int* __restrict__ bad)
+{
+    constexpr int VEC = Vec16<T>::N;
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x, id = ids[t];
+    int b, pos;
+    tp.locate(t, b, pos);
+    const bool id_ok = id >= 0 && id < vocab, pos_ok = pos >= 0 && pos < max_pos;
+    if (threadIdx.x == 0) {
+        if (!id_ok) atomicExch(bad, 1);
+        if (!pos_ok) atomicExch(bad + 1, 1);
+    }
+    for (int i = threadIdx.x; i < ld / VEC; i += blockDim.x) {
+        float a[VEC], p[VEC];
+#pragma unroll
+        for (int e = 0; e < VEC; e++) a[e] = p[e] = 0.f;
+        if (id_ok && pos_ok) {
+            Vec16<T>::load(table + (size_t)id * ld + (size_t)i * VEC, a);
+            Vec16<T>::load(pos_table + (size_t)pos * ld + (size_t)i * VEC, p);
+        }
+        float4* dst = reinterpret_cast<float4*>(out + (size_t)t * ld + (size_t)i * VEC);
+#pragma unroll
+        for (int e = 0; e < VEC; e += 4) dst[e / 4] = make_float4(a[e] + p[e], a[e + 1] + p[e + 1], a[e + 2] + p[e + 2], a[e + 3] + p[e + 3]);
+    }
+}
+
+// Launched with a full stream dependency (first kernel behind the step counter / the id upload).
+int embedding_pos_launch(int dtype, const int* ids, float* out, const void* table, const void* pos_table, int n_tokens, int ld, int vocab,
+                         int max_pos, const TokenPositions& tp, int* bad, cudaStream_t st)
+{
+    ONELLM_REQUIRE(ids && out && table && pos_table && bad && ld % 8 == 0, ONELLM_ERR_ARG, "embedding_pos: bad argument");
+    if (n_tokens <= 0) return ONELLM_OK;
+    note_launch();
+    if (dtype == ONELLM_F32) {
+        (void)prefer_max_shared((const void*)embedding_pos_kernel<float>);
+        embedding_pos_kernel<float><<<n_tokens, 256, 0, st>>>(ids, out, (const float*)table, (const float*)pos_table, ld, vocab, max_pos, tp, bad);
+    } else {
+        (void)prefer_max_shared((const void*)embedding_pos_kernel<__nv_bfloat16>);
+        embedding_pos_kernel<__nv_bfloat16><<<n_tokens, 256, 0, st>>>(ids, out, (const __nv_bfloat16*)table, (const __nv_bfloat16*)pos_table, ld,
+                                                                     vocab, max_pos, tp, bad);
+    }
+    ONELLM_CHECK_LAUNCH();
+    return ONELLM_OK;
+}
+}  // namespace onellm

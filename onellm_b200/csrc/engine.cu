@@ -104,8 +104,7 @@ int Engine::allocate()
     carve_common(real);
     carve(real);
     ONELLM_CUDA(cudaStreamCreateWithFlags(&stream, cudaStreamNonBlocking));
-    ONELLM_CUDA(cudaMemsetAsync(d_step, 0, 4 * sizeof(int), stream));
-    ONELLM_CUDA(cudaMemsetAsync(d_bad_id, 0, 4 * sizeof(int), stream));
+    ONELLM_CUDA(cudaMemsetAsync(arena, 0, arena_bytes, stream));
     ONELLM_CUDA(cudaStreamSynchronize(stream));
     return build_skip_table(d_skip, max_batch, &skip_ok, stream);
 }

@@ -5,6 +5,7 @@
 #include <mutex>
 #include <set>
 #include <utility>
+#include <vector>
 
 #include "common.cuh"
 
@@ -38,7 +39,25 @@ cudaError_t prefer_max_shared(const void* kernel)
     return e;
 }
 
+static std::vector<int (*)()>& timeout_flags()
+{
+    static std::vector<int (*)()> v;
+    return v;
+}
+TimeoutFlag::TimeoutFlag(int (*read_and_clear)()) { timeout_flags().push_back(read_and_clear); }
+
 }  // namespace onellm
+
+// 1 when a tensor-core block (projection or attention) gave up a bounded wait since the last call.
+extern "C" int onellm_gemm_timeout_flag(void)
+{
+    int any = 0;
+    for (auto read : onellm::timeout_flags()) {
+        const int v = read();
+        any = (v < 0 || any < 0) ? -1 : (any | v);
+    }
+    return any;
+}
 
 extern "C" const char* onellm_last_error(void) { return onellm::g_err; }
 

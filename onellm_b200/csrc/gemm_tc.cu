@@ -396,16 +396,6 @@ int gemm_bf16_large(const __nv_bfloat16* x, const __nv_bfloat16* W, const __nv_b
     return gemm_tc_launch<__nv_bfloat16>(x, W, W2, static_cast<__nv_bfloat16*>(y), M, N, K, W2 ? 2 : 0, st, epi);
 }
 
-int attn_tc_timeout_flag();  // context_attn_tc.cu
-int skinny_tc_flag();         // skinny_gemm_tc.cu
-
-// 1 when a tensor-core block (projection or context attention) gave up a bounded wait since the last call.
-int gemm_tc_timeout_flag()
-{
-    const int a = tc_flag_read_clear(), b = attn_tc_timeout_flag(), c = skinny_tc_flag();
-    return (a < 0 || b < 0 || c < 0) ? -1 : (a | b | c);
-}
+static const TimeoutFlag timeout_flag(tc_flag_read_clear);
 
 }  // namespace onellm
-
-extern "C" int onellm_gemm_timeout_flag(void) { return onellm::gemm_tc_timeout_flag(); }

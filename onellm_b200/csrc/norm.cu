@@ -170,6 +170,71 @@ extern "C" int onellm_row_sumsq(int dtype, const void* x, int rows, int cols, fl
     return ONELLM_OK;
 }
 
+namespace onellm {
+// RMSNorm with weights stored around zero, out of a float residual stream: for row r (or rows[r]) of x
+//     out_i[r] = x * rsqrt(mean(x^2) + eps) * (1 + w_i)          i = 1, 2 (out2 may be NULL)
+// into one or two buffers of element type T: two parallel branches that normalise the same stream with weights of their
+// own share one pass over it.  `width` columns count, `ld` is the row stride of all buffers (the columns behind `width`
+// hold zeros and get zeros).
+constexpr int kPairVec = 8;  // float4 per thread kept in registers
+template <typename T>
+__global__ void __launch_bounds__(kNormThreads)
+norm_pair_kernel(const float* __restrict__ x, const int* __restrict__ rows, const float* __restrict__ w1, const float* __restrict__ w2,
+                 T* __restrict__ out1, T* __restrict__ out2, float eps, int width, int ld)
+{
+    pdl_launch_dependents();
+    pdl_wait();
+    const float4* xr = reinterpret_cast<const float4*>(x + (size_t)(rows ? rows[blockIdx.x] : blockIdx.x) * ld);
+    const int nvec = ld / 4;
+    float4 keep[kPairVec];
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < kPairVec; j++) {
+        const int i = threadIdx.x + j * kNormThreads;
+        if (i < nvec) {
+            keep[j] = xr[i];
+            ss = fmaf(keep[j].x, keep[j].x, fmaf(keep[j].y, keep[j].y, fmaf(keep[j].z, keep[j].z, fmaf(keep[j].w, keep[j].w, ss))));
+        }
+    }
+    for (int i = threadIdx.x + kPairVec * kNormThreads; i < nvec; i += kNormThreads) {
+        const float4 v = xr[i];
+        ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+    }
+    const float inv = 1.0f / sqrtf(block_sum_256(ss) / (float)width + eps);
+    auto emit = [&](int i, const float4& v) {
+        auto one = [&](const float* w, T* out) {
+            const float4 g = reinterpret_cast<const float4*>(w)[i];
+            const float o[4] = {v.x * inv * (1.f + g.x), v.y * inv * (1.f + g.y), v.z * inv * (1.f + g.z), v.w * inv * (1.f + g.w)};
+            T* dst = out + (size_t)blockIdx.x * ld + 4 * i;
+            if constexpr (std::is_same<T, float>::value) *reinterpret_cast<float4*>(dst) = make_float4(o[0], o[1], o[2], o[3]);
+            else *reinterpret_cast<uint2*>(dst) = make_uint2(pack2<T>(o[0], o[1]), pack2<T>(o[2], o[3]));
+        };
+        one(w1, out1);
+        if (out2) one(w2, out2);
+    };
+#pragma unroll
+    for (int j = 0; j < kPairVec; j++) {
+        const int i = threadIdx.x + j * kNormThreads;
+        if (i < nvec) emit(i, keep[j]);
+    }
+    for (int i = threadIdx.x + kPairVec * kNormThreads; i < nvec; i += kNormThreads) emit(i, xr[i]);
+}
+
+int norm_pair(int dtype, const float* x, const int* rows, int n_rows, const float* w1, const float* w2, void* out1, void* out2, float eps,
+              int width, int ld, cudaStream_t st)
+{
+    ONELLM_REQUIRE(x && w1 && out1 && ld % 4 == 0 && width > 0 && width <= ld, ONELLM_ERR_ARG, "norm_pair: bad argument");
+    if (n_rows <= 0) return ONELLM_OK;
+    if (dtype == ONELLM_F32)
+        ONELLM_CUDA(launch_pdl(norm_pair_kernel<float>, dim3(n_rows), dim3(kNormThreads), 0, st, x, rows, w1, w2, (float*)out1, (float*)out2,
+                               eps, width, ld));
+    else
+        ONELLM_CUDA(launch_pdl(norm_pair_kernel<__nv_bfloat16>, dim3(n_rows), dim3(kNormThreads), 0, st, x, rows, w1, w2, (__nv_bfloat16*)out1,
+                               (__nv_bfloat16*)out2, eps, width, ld));
+    return ONELLM_OK;
+}
+}  // namespace onellm
+
 extern "C" int onellm_rmsnorm(int dtype, void* x, const void* gamma, float eps, int num_tokens, int hidden,
                               void* stream)
 {

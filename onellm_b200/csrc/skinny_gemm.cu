@@ -9,7 +9,8 @@
 #include <mutex>
 #include <utility>
 
-#include "common.cuh"
+#include "project.h"
+#include "skinny_common.cuh"
 
 namespace onellm {
 
@@ -85,9 +86,11 @@ skinny_nk_kernel(const __half* __restrict__ x, const __half* __restrict__ W, __h
 
 // Plain fp32 projection for the reference's own dtype: 64x64 tiles, 16x16 threads, 4x4 outputs
 // per thread.  Correctness path for fp32 callers, not a tuned kernel.
+// resid (row stride ldy, may be y): y = resid + result.  gate >= 0: y holds the gate product of a gated pair and becomes
+// act(y) * result.
 template <bool W_NK>
 __global__ void __launch_bounds__(256)
-sgemm_kernel(const float* __restrict__ x, const float* __restrict__ W, float* __restrict__ y, int M, int N, int K, long ldy)
+sgemm_kernel(const float* __restrict__ x, const float* __restrict__ W, float* y, int M, int N, int K, long ldy, const float* resid, int gate)
 {
     __shared__ float xs[16][64 + 1];
     __shared__ float ws[16][64 + 1];
@@ -129,7 +132,14 @@ sgemm_kernel(const float* __restrict__ x, const float* __restrict__ W, float* __
 #pragma unroll
         for (int j = 0; j < 4; j++) {
             const int m = m0 + ty * 4 + i, n = n0 + tx * 4 + j;
-            if (m < M && n < N) y[(size_t)m * ldy + n] = acc[i][j];
+            if (m < M && n < N) {
+                const size_t at = (size_t)m * ldy + n;
+                float v = acc[i][j];
+                if (resid) v += resid[at];
+                if (gate == GATE_RELU) v *= fmaxf(y[at], 0.f);
+                else if (gate == GATE_SILU) v *= y[at] / (1.0f + expf(-y[at]));
+                y[at] = v;
+            }
         }
 }
 
@@ -229,9 +239,9 @@ extern "C" int onellm_gemm_ld(int dtype, const void* x, const void* W, void* y, 
         ONELLM_REQUIRE(grid.y <= 65535, ONELLM_ERR_UNSUPPORTED, "gemm: M too large for the fp32 path");
         note_launch();
         if (w_layout == ONELLM_W_NK)
-            sgemm_kernel<true><<<grid, 256, 0, st>>>((const float*)x, (const float*)W, (float*)y, M, N, K, ldy);
+            sgemm_kernel<true><<<grid, 256, 0, st>>>((const float*)x, (const float*)W, (float*)y, M, N, K, ldy, nullptr, -1);
         else
-            sgemm_kernel<false><<<grid, 256, 0, st>>>((const float*)x, (const float*)W, (float*)y, M, N, K, ldy);
+            sgemm_kernel<false><<<grid, 256, 0, st>>>((const float*)x, (const float*)W, (float*)y, M, N, K, ldy, nullptr, -1);
         ONELLM_CHECK_LAUNCH();
         return ONELLM_OK;
     }
@@ -253,6 +263,46 @@ extern "C" int onellm_gemm(int dtype, const void* x, const void* W, void* y, int
 }
 
 namespace onellm {
+// project.h: one projection of a model design, any token count, bfloat16 or float
+template <typename T>
+cudaError_t skinny_kn_project(const T* x, const T* W0, const T* W1, T* y, int M, int N, int K, const EpilogueArgs& ep, cudaStream_t st);
+extern template cudaError_t skinny_kn_project<__nv_bfloat16>(const __nv_bfloat16*, const __nv_bfloat16*, const __nv_bfloat16*,
+                                                             __nv_bfloat16*, int, int, int, const EpilogueArgs&, cudaStream_t);
+int gemm_bf16_large(const __nv_bfloat16* x, const __nv_bfloat16* W, const __nv_bfloat16* W2, void* y, long ldy, int M, int N, int K, int act,
+                    int f32, const float* resid, cudaStream_t st);
+
+int project(const Projection& p, cudaStream_t st)
+{
+    ONELLM_REQUIRE(p.x && p.W && p.y && p.N > 0 && p.K > 0 && p.M >= 0, ONELLM_ERR_ARG, "project: bad argument");
+    const long ldy = p.ldy ? p.ldy : p.N;
+    if (p.M == 0) return ONELLM_OK;
+    if (p.dtype == ONELLM_F32) {
+        const dim3 grid((p.N + 63) / 64, (p.M + 63) / 64);
+        ONELLM_REQUIRE(grid.y <= 65535, ONELLM_ERR_UNSUPPORTED, "project: too many rows for the fp32 path");
+        ONELLM_CUDA(launch_pdl(sgemm_kernel<false>, grid, dim3(256), 0, st, (const float*)p.x, (const float*)p.W, (float*)p.y, p.M, p.N, p.K,
+                               ldy, p.W2 ? nullptr : p.resid, -1));
+        if (p.W2)
+            ONELLM_CUDA(launch_pdl(sgemm_kernel<false>, grid, dim3(256), 0, st, (const float*)p.x, (const float*)p.W2, (float*)p.y, p.M, p.N,
+                                   p.K, ldy, (const float*)nullptr, p.act));
+        return ONELLM_OK;
+    }
+    ONELLM_REQUIRE(p.dtype == ONELLM_BF16, ONELLM_ERR_UNSUPPORTED, "project: dtype %d", p.dtype);
+    ONELLM_REQUIRE(p.K % 16 == 0 && p.N % 8 == 0 && ldy % 8 == 0, ONELLM_ERR_UNSUPPORTED, "project: need K %% 16 == 0, N and ldy %% 8 == 0");
+    ONELLM_REQUIRE(aligned16(p.x) && aligned16(p.W) && aligned16(p.W2) && aligned16(p.y) && aligned16(p.resid), ONELLM_ERR_ARG,
+                   "project: pointers must be 16-byte aligned");
+    typedef __nv_bfloat16 bf16;
+    if (p.M > 64)
+        return gemm_bf16_large((const bf16*)p.x, (const bf16*)p.W, (const bf16*)p.W2, p.y, ldy, p.M, p.N, p.K, p.act, p.f32, p.resid, st);
+    EpilogueArgs ep = {};
+    ep.resid = p.resid;
+    ep.early_dependents = 1;
+    ep.act = p.act;
+    ep.ldy = ldy;
+    ep.f32 = p.f32;
+    ONELLM_CUDA(skinny_kn_project<bf16>((const bf16*)p.x, (const bf16*)p.W, (const bf16*)p.W2, (bf16*)p.y, p.M, p.N, p.K, ep, st));
+    return ONELLM_OK;
+}
+
 cudaError_t staged_plan_query(int M, int N, int K, bool dual, int* ks, int* nst, int* blocks);
 void staged_plan_override(int N, int K, bool dual, int ks, int nst);
 }  // namespace onellm

@@ -429,7 +429,7 @@ template cudaError_t skinny_tc_dispatch<__half>(const __half*, const __half*, co
 template cudaError_t skinny_tc_dispatch<__nv_bfloat16>(const __nv_bfloat16*, const __nv_bfloat16*, const __nv_bfloat16*, __nv_bfloat16*,
                                                        int, int, int, const EpilogueArgs&, cudaStream_t);
 
-int skinny_tc_flag() { return tc_flag_read_clear(); }
+static const TimeoutFlag timeout_flag(tc_flag_read_clear);
 
 }  // namespace onellm
 
