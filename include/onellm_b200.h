@@ -460,6 +460,93 @@ ONELLM_API int onellm_p2p_error(onellm_p2p* comm);
 ONELLM_API void onellm_p2p_destroy(onellm_p2p* comm);
 
 /* ---------------------------------------------------------------------------------------
+ * Mechanisms of the designs behind onellm_model_open (no counterpart in the reference).  Element type dtype: BF16 or
+ * F32 (then everything is true 32-bit).  Rows start at multiples of 16 bytes.
+ * ------------------------------------------------------------------------------------- */
+/* Where the tokens of a launch belong.  Context pass: cu [B+1] token offsets and hist [B] cached positions, tokens packed
+ * in sequence order.  Decode step (cu NULL): token t belongs to sequence t, at position *step - 1 + off[t].  All device
+ * pointers, complete before the kernel in front of the launch began. */
+typedef struct onellm_token_positions {
+    const int* cu;
+    const int* hist;
+    int B;
+    const int* step;
+    const int* off;
+} onellm_token_positions;
+
+/* Causal attention with key size dk and value size dv (multiples of 16, at most 256), H query heads over G key/value
+ * heads (head h reads h / (H / G)).  The score of a key d positions back, for a query at position p, is
+ *     (q . k) * q_factor[p] - penalty[h * S + d]          in units of log2.
+ * q, k, v: projections of the tokens, token t at + t * ld, heads dk / dv elements apart.  k_cache [B, G, S, dk], v_cache
+ * [B, G, S, dv].  out: token t, head h at + t * out_ld + h * dv, multiplied by out_scale. */
+typedef struct onellm_biased_attn {
+    int dtype;
+    int H, G, dk, dv;
+    const void *q, *k, *v;
+    long ld;
+    void *k_cache, *v_cache;
+    int S;
+    const float* q_factor; /* [S] */
+    const float* penalty;  /* [H, S] */
+    void* out;
+    long out_ld;
+    float out_scale;
+} onellm_biased_attn;
+/* q_factor[p] = scale * (1 + coef * ln(floor((p + 1) / every) + 1)) * log2(e) */
+ONELLM_API int onellm_query_factor(float* out, int S, double scale, double coef, double every, void* stream);
+/* penalty[h, d] = r1[h] * ln(1 + r2[h] * d) * log2(e) */
+ONELLM_API int onellm_distance_penalty(float* out, const float* r1, const float* r2, int H, int S, void* stream);
+/* Keys and values of `tokens` tokens into the cache; a position outside [0, S) is dropped and raises *overflow. */
+ONELLM_API int onellm_biased_attn_store(const onellm_biased_attn* a, const onellm_token_positions* tp, int tokens, int* overflow,
+                                        void* stream);
+/* Attention of `tokens` tokens over the cache, their own rows stored before.  max_new: most tokens of one sequence.
+ * BF16 context passes run on tensor cores unless `plain`. */
+ONELLM_API int onellm_biased_attn_context(const onellm_biased_attn* a, const onellm_token_positions* tp, int tokens, int max_new, int plain,
+                                          void* stream);
+/* Decode step (BF16): stores the new keys and values and attends.  step_bound: an upper bound of *tp->step. */
+ONELLM_API size_t onellm_biased_attn_decode_workspace(int B, int H, int dv);
+ONELLM_API int onellm_biased_attn_decode(const onellm_biased_attn* a, const onellm_token_positions* tp, int step_bound, void* workspace,
+                                         void* stream);
+
+/* Gated outer-product recurrence with a float state, per sequence and head (dk a multiple of 16, dv of 32, at most 256):
+ *     f = lower + (1 - lower) * sigmoid(z + zb)     state = diag(f) state + (1 - f) v^T     o = state^T silu(q)
+ *     out = o * rsqrt(sum(o^2) / norm_width + eps) * w * out_scale
+ * q, z, v: token t at + t * ld, heads dk / dk / dv apart; zb, lower [H * dk]; w [dv]; state [B, H, dk, dv], taken as zero
+ * for a sequence with hist 0. */
+typedef struct onellm_gated_recurrence {
+    int dtype;
+    int H, dk, dv;
+    const void *q, *z, *v;
+    long ld;
+    const float *zb, *lower;
+    const float* w;
+    float eps;
+    int norm_width;
+    float* state;
+    void* out;
+    long out_ld;
+    float out_scale;
+} onellm_gated_recurrence;
+ONELLM_API int onellm_gated_recurrence_run(const onellm_gated_recurrence* g, const onellm_token_positions* tp, int B, void* stream);
+
+/* RMSNorm with weights stored around zero, out of a float stream into one or two buffers (out2 may be NULL):
+ *     out_i[r] = x[r or rows[r]] * rsqrt(mean(x^2) + eps) * (1 + w_i)
+ * `width` columns count; ld is the row stride of every buffer, the columns behind width hold zeros. */
+ONELLM_API int onellm_norm_pair(int dtype, const float* x, const int* rows, int n_rows, const float* w1, const float* w2, void* out1,
+                                void* out2, float eps, int width, int ld, void* stream);
+
+/* Projection of any number of tokens, W and W2 [K,N]:  y = x.W,  y = act(x.W) * (x.W2)  (W2 given),  y = resid + x.W  (resid
+ * given, float, with f32).  f32: y is float.  ldy: row stride of y and resid (0: N).  BF16: K % 16 == 0, N and ldy % 8 == 0. */
+enum onellm_gate_act { ONELLM_GATE_SILU = 0, ONELLM_GATE_RELU = 1 };
+ONELLM_API int onellm_project(int dtype, const void* x, const void* W, const void* W2, void* y, long ldy, int M, int N, int K, int act, int f32,
+                              const float* resid, void* stream);
+
+/* out[t] = table[ids[t]] + pos_table[position of t] in float, rows of ld elements.  A bad id raises bad[0], a position
+ * outside [0, max_pos) bad[1]; the row is zero then. */
+ONELLM_API int onellm_embedding_pos(int dtype, const int* ids, float* out, const void* table, const void* pos_table, int n_tokens, int ld,
+                                    int vocab, int max_pos, const onellm_token_positions* tp, int* bad, void* stream);
+
+/* ---------------------------------------------------------------------------------------
  * LLaMA model: weights, KV cache and the generation loop (host side in C++).
  * Fills in the model class the reference leaves empty (src/models/llama/llama.h, outline in
  * src/models/llama/llama.cpp:1-50) with the kernel order of LlamaSelfDecoder::forward

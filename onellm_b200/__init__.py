@@ -36,6 +36,27 @@ class LlamaConfig(C.Structure):
     ]
 
 
+class TokenPositions(C.Structure):
+    """onellm_token_positions: cu / hist of a context pass, or step / off of a decode step (device addresses)."""
+    _fields_ = [("cu", C.c_void_p), ("hist", C.c_void_p), ("B", C.c_int), ("step", C.c_void_p), ("off", C.c_void_p)]
+
+
+class BiasedAttn(C.Structure):
+    """onellm_biased_attn (device addresses)."""
+    _fields_ = [("dtype", C.c_int), ("H", C.c_int), ("G", C.c_int), ("dk", C.c_int), ("dv", C.c_int),
+                ("q", C.c_void_p), ("k", C.c_void_p), ("v", C.c_void_p), ("ld", C.c_long),
+                ("k_cache", C.c_void_p), ("v_cache", C.c_void_p), ("S", C.c_int),
+                ("q_factor", C.c_void_p), ("penalty", C.c_void_p), ("out", C.c_void_p), ("out_ld", C.c_long), ("out_scale", C.c_float)]
+
+
+class GatedRecurrence(C.Structure):
+    """onellm_gated_recurrence (device addresses)."""
+    _fields_ = [("dtype", C.c_int), ("H", C.c_int), ("dk", C.c_int), ("dv", C.c_int),
+                ("q", C.c_void_p), ("z", C.c_void_p), ("v", C.c_void_p), ("ld", C.c_long), ("zb", C.c_void_p), ("lower", C.c_void_p),
+                ("w", C.c_void_p), ("eps", C.c_float), ("norm_width", C.c_int), ("state", C.c_void_p),
+                ("out", C.c_void_p), ("out_ld", C.c_long), ("out_scale", C.c_float)]
+
+
 def lib() -> C.CDLL:
     """Loads the CUDA library; raises if it has not been built."""
     global _lib
@@ -46,7 +67,8 @@ def lib() -> C.CDLL:
         l = C.CDLL(LIB_PATH)
         for name, restype in (("onellm_last_error", C.c_char_p), ("onellm_decode_attn_workspace_bytes", C.c_size_t),
                               ("onellm_decode_attn_static_scratch_bytes", C.c_size_t), ("onellm_llama_device_bytes", C.c_size_t),
-                              ("onellm_llama_stream", C.c_void_p), ("onellm_llama_destroy", None), ("onellm_model_design", C.c_char_p)):
+                              ("onellm_llama_stream", C.c_void_p), ("onellm_llama_destroy", None), ("onellm_model_design", C.c_char_p),
+                              ("onellm_biased_attn_decode_workspace", C.c_size_t)):
             if hasattr(l, name):  # a library built for one design has its entry points only
                 getattr(l, name).restype = restype
         _lib = l
@@ -288,6 +310,53 @@ def topk_sample(topk_id, topk_val, B, K, temperature, rng_step, vocab_size, end_
                                     _p(u_out), _stream(stream)))
 
 
+GATE_SILU, GATE_RELU = 0, 1
+
+
+def query_factor(out, S, scale, coef, every, stream=None):
+    _check(lib().onellm_query_factor(_p(out), C.c_int(S), C.c_double(scale), C.c_double(coef), C.c_double(every), _stream(stream)))
+
+
+def distance_penalty(out, r1, r2, H, S, stream=None):
+    _check(lib().onellm_distance_penalty(_p(out), _p(r1), _p(r2), C.c_int(H), C.c_int(S), _stream(stream)))
+
+
+def biased_attn_store(a, tp, tokens, overflow=None, stream=None):
+    _check(lib().onellm_biased_attn_store(C.byref(a), C.byref(tp), C.c_int(tokens), _p(overflow), _stream(stream)))
+
+
+def biased_attn_context(a, tp, tokens, max_new, plain=False, stream=None):
+    _check(lib().onellm_biased_attn_context(C.byref(a), C.byref(tp), C.c_int(tokens), C.c_int(max_new), C.c_int(1 if plain else 0),
+                                            _stream(stream)))
+
+
+def biased_attn_decode_workspace(B, H, dv):
+    return int(lib().onellm_biased_attn_decode_workspace(C.c_int(B), C.c_int(H), C.c_int(dv)))
+
+
+def biased_attn_decode(a, tp, step_bound, workspace, stream=None):
+    _check(lib().onellm_biased_attn_decode(C.byref(a), C.byref(tp), C.c_int(step_bound), _p(workspace), _stream(stream)))
+
+
+def gated_recurrence(g, tp, B, stream=None):
+    _check(lib().onellm_gated_recurrence_run(C.byref(g), C.byref(tp), C.c_int(B), _stream(stream)))
+
+
+def norm_pair(dtype, x, rows, n_rows, w1, w2, out1, out2, eps, width, ld, stream=None):
+    _check(lib().onellm_norm_pair(C.c_int(dtype), _p(x), _p(rows), C.c_int(n_rows), _p(w1), _p(w2), _p(out1), _p(out2), C.c_float(eps),
+                                  C.c_int(width), C.c_int(ld), _stream(stream)))
+
+
+def project(dtype, x, W, W2, y, M, N, K, ldy=0, act=GATE_SILU, f32=False, resid=None, stream=None):
+    _check(lib().onellm_project(C.c_int(dtype), _p(x), _p(W), _p(W2), _p(y), C.c_long(ldy), C.c_int(M), C.c_int(N), C.c_int(K),
+                                C.c_int(act), C.c_int(1 if f32 else 0), _p(resid), _stream(stream)))
+
+
+def embedding_pos(dtype, ids, out, table, pos_table, n_tokens, ld, vocab, max_pos, tp, bad, stream=None):
+    _check(lib().onellm_embedding_pos(C.c_int(dtype), _p(ids), _p(out), _p(table), _p(pos_table), C.c_int(n_tokens), C.c_int(ld),
+                                      C.c_int(vocab), C.c_int(max_pos), C.byref(tp), _p(bad), _stream(stream)))
+
+
 def p2p_two_shot_bytes(nbytes=-1):
     """Threshold (one-shot wire bytes per rank) from which the projections' exchange goes two-shot; returns the previous one."""
     f = lib().onellm_p2p_two_shot_bytes
@@ -484,6 +553,7 @@ class Engine:
         launches = C.c_long(0)
         _check(lib().onellm_llama_get_state(self._h, C.byref(cur), C.byref(launches), None, None))
         return cur.value, launches.value
+
 
 class Llama(Engine):
     """The LLaMA design from a shape (weights from the reference's .bin files or random)."""

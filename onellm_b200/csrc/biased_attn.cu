@@ -49,7 +49,7 @@ __global__ void __launch_bounds__(128) biased_attn_store_kernel(const BiasedAttn
     pdl_wait();
     const int t = blockIdx.x;
     int b, pos;
-    tp.locate(t, b, pos);
+    locate(tp, t, b, pos);
     if (pos < 0 || pos >= a.S) {
         if (threadIdx.x == 0 && overflow) atomicExch(overflow, 1);
         return;
@@ -86,7 +86,7 @@ __global__ void __launch_bounds__(128) biased_attn_plain_kernel(const BiasedAttn
     const int t = blockIdx.x, h = blockIdx.y * 4 + warp;
     if (h >= a.H) return;
     int b, pos;
-    tp.locate(t, b, pos);
+    locate(tp, t, b, pos);
     if (pos < 0 || pos >= a.S) return;
     const int g = h / (a.H / a.G);
     const T* q = reinterpret_cast<const T*>(a.q) + (size_t)t * a.ld + (size_t)h * a.dk;
@@ -202,7 +202,7 @@ __global__ void __launch_bounds__(kBdWarps * 32) biased_attn_decode_kernel(const
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
 
     int bb, n_cached;  // the query's position = rows already in the cache
-    p.tp.locate(b, bb, n_cached);
+    locate(p.tp, b, bb, n_cached);
     const int n_split = bd_splits(n_cached, p.chunk);
     if (split >= n_split || n_cached < 0 || n_cached >= p.a.S) {
         pdl_launch_dependents();
@@ -409,7 +409,7 @@ __global__ void __launch_bounds__(128) biased_attn_merge_kernel(const BdParams p
     pdl_wait();
     const int h = blockIdx.x, b = blockIdx.y, dv = p.a.dv;
     int bb, n_cached;
-    p.tp.locate(b, bb, n_cached);
+    locate(p.tp, b, bb, n_cached);
     const int n_split = bd_splits(n_cached, p.chunk);
     if (n_split == 1) return;  // the attention kernel wrote the output itself
     const size_t base = ((size_t)b * p.a.H + h) * p.n_split;
@@ -491,3 +491,41 @@ int biased_attn_decode(const BiasedAttn& a, const TokenPositions& tp, int step_b
 }
 
 }  // namespace onellm
+
+using namespace onellm;
+
+extern "C" int onellm_query_factor(float* out, int S, double scale, double coef, double every, void* stream)
+{
+    ONELLM_REQUIRE(out && S > 0 && every > 0.0, ONELLM_ERR_ARG, "query_factor: bad argument");
+    return build_query_factor(out, S, scale, coef, every, reinterpret_cast<cudaStream_t>(stream));
+}
+
+extern "C" int onellm_distance_penalty(float* out, const float* r1, const float* r2, int H, int S, void* stream)
+{
+    ONELLM_REQUIRE(out && r1 && r2 && H > 0 && H <= 65535 && S > 0, ONELLM_ERR_ARG, "distance_penalty: bad argument");
+    return build_distance_penalty(out, r1, r2, H, S, reinterpret_cast<cudaStream_t>(stream));
+}
+
+extern "C" int onellm_biased_attn_store(const onellm_biased_attn* a, const onellm_token_positions* tp, int tokens, int* overflow, void* stream)
+{
+    ONELLM_REQUIRE(a && tp && a->k && a->v, ONELLM_ERR_ARG, "biased_attn_store: null pointer");
+    const int rc = check_attn(*a);
+    if (rc) return rc;
+    return biased_attn_store(*a, *tp, tokens, overflow, reinterpret_cast<cudaStream_t>(stream));
+}
+
+extern "C" int onellm_biased_attn_context(const onellm_biased_attn* a, const onellm_token_positions* tp, int tokens, int max_new, int plain,
+                                          void* stream)
+{
+    ONELLM_REQUIRE(a && tp && tokens >= 0 && max_new >= 0, ONELLM_ERR_ARG, "biased_attn_context: bad argument");
+    return biased_attn_context(*a, *tp, tokens, max_new, plain != 0, reinterpret_cast<cudaStream_t>(stream));
+}
+
+extern "C" size_t onellm_biased_attn_decode_workspace(int B, int H, int dv) { return biased_attn_decode_workspace(B, H, dv); }
+
+extern "C" int onellm_biased_attn_decode(const onellm_biased_attn* a, const onellm_token_positions* tp, int step_bound, void* workspace,
+                                         void* stream)
+{
+    ONELLM_REQUIRE(a && tp && step_bound >= 1, ONELLM_ERR_ARG, "biased_attn_decode: bad argument");
+    return biased_attn_decode(*a, *tp, step_bound, workspace, reinterpret_cast<cudaStream_t>(stream));
+}

@@ -132,7 +132,7 @@ embedding_pos_kernel(const int* __restrict__ ids, float* __restrict__ out, const
     pdl_wait();
     const int t = blockIdx.x, id = ids[t];
     int b, pos;
-    tp.locate(t, b, pos);
+    locate(tp, t, b, pos);
     const bool id_ok = id >= 0 && id < vocab, pos_ok = pos >= 0 && pos < max_pos;
     if (threadIdx.x == 0) {
         if (!id_ok) atomicExch(bad, 1);
@@ -171,3 +171,11 @@ int embedding_pos_launch(int dtype, const int* ids, float* out, const void* tabl
     return ONELLM_OK;
 }
 }  // namespace onellm
+
+extern "C" int onellm_embedding_pos(int dtype, const int* ids, float* out, const void* table, const void* pos_table, int n_tokens, int ld,
+                                    int vocab, int max_pos, const onellm_token_positions* tp, int* bad, void* stream)
+{
+    ONELLM_REQUIRE(tp, ONELLM_ERR_ARG, "embedding_pos: null pointer");
+    ONELLM_REQUIRE(dtype == ONELLM_BF16 || dtype == ONELLM_F32, ONELLM_ERR_UNSUPPORTED, "embedding_pos: dtype %d", dtype);
+    return embedding_pos_launch(dtype, ids, out, table, pos_table, n_tokens, ld, vocab, max_pos, *tp, bad, reinterpret_cast<cudaStream_t>(stream));
+}

@@ -258,3 +258,9 @@ int gated_recurrence(const GatedRecurrence& g, const TokenPositions& tp, int B, 
 }
 
 }  // namespace onellm
+
+extern "C" int onellm_gated_recurrence_run(const onellm_gated_recurrence* g, const onellm_token_positions* tp, int B, void* stream)
+{
+    ONELLM_REQUIRE(g && tp, ONELLM_ERR_ARG, "gated_recurrence: null pointer");
+    return onellm::gated_recurrence(*g, *tp, B, reinterpret_cast<cudaStream_t>(stream));
+}

@@ -267,3 +267,10 @@ extern "C" int onellm_add_residual_rmsnorm(int dtype, void* residual, void* deco
     ONELLM_CHECK_LAUNCH();
     return ONELLM_OK;
 }
+
+extern "C" int onellm_norm_pair(int dtype, const float* x, const int* rows, int n_rows, const float* w1, const float* w2, void* out1,
+                                void* out2, float eps, int width, int ld, void* stream)
+{
+    ONELLM_REQUIRE(dtype == ONELLM_BF16 || dtype == ONELLM_F32, ONELLM_ERR_UNSUPPORTED, "norm_pair: dtype %d", dtype);
+    return norm_pair(dtype, x, rows, n_rows, w1, w2, out1, out2, eps, width, ld, reinterpret_cast<cudaStream_t>(stream));
+}

@@ -384,3 +384,11 @@ extern "C" int onellm_gemm_swiglu(int dtype, const void* x, const void* Wg, cons
                                    true, reinterpret_cast<cudaStream_t>(stream)));
     return ONELLM_OK;
 }
+
+extern "C" int onellm_project(int dtype, const void* x, const void* W, const void* W2, void* y, long ldy, int M, int N, int K, int act, int f32,
+                              const float* resid, void* stream)
+{
+    ONELLM_REQUIRE(!resid || f32 || dtype == ONELLM_F32, ONELLM_ERR_ARG, "project: a residual needs a float output");
+    const Projection p = {dtype, x, W, W2, y, ldy, M, N, K, act, f32, resid};
+    return project(p, reinterpret_cast<cudaStream_t>(stream));
+}

@@ -64,7 +64,7 @@ int NAME() { TensorMap m{{"a", Tensor(CPU, getTensorType<int>(), {1})}}; return 
     assert subprocess.call([exe]) == 0
 
 
-@pytest.mark.skipif(not os.path.isdir(REFERENCE_TREE), reason="needs a oneLLM source tree")
+@pytest.mark.skipif(not os.path.isdir(os.path.join(REFERENCE_TREE, "src")), reason="needs a oneLLM source tree")
 def test_reference_layers_examples_and_unit_tests_build_unchanged(ob):
     sys.path.insert(0, os.path.join(ROOT, "oracle"))
     try:
