@@ -642,8 +642,132 @@ def run_ours(args, workload):
         sys.exit(1)
 
 
+# ---------------------------------------------------------------------------------------------
+# --design finuvik: the Finuvik design beside the LLaMA design at equal width, depth, heads and feed-forward
+# ---------------------------------------------------------------------------------------------
+DESIGN_SIZES = {
+    # width, layers, heads, kv_heads, head size, ff, recurrence heads x (key, value), vocabulary
+    "w2048": dict(hidden=2048, num_layers=16, head_num=16, kv_head_num=4, head_size=128, inter_size=5632, rec=(16, 128, 128), vocab_size=32000),
+    "w4096": dict(hidden=4096, num_layers=8, head_num=32, kv_head_num=8, head_size=128, inter_size=11008, rec=(32, 128, 128), vocab_size=32000),
+}
+
+
+def finuvik_config(s, max_positions):
+    layer = {"type": "parallel",
+             "mixer": {"left": {"heads": s["head_num"], "kv_heads": s["kv_head_num"], "dim": s["head_size"], "vdim": s["head_size"],
+                                "scale": s["head_size"] ** -0.5, "q_temp": {"coef": 0.1, "every": 1024}},
+                       "left_scale": 1.0, "right_scale": 1.0,
+                       "right": {"heads": s["rec"][0], "dim": s["rec"][1], "vdim": s["rec"][2]}},
+             "mlp": {"kind": "dense", "ff": s["inter_size"]}}
+    return {"architecture": "Finuvik", "vocab": s["vocab_size"], "width": s["hidden"], "max_positions": max_positions,
+            "norm": {"eps": 1e-6}, "layers": [layer] * s["num_layers"]}
+
+
+def run_design(args):
+    """Prefill and decode throughput of both designs and their like kernels side by side; one JSON line."""
+    import torch
+    import onellm_b200 as ob
+    from onellm_b200 import kernel_cases as kc
+    torch.cuda.set_device(0)
+    hbm_peak, tf_peak, peak_kind = peaks()
+    smax = 4096
+    out = {"design": "finuvik", "beside": "llama", "data": "synthetic", "peak_kind": peak_kind, "hbm_gbs": hbm_peak, "bf16_tflops": tf_peak,
+           "models": {}, "kernels": {}}
+
+    def timed(m, fn, n, warm):
+        st = torch.cuda.ExternalStream(m.stream)
+        ts = []
+        for i in range(warm + n):
+            torch.cuda.synchronize()
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record(st)
+            fn()
+            e1.record(st)
+            torch.cuda.synchronize()
+            if i >= warm:
+                ts.append(e0.elapsed_time(e1) * 1e-3)
+        return float(np.median(ts))
+
+    def open_design(kind, s, batch):
+        if kind == "finuvik":
+            m = ob.Model(finuvik_config(s, smax), ob.BF16, batch, smax)
+        else:
+            m = ob.Llama(max_seq_len=smax, max_batch=batch, **{k: s[k] for k in ("num_layers", "hidden", "head_num", "kv_head_num", "head_size",
+                                                                                 "inter_size", "vocab_size")})
+        m.init_random(seed=1, std=0.02)
+        m.set_sampling(top_k=1)
+        return m
+
+    rng = np.random.default_rng(0)
+    with ClockSampler(0) as clk:
+        clk.wait_first(3.0)
+        clk.mark_start()
+        for size, s in DESIGN_SIZES.items():
+            W, L, H, G, D, I, V = (s[k] for k in ("hidden", "num_layers", "head_num", "kv_head_num", "head_size", "inter_size", "vocab_size"))
+            RH, RK, RV = s["rec"]
+            res = out["models"][size] = {"shape": {k: v for k, v in s.items()}}
+            for kind in ("llama", "finuvik"):
+                proj = W * (H + 2 * G) * D + H * D * W + 3 * W * I
+                state = 0
+                if kind == "finuvik":
+                    proj += W * RH * (2 * RK + 2 * RV)
+                    state = RH * RK * RV * 4 * 2
+                r = res[kind] = {"projection_weights": proj * L, "prefill": {}, "decode": {}}
+                m = open_design(kind, s, 8)
+                for b, n in ((1, 2048), (8, 512)):
+                    ids = rng.integers(0, V, (b, n)).astype(np.int32)
+                    t = timed(m, lambda: m.prefill(ids), 5, 2)
+                    r["prefill"][f"{b}x{n}"] = {"tokens_per_s": b * n / t, "ms": t * 1e3, "projection_tflops": 2.0 * proj * L * b * n / t / 1e12}
+                m.close()
+                for b in (1, 8, 32):
+                    m = open_design(kind, s, b)
+                    ctx = 2000
+                    first = rng.integers(0, V, b).astype(np.int32)
+
+                    def block():
+                        for _ in range(16):
+                            m.decode_step(None, None)
+                    m.seek(b, ctx, first)
+                    block()
+                    m.seek(b, ctx, first)
+                    t = timed(m, block, 5, 1) / 16
+                    nbytes = proj * L * 2 + V * W * 2 + L * b * (2 * (ctx + 64) * G * D * 2 + state)
+                    r["decode"][f"b{b}_ctx{ctx}"] = {"tokens_per_s": b / t, "ms_per_step": t * 1e3, "bytes_per_step": nbytes,
+                                                     "frac_of_hbm": nbytes / t / 1e9 / hbm_peak}
+                    m.close()
+                torch.cuda.empty_cache()
+        pairs = [("fv_mix", "qkv"), ("fv_gate_up", "gate_up"), ("fv_out", "down"), ("fv_attn", "attn"), ("fv_rec", "attn"), ("fv_norm", "norm"),
+                 ("prefill_fv_mix", "prefill_qkv"), ("prefill_fv_gate", "prefill_gate"), ("prefill_fv_out", "prefill_down"),
+                 ("prefill_fv_attn", "prefill_attn"), ("prefill_fv_rec", None)]
+        fp32_peak = 148 * 128 * 2 * 1.965e9 / 1e12  # nominal: the recurrence runs on the fp32 pipes
+        done = {}
+        for mine, like in pairs:
+            for name in (mine, like):
+                if name is None or name in done:
+                    continue
+                prefill = name.startswith("prefill_")
+                for b, ctx in (((1, 2048), (8, 512)) if prefill else ((8, 2040), (32, 2040)) if name in ("fv_attn", "attn", "fv_rec") else ((8, 2040),)):
+                    case = kc.make_case(name, torch, "7b", b, ctx, 1)
+                    t = kc.time_case(case, torch, iters=20, warm=5, graph=not prefill)
+                    peak = fp32_peak * 1e12 if name == "prefill_fv_rec" else tf_peak * 1e12 if case.unit == "flop" else hbm_peak * 1e9
+                    done[name] = True
+                    out["kernels"][f"{name}_b{b}_{ctx}"] = {"us": t * 1e6, "amount": case.amount, "unit": case.unit, "frac": case.amount / t / peak,
+                                                           "beside": like if name == mine else None}
+                    del case
+                    torch.cuda.empty_cache()
+        clk.mark_end()
+    out["clocks"] = clk.summary()
+    out["timeout_flag"] = int(ob.lib().onellm_gemm_timeout_flag())
+    print(json.dumps(out), flush=True)
+    if out["timeout_flag"]:
+        sys.exit(1)
+
+
 def main():
     ap = argparse.ArgumentParser()
+    ap.add_argument("--design", default="llama", choices=["llama", "finuvik"],
+                    help="finuvik: throughput of the Finuvik design and its kernels beside the LLaMA design at equal size (one GPU; other "
+                         "options do not apply)")
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=128)
     ap.add_argument("--warmup", type=int, default=8)
@@ -660,7 +784,9 @@ def main():
     args = ap.parse_args()
     if args.warmup < 3 and args.impl == "ours":
         args.warmup = 3
-    if args.impl == "reference":
+    if args.design == "finuvik":
+        run_design(args)
+    elif args.impl == "reference":
         run_reference(args, args.workload)
     else:
         run_ours(args, args.workload)

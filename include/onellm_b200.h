@@ -512,7 +512,7 @@ ONELLM_API int onellm_biased_attn_decode(const onellm_biased_attn* a, const onel
  *     f = lower + (1 - lower) * sigmoid(z + zb)     state = diag(f) state + (1 - f) v^T     o = state^T silu(q)
  *     out = o * rsqrt(sum(o^2) / norm_width + eps) * w * out_scale
  * q, z, v: token t at + t * ld, heads dk / dk / dv apart; zb, lower [H * dk]; w [dv]; state [B, H, dk, dv], taken as zero
- * for a sequence with hist 0. */
+ * for a sequence at its first position. */
 typedef struct onellm_gated_recurrence {
     int dtype;
     int H, dk, dv;

@@ -175,6 +175,7 @@ int Engine::enqueue_step(int mode, int step_bound, int prompt_len)
 int Engine::run_step(int mode, int prompt_len)
 {
     const int step = cur_len + 1;
+    last_logits = logits;
     ONELLM_REQUIRE(step <= max_seq_len, ONELLM_ERR_STATE, "decode: sequence length %d exceeds max_seq_len %d", step,
                    max_seq_len);
     int bound = (step + 255) / 256 * 256;
@@ -187,7 +188,6 @@ int Engine::run_step(int mode, int prompt_len)
         return ONELLM_OK;
     }
     const long key = ((long)bound << 20) | ((long)batch << 8) | ((long)mode << 4) | (top_k > 1 ? 1 : 0);
-    last_logits = logits;
     // prompt_len, top_k, temperature are baked into the captured nodes: changing them drops the cache
     auto it = graphs.find(key);
     if (it == graphs.end() && !warmed.count(key)) {
@@ -397,7 +397,6 @@ extern "C" int onellm_llama_prefill(onellm_llama* h, const int* host_ids, int ba
     ONELLM_CUDA(cudaMemsetAsync(m->d_finished, 0, (size_t)batch, st));
     ONELLM_CUDA(cudaMemsetAsync(m->d_bad_id, 0, 4 * sizeof(int), st));
     ONELLM_CUDA(cudaStreamSynchronize(st));  // `first_step` lives on this stack frame
-    RC(m->reset_sequences());
     if (m->prefill_by_decode) {
         ONELLM_REQUIRE(m->want_rows.empty(), ONELLM_ERR_STATE, "llama_prefill: logits of single rows need the context-phase kernels");
         // one position at a time through the decode kernels; only the last position needs the LM head
@@ -439,7 +438,6 @@ extern "C" int onellm_llama_prefill_ragged(onellm_llama* h, const int* host_ids,
     ONELLM_CUDA(cudaMemsetAsync(m->d_finished, 0, (size_t)batch, st));
     ONELLM_CUDA(cudaMemsetAsync(m->d_bad_id, 0, 4 * sizeof(int), st));
     ONELLM_CUDA(cudaStreamSynchronize(st));  // `longest` lives on this stack frame
-    RC(m->reset_sequences());
     RC(m->prefill_context(batch, lens));
     return m->finish_context(host_first_ids, "llama_prefill_ragged");
 }

@@ -100,8 +100,6 @@ struct Engine {
     // All tokens of a context pass through all layers, and the logits of c.rows into c.logits.
     virtual int context_layers(const ContextBatch& c) = 0;
     virtual int init_random(uint64_t seed, float std) = 0;
-    // Called when sequences start from nothing: designs whose memory is not addressed by position alone clear it.
-    virtual int reset_sequences() { return ONELLM_OK; }
     // Around every point where the host waits for the stream (see llama.cu: tensor-parallel peers).
     virtual int queue_comm_check() { return ONELLM_OK; }
     virtual int comm_check(const char*) { return ONELLM_OK; }

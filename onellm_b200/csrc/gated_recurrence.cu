@@ -1,15 +1,20 @@
-// Gated outer-product recurrence (the HGRN2 form of linear attention: the forget gate also decides what is written),
-// for a context pass of any length and for one decode step; gates, recurrence and the per-head RMS norm of the
-// output are computed in float.
+// Gated outer-product recurrence (the HGRN2 form of linear attention: the forget gate also decides what is written);
+// gates, recurrence and the per-head RMS norm of the output are computed in float.  With g = 1 - f a state element
+// moves as
+//     s <- s + g (v - s)
+// which needs one multiply-add and keeps the digits of a gate near one (g comes from the complementary sigmoid).
 //
-// A thread block owns 32 value columns of one (sequence, head) and keeps that part of the state, dk x 32 floats, in
-// registers over all tokens of the call: columns of the state never meet, only the dk rows are summed into the output.
-// A thread holds R rows x 4 columns; the 8 lanes of a row group cover the 32 columns, the 4 row groups of each of
-// the 4 warps the dk = 16 R rows.  Tokens come in blocks of 32 through a double-buffered cp.async ring, are turned
-// into f, 1 - f and silu(q) once per block (1 - f from the complementary sigmoid, so that a gate near one keeps its
-// digits), and each warp leaves its partial outputs in shared memory; one reduction per token block adds the warps.
-// The blocks of a head form a cluster: its RMS norm needs all value columns, and the sums of squares of a token block
-// are exchanged through distributed shared memory.
+// Context pass (gated_recurrence_kernel).  A thread block owns 32 value columns of one (sequence, head) and keeps that
+// part of the state, dk x 32 floats, in registers over all tokens of the call: columns of the state never meet, only the
+// dk rows are summed into the output.  A thread holds R rows x 4 columns as pairs of rows for the packed fma.rn.f32x2;
+// the 8 lanes of a row group cover the 32 columns, the 4 row groups of each of the 4 warps the dk <= 16 R rows.  Tokens
+// come in blocks through a double-buffered cp.async ring, are turned into g and silu(q) once per block, and are taken
+// four at a time so that their sums over the row groups overlap; each warp leaves partial outputs in shared memory and
+// one reduction per token block adds the warps.  The blocks of a head form a cluster: its RMS norm needs all value
+// columns, and the sums of squares of a token block are exchanged through distributed shared memory.
+//
+// Decode step (gated_recurrence_step_kernel).  One token per sequence: the state is streamed once through registers,
+// HBM-bound; its first rows are requested before the dependency wait, because they do not depend on the kernel in front.
 #include <cooperative_groups.h>
 
 #include "mixers.h"
@@ -23,16 +28,61 @@ constexpr int kGrThreads = 128, kGrCols = 32;
 template <typename T, int R>
 constexpr int gr_tok() { return sizeof(T) == 4 && R > 8 ? 16 : 32; }
 
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 pack_f2(float lo, float hi)
+{
+    f32x2 r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+    return r;
+}
+__device__ __forceinline__ float sum_f2(f32x2 v)
+{
+    float lo, hi;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v));
+    return lo + hi;
+}
+__device__ __forceinline__ f32x2 fma_f2(f32x2 a, f32x2 b, f32x2 c)
+{
+    f32x2 r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+__device__ __forceinline__ f32x2 sub_f2(f32x2 a, f32x2 b)
+{
+    f32x2 r;
+    asm("sub.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+
+// sigmoid(x) and 1 - sigmoid(x), both with full relative precision; the fast exponential and division where the
+// projections are bfloat16 (their error is far below the rounding of x)
+template <typename T>
+__device__ __forceinline__ void sigmoid_pair(float x, float& s, float& c)
+{
+    float e, r;
+    if constexpr (sizeof(T) == 2) {
+        e = __expf(-fabsf(x));
+        r = __fdividef(1.f, 1.f + e);
+    } else {
+        e = expf(-fabsf(x));
+        r = 1.f / (1.f + e);
+    }
+    s = x >= 0.f ? r : e * r;
+    c = x >= 0.f ? e * r : r;
+}
+// 1 - f and silu(q) of one channel
+template <typename T>
+__device__ __forceinline__ void gate(float q, float z, float zb, float lower, float& g, float& qs)
+{
+    float s, c;
+    sigmoid_pair<T>(z + zb, s, c);
+    g = (1.f - lower) * c;
+    sigmoid_pair<T>(q, s, c);
+    qs = q * s;
+}
+
 struct GrParams {
-    const void *q, *z, *v;
-    long ld;
-    const float *zb, *lower, *w;
-    float eps;
-    int H, dk, dv, norm_width;
-    float* state;
-    void* out;
-    long out_ld;
-    float out_scale;
+    GatedRecurrence g;
     TokenPositions tp;
 };
 
@@ -42,46 +92,54 @@ __host__ __device__ constexpr size_t gr_raw_bytes(int dk) { return (size_t)gr_to
 template <typename T, int R>
 static size_t gr_smem_bytes(int dk)
 {
-    constexpr int kGrTok = gr_tok<T, R>();
-    return 2 * gr_raw_bytes<T, R>(dk) + sizeof(float) * ((size_t)kGrTok * (3 * 16 * R + kGrCols) + 4 * kGrTok * kGrCols + 2 * kGrTok);
+    constexpr int TOK = gr_tok<T, R>();
+    return 2 * gr_raw_bytes<T, R>(dk) + sizeof(float) * ((size_t)TOK * (2 * 16 * R + kGrCols) + 4 * TOK * kGrCols + 2 * TOK);
 }
 
 template <typename T, int R>
-__global__ void __launch_bounds__(kGrThreads) gated_recurrence_kernel(const GrParams p)
+__global__ void __launch_bounds__(kGrThreads) gated_recurrence_kernel(const GrParams pp)
 {
-    constexpr int kGrTok = gr_tok<T, R>();
+    constexpr int TOK = gr_tok<T, R>();
     constexpr int DKP = 16 * R;  // dk padded to whole thread tiles; the extra rows have zero gates and queries
     constexpr int VEC = Vec16<T>::N;
+    const GatedRecurrence& p = pp.g;
     extern __shared__ __align__(16) unsigned char smem[];
     const int dk = p.dk, h = blockIdx.y, b = blockIdx.z, c0 = blockIdx.x * kGrCols;
     const size_t raw = gr_raw_bytes<T, R>(dk);
-    float* sf = reinterpret_cast<float*>(smem + 2 * raw);
-    float* sg = sf + kGrTok * DKP;
-    float* sq = sg + kGrTok * DKP;
-    float* sv = sq + kGrTok * DKP;
-    float* part = sv + kGrTok * kGrCols;        // [4 warps][kGrTok][32]
-    float* ssq = part + 4 * kGrTok * kGrCols;   // [2][kGrTok]
+    float* sg = reinterpret_cast<float*>(smem + 2 * raw);
+    float* sq = sg + TOK * DKP;
+    float* sv = sq + TOK * DKP;
+    float* part = sv + TOK * kGrCols;        // [4 warps][TOK][32]
+    float* ssq = part + 4 * TOK * kGrCols;   // [2][TOK]
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int k0 = (warp * 4 + (lane >> 3)) * R, col = (lane & 7) * 4;
     cg::cluster_group cluster = cg::this_cluster();
     const int n_peers = gridDim.x;
 
-    const int tok0 = p.tp.cu ? p.tp.cu[b] : b;
-    const int n_tok = p.tp.cu ? p.tp.cu[b + 1] - tok0 : 1;
-    const bool fresh = p.tp.cu && p.tp.hist[b] == 0;
+    const int tok0 = pp.tp.cu[b], n_tok = pp.tp.cu[b + 1] - tok0;
+    const bool fresh = pp.tp.hist[b] == 0;
     float4* st = reinterpret_cast<float4*>(p.state + (((size_t)b * p.H + h) * dk) * p.dv + c0 + col);
     const size_t st_row = (size_t)p.dv / 4;
-
-    // The state was written by the same layer of an earlier step: it does not depend on the kernel before this one.
-    float S[R][4];
+    f32x2 S[R / 2][4];
 #pragma unroll
-    for (int r = 0; r < R; r++) {
-        float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (!fresh && k0 + r < dk) s = st[(size_t)(k0 + r) * st_row];
-        S[r][0] = s.x;
-        S[r][1] = s.y;
-        S[r][2] = s.z;
-        S[r][3] = s.w;
+    for (int r = 0; r < R; r += 2) {
+        float4 a = make_float4(0.f, 0.f, 0.f, 0.f), c = a;
+        if (!fresh && k0 + r < dk) a = st[(size_t)(k0 + r) * st_row];
+        if (!fresh && k0 + r + 1 < dk) c = st[(size_t)(k0 + r + 1) * st_row];
+        S[r / 2][0] = pack_f2(a.x, c.x);
+        S[r / 2][1] = pack_f2(a.y, c.y);
+        S[r / 2][2] = pack_f2(a.z, c.z);
+        S[r / 2][3] = pack_f2(a.w, c.w);
+    }
+    // this thread's channels when it makes gates: k = tid % DKP of tokens tid / DKP, + 128 / DKP, ... (two channels when
+    // there are more of them than threads)
+    constexpr int KPT = DKP > kGrThreads ? DKP / kGrThreads : 1, TSTEP = DKP > kGrThreads ? 1 : kGrThreads / DKP;
+    float zb[KPT], lower[KPT];
+#pragma unroll
+    for (int i = 0; i < KPT; i++) {
+        const int k = tid % DKP + i * kGrThreads;
+        zb[i] = k < dk ? p.zb[h * dk + k] : 0.f;
+        lower[i] = k < dk ? p.lower[h * dk + k] : 0.f;
     }
     pdl_wait();
     pdl_launch_dependents();
@@ -92,7 +150,7 @@ __global__ void __launch_bounds__(kGrThreads) gated_recurrence_kernel(const GrPa
     const int kc = dk / VEC, vc = kGrCols / VEC, per_tok = 2 * kc + vc;
     const uint32_t raw_base = (uint32_t)__cvta_generic_to_shared(smem);
     auto issue = [&](int blk) {
-        const int t0 = blk * kGrTok, n = min(kGrTok, n_tok - t0);
+        const int t0 = blk * TOK, n = min(TOK, n_tok - t0);
         const uint32_t dst = raw_base + (uint32_t)((blk & 1) * raw);
         for (int i = tid; i < n * per_tok; i += kGrThreads) {
             const int t = i / per_tok, c = i % per_tok;
@@ -101,7 +159,8 @@ __global__ void __launch_bounds__(kGrThreads) gated_recurrence_kernel(const GrPa
             cp_async16(dst + (uint32_t)i * 16u, src, 16);
         }
     };
-    const int n_blk = (n_tok + kGrTok - 1) / kGrTok;
+    const float wn = p.w[c0 + lane] * p.out_scale;
+    const int n_blk = (n_tok + TOK - 1) / TOK;
     if (n_blk > 0) issue(0);
     cp_async_commit();
     for (int blk = 0; blk < n_blk; blk++) {
@@ -109,77 +168,73 @@ __global__ void __launch_bounds__(kGrThreads) gated_recurrence_kernel(const GrPa
         cp_async_commit();
         cp_async_wait<1>();
         __syncthreads();
-        const int n = min(kGrTok, n_tok - blk * kGrTok);
+        const int n = min(TOK, n_tok - blk * TOK), n4 = (n + 3) & ~3;  // tokens n .. n4 - 1 change nothing: g = q = 0
         const T* rb = reinterpret_cast<const T*>(smem + (size_t)(blk & 1) * raw);
         const int row_el = 2 * dk + kGrCols;
-        for (int i = tid; i < n * DKP; i += kGrThreads) {
-            const int t = i / DKP, k = i % DKP;
-            float f = 0.f, g = 0.f, qs = 0.f;
-            if (k < dk) {
-                const float qv = to_float(rb[t * row_el + k]);
-                const float zv = to_float(rb[t * row_el + dk + k]) + p.zb[h * dk + k];
-                const float l = p.lower[h * dk + k];
-                const float e = expf(-fabsf(zv)), s = 1.f / (1.f + e), es = e * s;
-                f = l + (1.f - l) * (zv >= 0.f ? s : es);
-                g = (1.f - l) * (zv >= 0.f ? es : s);
-                const float eq = expf(-fabsf(qv)), sg1 = 1.f / (1.f + eq);
-                qs = qv * (qv >= 0.f ? sg1 : eq * sg1);
+#pragma unroll
+        for (int i = 0; i < KPT; i++) {
+            const int k = tid % DKP + i * kGrThreads;
+#pragma unroll 4
+            for (int t = tid / DKP; t < n4; t += TSTEP) {
+                float g = 0.f, qs = 0.f;
+                if (k < dk && t < n) gate<T>(to_float(rb[t * row_el + k]), to_float(rb[t * row_el + dk + k]), zb[i], lower[i], g, qs);
+                sg[t * DKP + k] = g;
+                sq[t * DKP + k] = qs;
             }
-            sf[i] = f;
-            sg[i] = g;
-            sq[i] = qs;
         }
-        for (int i = tid; i < n * kGrCols; i += kGrThreads) sv[i] = to_float(rb[(i / kGrCols) * row_el + 2 * dk + i % kGrCols]);
+        for (int t = warp; t < n4; t += 4) sv[t * kGrCols + lane] = t < n ? to_float(rb[t * row_el + 2 * dk + lane]) : 0.f;
         __syncthreads();
-#pragma unroll 2
-        for (int t = 0; t < n; t++) {
-            const float4 v4 = *reinterpret_cast<const float4*>(sv + t * kGrCols + col);
-            const float vv[4] = {v4.x, v4.y, v4.z, v4.w};
-            float o[4] = {0.f, 0.f, 0.f, 0.f};
-            const float *ft = sf + t * DKP + k0, *gt = sg + t * DKP + k0, *qt = sq + t * DKP + k0;
-            float f[R], g[R], qq[R];
-            if constexpr (R % 4 == 0) {
+        for (int t = 0; t < n4; t += 4) {
+            f32x2 o2[4][4];
 #pragma unroll
-                for (int r = 0; r < R; r += 4) {
-                    *reinterpret_cast<float4*>(&f[r]) = *reinterpret_cast<const float4*>(ft + r);
-                    *reinterpret_cast<float4*>(&g[r]) = *reinterpret_cast<const float4*>(gt + r);
-                    *reinterpret_cast<float4*>(&qq[r]) = *reinterpret_cast<const float4*>(qt + r);
-                }
-            } else {
+            for (int u = 0; u < 4; u++) {
+                const float4 v4 = *reinterpret_cast<const float4*>(sv + (t + u) * kGrCols + col);
+                const f32x2 vv[4] = {pack_f2(v4.x, v4.x), pack_f2(v4.y, v4.y), pack_f2(v4.z, v4.z), pack_f2(v4.w, v4.w)};
+                f32x2 g2[R / 2], q2[R / 2];
+                const float *gt = sg + (t + u) * DKP + k0, *qt = sq + (t + u) * DKP + k0;
+                if constexpr (R >= 4) {
 #pragma unroll
-                for (int r = 0; r < R; r++) {
-                    f[r] = ft[r];
-                    g[r] = gt[r];
-                    qq[r] = qt[r];
+                    for (int r = 0; r < R / 2; r += 2) {
+                        *reinterpret_cast<ulonglong2*>(&g2[r]) = *reinterpret_cast<const ulonglong2*>(gt + 2 * r);
+                        *reinterpret_cast<ulonglong2*>(&q2[r]) = *reinterpret_cast<const ulonglong2*>(qt + 2 * r);
+                    }
+                } else {
+                    g2[0] = *reinterpret_cast<const f32x2*>(gt);
+                    q2[0] = *reinterpret_cast<const f32x2*>(qt);
                 }
+#pragma unroll
+                for (int c = 0; c < 4; c++) o2[u][c] = 0ull;
+#pragma unroll
+                for (int r = 0; r < R / 2; r++)
+#pragma unroll
+                    for (int c = 0; c < 4; c++) {
+                        S[r][c] = fma_f2(g2[r], sub_f2(vv[c], S[r][c]), S[r][c]);
+                        o2[u][c] = fma_f2(q2[r], S[r][c], o2[u][c]);
+                    }
             }
-#pragma unroll
-            for (int r = 0; r < R; r++)
-#pragma unroll
-                for (int c = 0; c < 4; c++) {
-                    S[r][c] = fmaf(f[r], S[r][c], g[r] * vv[c]);
-                    o[c] = fmaf(qq[r], S[r][c], o[c]);
-                }
-            // sum over the four row groups of the warp; lane keeps one column: first halves (columns 0-1 | 2-3), then one of two
+            // sum over the row groups of the warp; a lane keeps one column: halves first (columns 0-1 | 2-3), then one of two
             const bool hi2 = lane & 16, hi1 = lane & 8;
-            float a0 = hi2 ? o[2] : o[0], a1 = hi2 ? o[3] : o[1], b0 = hi2 ? o[0] : o[2], b1 = hi2 ? o[1] : o[3];
-            a0 += __shfl_xor_sync(0xffffffffu, b0, 16);
-            a1 += __shfl_xor_sync(0xffffffffu, b1, 16);
-            float a = hi1 ? a1 : a0;
-            const float bb = hi1 ? a0 : a1;
-            a += __shfl_xor_sync(0xffffffffu, bb, 8);
-            part[(warp * kGrTok + t) * kGrCols + col + (hi2 ? 2 : 0) + (hi1 ? 1 : 0)] = a;
+#pragma unroll
+            for (int u = 0; u < 4; u++) {
+                const float o[4] = {sum_f2(o2[u][0]), sum_f2(o2[u][1]), sum_f2(o2[u][2]), sum_f2(o2[u][3])};
+                float a0 = hi2 ? o[2] : o[0], a1 = hi2 ? o[3] : o[1];
+                a0 += __shfl_xor_sync(0xffffffffu, hi2 ? o[0] : o[2], 16);
+                a1 += __shfl_xor_sync(0xffffffffu, hi2 ? o[1] : o[3], 16);
+                const float a = (hi1 ? a1 : a0) + __shfl_xor_sync(0xffffffffu, hi1 ? a0 : a1, 8);
+                part[(warp * TOK + t + u) * kGrCols + col + (hi2 ? 2 : 0) + (hi1 ? 1 : 0)] = a;
+            }
         }
         __syncthreads();
         // one warp per token row: add the warps' partial sums, sum of squares of the 32 columns
-        float o[kGrTok / 4];
-        float* ss_now = ssq + (blk & 1) * kGrTok;
+        float o[TOK / 4];
+        float* ss_now = ssq + (blk & 1) * TOK;
 #pragma unroll
-        for (int i = 0; i < kGrTok / 4; i++) {
+        for (int i = 0; i < TOK / 4; i++) {
             const int t = warp + 4 * i;
             o[i] = 0.f;
             if (t < n) {
-                for (int w = 0; w < 4; w++) o[i] += part[(w * kGrTok + t) * kGrCols + lane];
+#pragma unroll
+                for (int w = 0; w < 4; w++) o[i] += part[(w * TOK + t) * kGrCols + lane];
                 const float s = warp_sum(o[i] * o[i]);
                 if (lane == 0) ss_now[t] = s;
             }
@@ -187,25 +242,148 @@ __global__ void __launch_bounds__(kGrThreads) gated_recurrence_kernel(const GrPa
         // Every block of the cluster has written its sums; they stay valid for one more round (two buffers), and a block
         // that writes that buffer again has passed the next round's barrier, behind everyone's reads of this one.
         cluster.sync();
+        // lane t of every warp adds the cluster's sums of token t
+        float inv = 0.f;
+        if (lane < n) {
+            float s = 0.f;
+            for (int r = 0; r < n_peers; r++) s += cluster.map_shared_rank(ss_now, r)[lane];
+            inv = 1.0f / sqrtf(s / (float)p.norm_width + p.eps);
+        }
 #pragma unroll
-        for (int i = 0; i < kGrTok / 4; i++) {
+        for (int i = 0; i < TOK / 4; i++) {
             const int t = warp + 4 * i;
+            const float f = __shfl_sync(0xffffffffu, inv, t);
             if (t < n) {
-                float s = 0.f;
-                for (int r = 0; r < n_peers; r++) s += cluster.map_shared_rank(ss_now, r)[t];
-                const float inv = 1.0f / sqrtf(s / (float)p.norm_width + p.eps);
-                T* dst = reinterpret_cast<T*>(p.out) + (size_t)(tok0 + blk * kGrTok + t) * p.out_ld + (size_t)h * p.dv + c0 + lane;
-                *dst = from_float<T>(o[i] * inv * p.w[c0 + lane] * p.out_scale);
+                T* dst = reinterpret_cast<T*>(p.out) + (size_t)(tok0 + blk * TOK + t) * p.out_ld + (size_t)h * p.dv + c0 + lane;
+                *dst = from_float<T>(o[i] * f * wn);
             }
         }
     }
     cp_async_wait<0>();
     if (n_tok > 0) {
 #pragma unroll
-        for (int r = 0; r < R; r++)
-            if (k0 + r < dk) st[(size_t)(k0 + r) * st_row] = make_float4(S[r][0], S[r][1], S[r][2], S[r][3]);
+        for (int r = 0; r < R; r += 2) {
+            float a[4], c[4];
+#pragma unroll
+            for (int j = 0; j < 4; j++) asm("mov.b64 {%0, %1}, %2;" : "=f"(a[j]), "=f"(c[j]) : "l"(S[r / 2][j]));
+            if (k0 + r < dk) st[(size_t)(k0 + r) * st_row] = make_float4(a[0], a[1], a[2], a[3]);
+            if (k0 + r + 1 < dk) st[(size_t)(k0 + r + 1) * st_row] = make_float4(c[0], c[1], c[2], c[3]);
+        }
     }
     cluster.sync();  // peers may still be reading this block's sums
+}
+
+// One token per sequence.  A block owns `cols` value columns of one (sequence, head); cols / 4 threads share a row and
+// every thread walks the rows of its column group, kGsBatch at a time.
+constexpr int kGsThreads = 256, kGsBatch = 8;
+
+template <typename T>
+__global__ void __launch_bounds__(kGsThreads) gated_recurrence_step_kernel(const GrParams pp, int cols)
+{
+    const GatedRecurrence& p = pp.g;
+    __shared__ float sg[256], sq[256];
+    __shared__ __align__(16) float part[kGsThreads * 4];
+    __shared__ float ssq, wsum[kGsThreads / 32];
+    const int dk = p.dk, h = blockIdx.y, b = blockIdx.z, c0 = blockIdx.x * cols, tid = threadIdx.x;
+    const int tpr = cols / 4, rows_par = kGsThreads / tpr;  // threads per row, rows at a time
+    const int r0 = tid / tpr, col = (tid % tpr) * 4;
+    const bool works = r0 < rows_par;  // 256 need not be a multiple of tpr
+    const bool fresh = *pp.tp.step - 1 + pp.tp.off[b] == 0;
+    float* base = p.state + (((size_t)b * p.H + h) * dk) * p.dv + c0 + col;
+    float4 s[kGsBatch];
+    auto fetch = [&](int first) {
+#pragma unroll
+        for (int i = 0; i < kGsBatch; i++) {
+            const int r = first + i * rows_par;
+            s[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (works && !fresh && r < dk) s[i] = *reinterpret_cast<const float4*>(base + (size_t)r * p.dv);
+        }
+    };
+    fetch(r0);
+    float zb = 0.f, lower = 0.f;
+    if (tid < dk) {
+        zb = p.zb[h * dk + tid];
+        lower = p.lower[h * dk + tid];
+    }
+    pdl_wait();
+    pdl_launch_dependents();
+    if (tid < dk) {
+        const T* q = reinterpret_cast<const T*>(p.q) + (size_t)b * p.ld + (size_t)h * dk;
+        const T* z = reinterpret_cast<const T*>(p.z) + (size_t)b * p.ld + (size_t)h * dk;
+        gate<T>(to_float(q[tid]), to_float(z[tid]), zb, lower, sg[tid], sq[tid]);
+    }
+    float v[4] = {0.f, 0.f, 0.f, 0.f};
+    if (works) {
+        const T* vp = reinterpret_cast<const T*>(p.v) + (size_t)b * p.ld + (size_t)h * p.dv + c0 + col;
+#pragma unroll
+        for (int i = 0; i < 4; i++) v[i] = to_float(vp[i]);
+    }
+    __syncthreads();
+    float o[4] = {0.f, 0.f, 0.f, 0.f};
+    for (int first = r0; first < dk; first += kGsBatch * rows_par) {
+        if (first != r0) fetch(first);
+#pragma unroll
+        for (int i = 0; i < kGsBatch; i++) {
+            const int r = first + i * rows_par;
+            if (works && r < dk) {
+                const float g = sg[r], q = sq[r];
+                s[i].x = fmaf(g, v[0] - s[i].x, s[i].x);
+                s[i].y = fmaf(g, v[1] - s[i].y, s[i].y);
+                s[i].z = fmaf(g, v[2] - s[i].z, s[i].z);
+                s[i].w = fmaf(g, v[3] - s[i].w, s[i].w);
+                o[0] = fmaf(q, s[i].x, o[0]);
+                o[1] = fmaf(q, s[i].y, o[1]);
+                o[2] = fmaf(q, s[i].z, o[2]);
+                o[3] = fmaf(q, s[i].w, o[3]);
+                *reinterpret_cast<float4*>(base + (size_t)r * p.dv) = s[i];
+            }
+        }
+    }
+    if (works) *reinterpret_cast<float4*>(&part[r0 * cols + col]) = make_float4(o[0], o[1], o[2], o[3]);  // rows_par * cols <= 1024
+    __syncthreads();
+    float y = 0.f;
+    if (tid < cols)
+        for (int r = 0; r < rows_par; r++) y += part[r * cols + tid];
+    const float sq1 = warp_sum(y * y);
+    if ((tid & 31) == 0) wsum[tid >> 5] = sq1;
+    __syncthreads();
+    if (tid == 0) {
+        float t = 0.f;
+        for (int i = 0; i < kGsThreads / 32; i++) t += wsum[i];
+        ssq = t;
+    }
+    cg::cluster_group cluster = cg::this_cluster();
+    cluster.sync();  // a barrier of the block too when it is alone
+    float t = 0.f;
+    for (int r = 0; r < (int)gridDim.x; r++) t += *cluster.map_shared_rank(&ssq, r);
+    if (tid < cols) {
+        const float inv = 1.0f / sqrtf(t / (float)p.norm_width + p.eps);
+        reinterpret_cast<T*>(p.out)[(size_t)b * p.out_ld + (size_t)h * p.dv + c0 + tid] = from_float<T>(y * inv * p.w[c0 + tid] * p.out_scale);
+    }
+    cluster.sync();  // peers may still be reading this block's sum
+}
+
+template <typename Kernel, typename... Args>
+static int launch_cluster(Kernel kern, dim3 grid, int threads, size_t smem, cudaStream_t st, Args... args)
+{
+    (void)prefer_max_shared((const void*)kern);
+    cudaLaunchConfig_t cfg = {};
+    cudaLaunchAttribute at[2];
+    at[0].id = cudaLaunchAttributeClusterDimension;
+    at[0].val.clusterDim.x = grid.x;
+    at[0].val.clusterDim.y = 1;
+    at[0].val.clusterDim.z = 1;
+    at[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    at[1].val.programmaticStreamSerializationAllowed = 1;
+    cfg.gridDim = grid;
+    cfg.blockDim = dim3(threads);
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = st;
+    cfg.attrs = at;
+    cfg.numAttrs = 2;
+    note_launch();
+    ONELLM_CUDA(cudaLaunchKernelEx(&cfg, kern, args...));
+    return ONELLM_OK;
 }
 
 template <typename T, int R>
@@ -213,37 +391,24 @@ static int launch_gr(const GrParams& p, int B, cudaStream_t st)
 {
     auto kern = gated_recurrence_kernel<T, R>;
     static DeviceOnce attr;
-    ONELLM_CUDA(attr.run([kern] {
-        const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024);
-        return e != cudaSuccess ? e : prefer_max_shared((const void*)kern);
-    }));
-    cudaLaunchConfig_t cfg = {};
-    cudaLaunchAttribute at[2];
-    at[0].id = cudaLaunchAttributeClusterDimension;
-    at[0].val.clusterDim.x = p.dv / kGrCols;
-    at[0].val.clusterDim.y = 1;
-    at[0].val.clusterDim.z = 1;
-    at[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    at[1].val.programmaticStreamSerializationAllowed = 1;
-    cfg.gridDim = dim3(p.dv / kGrCols, p.H, B);
-    cfg.blockDim = dim3(kGrThreads);
-    cfg.dynamicSmemBytes = gr_smem_bytes<T, R>(p.dk);
-    cfg.stream = st;
-    cfg.attrs = at;
-    cfg.numAttrs = 2;
-    note_launch();
-    ONELLM_CUDA(cudaLaunchKernelEx(&cfg, kern, p));
-    return ONELLM_OK;
+    ONELLM_CUDA(attr.run([kern] { return cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024); }));
+    return launch_cluster(kern, dim3(p.g.dv / kGrCols, p.g.H, B), kGrThreads, gr_smem_bytes<T, R>(p.g.dk), st, p);
 }
 
 template <typename T>
 static int dispatch_gr(const GrParams& p, int B, cudaStream_t st)
 {
-    const int R = p.dk / 16;
-    if (R <= 1) return launch_gr<T, 1>(p, B, st);
-    if (R <= 2) return launch_gr<T, 2>(p, B, st);
-    if (R <= 4) return launch_gr<T, 4>(p, B, st);
-    if (R <= 8) return launch_gr<T, 8>(p, B, st);
+    if (!p.tp.cu) {
+        // columns of a head over several blocks only while whole heads leave SMs without work
+        int cols = p.g.dv;
+        for (int n = 2; n <= 8 && (long)B * p.g.H * (p.g.dv / cols) < 2L * num_sms(); n *= 2)
+            if (p.g.dv % (32 * n) == 0) cols = p.g.dv / n;
+        return launch_cluster(gated_recurrence_step_kernel<T>, dim3(p.g.dv / cols, p.g.H, B), kGsThreads, 0, st, p, cols);
+    }
+    const int dk = p.g.dk;
+    if (dk <= 32) return launch_gr<T, 2>(p, B, st);
+    if (dk <= 64) return launch_gr<T, 4>(p, B, st);
+    if (dk <= 128) return launch_gr<T, 8>(p, B, st);
     return launch_gr<T, 16>(p, B, st);
 }
 
@@ -252,8 +417,9 @@ int gated_recurrence(const GatedRecurrence& g, const TokenPositions& tp, int B, 
     ONELLM_REQUIRE(g.q && g.z && g.v && g.zb && g.lower && g.w && g.state && g.out, ONELLM_ERR_ARG, "gated_recurrence: null pointer");
     ONELLM_REQUIRE(g.dk > 0 && g.dk % 16 == 0 && g.dk <= 256 && g.dv > 0 && g.dv % kGrCols == 0 && g.dv <= 8 * kGrCols, ONELLM_ERR_UNSUPPORTED,
                    "gated_recurrence: key size %d must be a multiple of 16 and value size %d of 32, both at most 256", g.dk, g.dv);
-    ONELLM_REQUIRE(g.H > 0 && g.H <= 65535 && B > 0 && B <= 65535 && g.ld % 8 == 0, ONELLM_ERR_ARG, "gated_recurrence: bad size");
-    const GrParams p = {g.q, g.z, g.v, g.ld, g.zb, g.lower, g.w, g.eps, g.H, g.dk, g.dv, g.norm_width, g.state, g.out, g.out_ld, g.out_scale, tp};
+    ONELLM_REQUIRE(g.H > 0 && g.H <= 65535 && B > 0 && B <= 65535 && g.ld % 8 == 0 && (tp.cu ? tp.hist != nullptr : tp.step && tp.off),
+                   ONELLM_ERR_ARG, "gated_recurrence: bad argument");
+    const GrParams p = {g, tp};
     return g.dtype == ONELLM_F32 ? dispatch_gr<float>(p, B, st) : dispatch_gr<__nv_bfloat16>(p, B, st);
 }
 

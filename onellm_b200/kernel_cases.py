@@ -21,6 +21,14 @@ Context-phase cases (reported in TFLOP/s, except prefill_rope):
     prefill_layer                  one whole decoder layer on --batch x --ctx tokens as the model runs it: QKV projection (RMS scale
                                    in its epilogue), RoPE + cache write, attention, o_proj (+ residual), gate/up + SwiGLU, down (+ residual)
 
+Cases of the mechanisms behind onellm_model_open (bfloat16; widths and heads of --model, keys and values of head_size, as
+many recurrence heads as attention heads), each beside the like case above:
+    fv_mix, fv_gate_up, fv_out     decode: all mixer projections at once, ReLU-gated pair, stacked output projections added to
+                                   the float stream
+    fv_attn, fv_rec, fv_norm       decode attention with factor and penalty tables; one recurrence step; two norms of a float
+                                   stream of 4096 rows
+    prefill_fv_mix, prefill_fv_gate, prefill_fv_out, prefill_fv_attn, prefill_fv_rec       the same in the context phase
+
 Every case holds a few hundred MB on the device (more than the 126 MB L2, far less than a model) and runs on
 rotating buffers.  `--tp T` uses the per-rank shapes of T-way tensor parallelism; `--graph` times the launches as
 one CUDA graph, i.e. back to back on the device without the host's launch cost (what a decode step sees).
@@ -39,9 +47,9 @@ MODELS = {
 }
 
 DECODE_CASES = ["qkv", "o_proj", "gate_up", "down", "lm_head_kn", "lm_head", "attn", "attn_c1", "norm", "rmsnorm", "norm8",
-                "topk", "sample", "decode_layer"]
+                "topk", "sample", "decode_layer", "fv_mix", "fv_gate_up", "fv_out", "fv_attn", "fv_rec", "fv_norm"]
 PREFILL_CASES = ["prefill_qkv", "prefill_o", "prefill_gate", "prefill_down", "prefill_lm", "prefill_attn", "prefill_rope",
-                 "prefill_layer"]
+                 "prefill_layer", "prefill_fv_mix", "prefill_fv_gate", "prefill_fv_out", "prefill_fv_attn", "prefill_fv_rec"]
 
 
 @dataclass
@@ -63,8 +71,90 @@ def _projection_kernel(tokens, dual):
     return f"skinny_kn_staged_kernel<{mb},{'true' if dual else 'false'},false>"
 
 
+def make_mechanism_case(name, torch, m, B, ctx, plain=False) -> Case:
+    """The fv_ cases: m as in MODELS, optionally with kv_heads, value_size, rec_heads, rec_key, rec_value."""
+    prefill = name.startswith("prefill_")
+    what = name.rsplit("_", 1)[1] if not name.endswith("gate_up") else "gate"
+    W, H, D, INTER = m["hidden"], m["head_num"], m["head_size"], m["inter_size"]
+    G, DV = m.get("kv_heads", H), m.get("value_size", D)
+    RH, RK, RV = m.get("rec_heads", H), m.get("rec_key", D), m.get("rec_value", D)
+    n_mix = (H + G) * D + G * DV + RH * (2 * RK + RV)
+    n_cat = H * DV + RH * RV + INTER
+    T = B * ctx if prefill else B
+    bf = dict(device="cuda", dtype=torch.bfloat16)
+    f32 = dict(device="cuda", dtype=torch.float32)
+    rnd = lambda *s: 0.02 * torch.randn(*s, **bf)
+    n_rot = lambda nbytes, target=400e6: 2 if prefill else max(2, int(target // nbytes) + 1)
+    BF = ob.BF16
+    if what in ("mix", "gate", "out"):
+        K, N = {"mix": (W, n_mix), "gate": (W, INTER), "out": (n_cat, W)}[what]
+        dual = what == "gate"
+        rot = n_rot(K * N * 2 * (2 if dual else 1))
+        x, w = torch.randn(T, K, **bf), [rnd(K, N) for _ in range(rot)]
+        wu = [rnd(K, N) for _ in range(rot)] if dual else [None] * rot
+        if what == "out":
+            y = torch.randn(T, N, **f32)
+            fn = lambda i: ob.project(BF, x, w[i], None, y, T, N, K, f32=True, resid=y)
+        elif dual:
+            y = torch.zeros(T, n_cat, **bf)
+            fn = lambda i: ob.project(BF, x, w[i], wu[i], y.data_ptr() + (n_cat - INTER) * 2, T, N, K, ldy=n_cat, act=ob.GATE_RELU)
+        else:
+            y = torch.zeros(T, N, **bf)
+            fn = lambda i: ob.project(BF, x, w[i], None, y, T, N, K)
+        if prefill:
+            return Case(fn, rot, 2.0 * T * N * K * (2 if dual else 1), "flop", "gemm_tc_kernel (bf16)", keep=(x, w, wu, y))
+        nbytes = K * N * 2 * (2 if dual else 1) + T * K * 2 + T * N * (8 if what == "out" else 2)
+        return Case(fn, rot, nbytes, "B", _projection_kernel(T, dual) + " (bf16)", keep=(x, w, wu, y))
+    if what == "norm":
+        rows = 4096
+        xs = [torch.randn(rows, W, **f32) for _ in range(4)]
+        w1, w2, o1, o2 = torch.zeros(W, **f32), torch.zeros(W, **f32), torch.empty(rows, W, **bf), torch.empty(rows, W, **bf)
+        fn = lambda i: ob.norm_pair(BF, xs[i], None, rows, w1, w2, o1, o2, 1e-6, W, W)
+        return Case(fn, 4, rows * W * 8, "B", "norm_pair_kernel", keep=(xs, w1, w2, o1, o2))
+    mix, cat = torch.randn(T, n_mix, **bf), torch.zeros(T, n_cat, **bf)
+    cu = torch.arange(0, B + 1, device="cuda", dtype=torch.int32) * ctx
+    hist, off = torch.zeros(B, device="cuda", dtype=torch.int32), torch.zeros(B, device="cuda", dtype=torch.int32)
+    step = torch.full((1,), ctx + 1, device="cuda", dtype=torch.int32)
+    tp = ob.TokenPositions(cu.data_ptr(), hist.data_ptr(), B, None, None) if prefill else \
+        ob.TokenPositions(None, None, B, step.data_ptr(), off.data_ptr())
+    p = mix.data_ptr()
+    if what == "attn":
+        S = max(2048, ctx + 8)
+        rot = n_rot(B * G * S * (D + DV) * 2, 300e6)
+        kc, vc = [torch.randn(B, G, S, D, **bf) for _ in range(rot)], [torch.randn(B, G, S, DV, **bf) for _ in range(rot)]
+        qf, pen = torch.empty(S, **f32), torch.empty(H, S, **f32)
+        ob.query_factor(qf, S, D ** -0.5, 0.1, 1024)
+        ob.distance_penalty(pen, torch.ones(H, **f32), torch.full((H,), 0.1, **f32), H, S)
+        a = [ob.BiasedAttn(BF, H, G, D, DV, p, p + H * D * 2, p + (H + G) * D * 2, n_mix, kc[i].data_ptr(), vc[i].data_ptr(), S,
+                           qf.data_ptr(), pen.data_ptr(), cat.data_ptr(), n_cat, 1.0) for i in range(rot)]
+        ws = torch.empty(ob.biased_attn_decode_workspace(B, H, DV), device="cuda", dtype=torch.uint8)
+        keep = (mix, cat, cu, hist, off, step, kc, vc, qf, pen, ws)
+        if prefill:
+            fn = lambda i: ob.biased_attn_context(a[i], tp, T, ctx, plain)
+            return Case(fn, rot, float(B * H * 2 * (D + DV) * ctx * (ctx + 1) / 2), "flop", "biased_attn_tc_kernel", keep=keep)
+        fn = lambda i: ob.biased_attn_decode(a[i], tp, ctx + 1, ws)
+        nbytes = ctx * B * G * (D + DV) * 2 + B * (H * D + 2 * G * (D + DV) + H * DV) * 2
+        return Case(fn, rot, nbytes, "B", "biased_attn_decode_kernel", keep=keep)
+    if what == "rec":
+        rot = n_rot(2 * B * RH * RK * RV * 4, 300e6)
+        state = [torch.zeros(B, RH, RK, RV, **f32) for _ in range(rot)]
+        zb, lower, w = torch.full((RH * RK,), 2.0, **f32), torch.full((RH * RK,), 0.5, **f32), torch.ones(RV, **f32)
+        c0 = (H + G) * D + G * DV
+        g = [ob.GatedRecurrence(BF, RH, RK, RV, p + c0 * 2, p + (c0 + RH * RK) * 2, p + (c0 + 2 * RH * RK) * 2, n_mix, zb.data_ptr(),
+                                lower.data_ptr(), w.data_ptr(), 1e-6, RV, state[i].data_ptr(), cat.data_ptr() + H * DV * 2, n_cat, 1.0)
+             for i in range(rot)]
+        fn = lambda i: ob.gated_recurrence(g[i], tp, B)
+        keep = (mix, cat, cu, hist, off, step, state, zb, lower, w)
+        if prefill:  # decay and write (a product and a multiply-add), read (a multiply-add) per state element and token
+            return Case(fn, rot, 5.0 * T * RH * RK * RV, "flop", "gated_recurrence_kernel", keep=keep)
+        return Case(fn, rot, 2 * B * RH * RK * RV * 4 + B * RH * (2 * RK + 2 * RV) * 2, "B", "gated_recurrence_kernel", keep=keep)
+    raise ValueError(f"unknown case {name}")
+
+
 def make_case(name, torch, model="7b", batch=8, ctx=2040, tp=1, plain=False) -> Case:
     m = MODELS[model] if isinstance(model, str) else model
+    if "fv_" in name:
+        return make_mechanism_case(name, torch, m, batch, ctx, plain)
     HID, D, V = m["hidden"], m["head_size"], m["vocab_size"]
     H, INTER = m["head_num"] // tp, m["inter_size"] // tp
     B = batch
