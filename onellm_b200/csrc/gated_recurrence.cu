@@ -6,12 +6,13 @@
 //
 // Context pass (gated_recurrence_kernel).  A thread block owns 32 value columns of one (sequence, head) and keeps that
 // part of the state, dk x 32 floats, in registers over all tokens of the call: columns of the state never meet, only the
-// dk rows are summed into the output.  A thread holds R rows x 4 columns as pairs of rows for the packed fma.rn.f32x2;
-// the 8 lanes of a row group cover the 32 columns, the 4 row groups of each of the 4 warps the dk <= 16 R rows.  Tokens
-// come in blocks through a double-buffered cp.async ring, are turned into g and silu(q) once per block, and are taken
-// four at a time so that their sums over the row groups overlap; each warp leaves partial outputs in shared memory and
-// one reduction per token block adds the warps.  The blocks of a head form a cluster: its RMS norm needs all value
-// columns, and the sums of squares of a token block are exchanged through distributed shared memory.
+// dk rows are summed into the output.  Eight warps do nothing but the recurrence: a thread holds R rows x 4 columns as
+// pairs of rows for the packed fma.rn.f32x2; the 8 lanes of a row group cover the 32 columns, the 4 row groups of each
+// warp and the warps the dk <= 32 R rows; tokens are taken four at a time so that their sums over the row groups overlap.
+// Four more warps feed and drain them, a block of tokens ahead and behind: they copy the projections (cp.async), turn
+// them into g and silu(q), add the partial outputs of the eight warps, and norm and store the result.  The blocks of a
+// head form a cluster: the RMS norm needs all value columns, and the sums of squares of a token block are exchanged
+// through distributed shared memory.  One cluster barrier per token block orders everything.
 //
 // Decode step (gated_recurrence_step_kernel).  One token per sequence: the state is streamed once through registers,
 // HBM-bound; its first rows are requested before the dependency wait, because they do not depend on the kernel in front.
@@ -23,10 +24,8 @@ namespace cg = cooperative_groups;
 
 namespace onellm {
 
-constexpr int kGrThreads = 128, kGrCols = 32;
-// tokens of a block: 32, fewer where the widest float heads would not fit shared memory
-template <typename T, int R>
-constexpr int gr_tok() { return sizeof(T) == 4 && R > 8 ? 16 : 32; }
+constexpr int kGrCols = 32, kGrWarps = 8, kGrFeed = 128;  // value columns of a block; recurrence warps; feeding threads
+constexpr int kGrThreads = kGrWarps * 32 + kGrFeed;
 
 typedef unsigned long long f32x2;
 __device__ __forceinline__ f32x2 pack_f2(float lo, float hi)
@@ -87,190 +86,228 @@ struct GrParams {
 };
 
 // bytes of one raw token block: q and z rows of dk, v rows of 32 columns
-template <typename T, int R>
-__host__ __device__ constexpr size_t gr_raw_bytes(int dk) { return (size_t)gr_tok<T, R>() * (2 * dk + kGrCols) * sizeof(T); }
-template <typename T, int R>
+template <typename T, int TOK>
+__host__ __device__ constexpr size_t gr_raw_bytes(int dk) { return (size_t)TOK * (2 * dk + kGrCols) * sizeof(T); }
+// floats of one prepared token block
+template <int R, int TOK>
+__host__ __device__ constexpr int gr_block_floats() { return TOK * (2 * 32 * R + kGrCols); }
+template <typename T, int R, int TOK>
 static size_t gr_smem_bytes(int dk)
 {
-    constexpr int TOK = gr_tok<T, R>();
-    return 2 * gr_raw_bytes<T, R>(dk) + sizeof(float) * ((size_t)TOK * (2 * 16 * R + kGrCols) + 4 * TOK * kGrCols + 2 * TOK);
+    return 2 * gr_raw_bytes<T, TOK>(dk) + sizeof(float) * 2 * ((size_t)gr_block_floats<R, TOK>() + kGrWarps * TOK * kGrCols + TOK);
 }
 
-template <typename T, int R>
+template <typename T, int R, int TOK>
 __global__ void __launch_bounds__(kGrThreads) gated_recurrence_kernel(const GrParams pp)
 {
-    constexpr int TOK = gr_tok<T, R>();
-    constexpr int DKP = 16 * R;  // dk padded to whole thread tiles; the extra rows have zero gates and queries
+    constexpr int DKP = 32 * R;  // dk padded to whole thread tiles; the extra rows have zero gates and queries
     constexpr int VEC = Vec16<T>::N;
+    constexpr int BLK = gr_block_floats<R, TOK>(), PART = kGrWarps * TOK * kGrCols;
     const GatedRecurrence& p = pp.g;
     extern __shared__ __align__(16) unsigned char smem[];
     const int dk = p.dk, h = blockIdx.y, b = blockIdx.z, c0 = blockIdx.x * kGrCols;
-    const size_t raw = gr_raw_bytes<T, R>(dk);
-    float* sg = reinterpret_cast<float*>(smem + 2 * raw);
-    float* sq = sg + TOK * DKP;
-    float* sv = sq + TOK * DKP;
-    float* part = sv + TOK * kGrCols;        // [4 warps][TOK][32]
-    float* ssq = part + 4 * TOK * kGrCols;   // [2][TOK]
+    const size_t raw = gr_raw_bytes<T, TOK>(dk);
+    float* ready = reinterpret_cast<float*>(smem + 2 * raw);  // two blocks of g [TOK][DKP], silu(q) [TOK][DKP], v [TOK][32]
+    float* part = ready + 2 * BLK;                            // two blocks of [warp][TOK][32]
+    float* ssq = part + 2 * PART;                             // [2][TOK]
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int k0 = (warp * 4 + (lane >> 3)) * R, col = (lane & 7) * 4;
     cg::cluster_group cluster = cg::this_cluster();
-    const int n_peers = gridDim.x;
 
     const int tok0 = pp.tp.cu[b], n_tok = pp.tp.cu[b + 1] - tok0;
-    const bool fresh = pp.tp.hist[b] == 0;
-    float4* st = reinterpret_cast<float4*>(p.state + (((size_t)b * p.H + h) * dk) * p.dv + c0 + col);
-    const size_t st_row = (size_t)p.dv / 4;
-    f32x2 S[R / 2][4];
-#pragma unroll
-    for (int r = 0; r < R; r += 2) {
-        float4 a = make_float4(0.f, 0.f, 0.f, 0.f), c = a;
-        if (!fresh && k0 + r < dk) a = st[(size_t)(k0 + r) * st_row];
-        if (!fresh && k0 + r + 1 < dk) c = st[(size_t)(k0 + r + 1) * st_row];
-        S[r / 2][0] = pack_f2(a.x, c.x);
-        S[r / 2][1] = pack_f2(a.y, c.y);
-        S[r / 2][2] = pack_f2(a.z, c.z);
-        S[r / 2][3] = pack_f2(a.w, c.w);
-    }
-    // this thread's channels when it makes gates: k = tid % DKP of tokens tid / DKP, + 128 / DKP, ... (two channels when
-    // there are more of them than threads)
-    constexpr int KPT = DKP > kGrThreads ? DKP / kGrThreads : 1, TSTEP = DKP > kGrThreads ? 1 : kGrThreads / DKP;
-    float zb[KPT], lower[KPT];
-#pragma unroll
-    for (int i = 0; i < KPT; i++) {
-        const int k = tid % DKP + i * kGrThreads;
-        zb[i] = k < dk ? p.zb[h * dk + k] : 0.f;
-        lower[i] = k < dk ? p.lower[h * dk + k] : 0.f;
-    }
-    pdl_wait();
-    pdl_launch_dependents();
-
-    const T* q = reinterpret_cast<const T*>(p.q) + (size_t)h * dk;
-    const T* z = reinterpret_cast<const T*>(p.z) + (size_t)h * dk;
-    const T* v = reinterpret_cast<const T*>(p.v) + (size_t)h * p.dv + c0;
-    const int kc = dk / VEC, vc = kGrCols / VEC, per_tok = 2 * kc + vc;
-    const uint32_t raw_base = (uint32_t)__cvta_generic_to_shared(smem);
-    auto issue = [&](int blk) {
-        const int t0 = blk * TOK, n = min(TOK, n_tok - t0);
-        const uint32_t dst = raw_base + (uint32_t)((blk & 1) * raw);
-        for (int i = tid; i < n * per_tok; i += kGrThreads) {
-            const int t = i / per_tok, c = i % per_tok;
-            const size_t row = (size_t)(tok0 + t0 + t) * p.ld;
-            const T* src = c < kc ? q + row + c * VEC : c < 2 * kc ? z + row + (c - kc) * VEC : v + row + (c - 2 * kc) * VEC;
-            cp_async16(dst + (uint32_t)i * 16u, src, 16);
-        }
-    };
-    const float wn = p.w[c0 + lane] * p.out_scale;
     const int n_blk = (n_tok + TOK - 1) / TOK;
-    if (n_blk > 0) issue(0);
-    cp_async_commit();
-    for (int blk = 0; blk < n_blk; blk++) {
-        if (blk + 1 < n_blk) issue(blk + 1);
-        cp_async_commit();
-        cp_async_wait<1>();
-        __syncthreads();
-        const int n = min(TOK, n_tok - blk * TOK), n4 = (n + 3) & ~3;  // tokens n .. n4 - 1 change nothing: g = q = 0
-        const T* rb = reinterpret_cast<const T*>(smem + (size_t)(blk & 1) * raw);
-        const int row_el = 2 * dk + kGrCols;
-#pragma unroll
-        for (int i = 0; i < KPT; i++) {
-            const int k = tid % DKP + i * kGrThreads;
-#pragma unroll 4
-            for (int t = tid / DKP; t < n4; t += TSTEP) {
-                float g = 0.f, qs = 0.f;
-                if (k < dk && t < n) gate<T>(to_float(rb[t * row_el + k]), to_float(rb[t * row_el + dk + k]), zb[i], lower[i], g, qs);
-                sg[t * DKP + k] = g;
-                sq[t * DKP + k] = qs;
-            }
-        }
-        for (int t = warp; t < n4; t += 4) sv[t * kGrCols + lane] = t < n ? to_float(rb[t * row_el + 2 * dk + lane]) : 0.f;
-        __syncthreads();
-        for (int t = 0; t < n4; t += 4) {
-            f32x2 o2[4][4];
-#pragma unroll
-            for (int u = 0; u < 4; u++) {
-                const float4 v4 = *reinterpret_cast<const float4*>(sv + (t + u) * kGrCols + col);
-                const f32x2 vv[4] = {pack_f2(v4.x, v4.x), pack_f2(v4.y, v4.y), pack_f2(v4.z, v4.z), pack_f2(v4.w, v4.w)};
-                f32x2 g2[R / 2], q2[R / 2];
-                const float *gt = sg + (t + u) * DKP + k0, *qt = sq + (t + u) * DKP + k0;
-                if constexpr (R >= 4) {
-#pragma unroll
-                    for (int r = 0; r < R / 2; r += 2) {
-                        *reinterpret_cast<ulonglong2*>(&g2[r]) = *reinterpret_cast<const ulonglong2*>(gt + 2 * r);
-                        *reinterpret_cast<ulonglong2*>(&q2[r]) = *reinterpret_cast<const ulonglong2*>(qt + 2 * r);
-                    }
-                } else {
-                    g2[0] = *reinterpret_cast<const f32x2*>(gt);
-                    q2[0] = *reinterpret_cast<const f32x2*>(qt);
-                }
-#pragma unroll
-                for (int c = 0; c < 4; c++) o2[u][c] = 0ull;
-#pragma unroll
-                for (int r = 0; r < R / 2; r++)
-#pragma unroll
-                    for (int c = 0; c < 4; c++) {
-                        S[r][c] = fma_f2(g2[r], sub_f2(vv[c], S[r][c]), S[r][c]);
-                        o2[u][c] = fma_f2(q2[r], S[r][c], o2[u][c]);
-                    }
-            }
-            // sum over the row groups of the warp; a lane keeps one column: halves first (columns 0-1 | 2-3), then one of two
-            const bool hi2 = lane & 16, hi1 = lane & 8;
-#pragma unroll
-            for (int u = 0; u < 4; u++) {
-                const float o[4] = {sum_f2(o2[u][0]), sum_f2(o2[u][1]), sum_f2(o2[u][2]), sum_f2(o2[u][3])};
-                float a0 = hi2 ? o[2] : o[0], a1 = hi2 ? o[3] : o[1];
-                a0 += __shfl_xor_sync(0xffffffffu, hi2 ? o[0] : o[2], 16);
-                a1 += __shfl_xor_sync(0xffffffffu, hi2 ? o[1] : o[3], 16);
-                const float a = (hi1 ? a1 : a0) + __shfl_xor_sync(0xffffffffu, hi1 ? a0 : a1, 8);
-                part[(warp * TOK + t + u) * kGrCols + col + (hi2 ? 2 : 0) + (hi1 ? 1 : 0)] = a;
-            }
-        }
-        __syncthreads();
-        // one warp per token row: add the warps' partial sums, sum of squares of the 32 columns
-        float o[TOK / 4];
-        float* ss_now = ssq + (blk & 1) * TOK;
-#pragma unroll
-        for (int i = 0; i < TOK / 4; i++) {
-            const int t = warp + 4 * i;
-            o[i] = 0.f;
-            if (t < n) {
-#pragma unroll
-                for (int w = 0; w < 4; w++) o[i] += part[(w * TOK + t) * kGrCols + lane];
-                const float s = warp_sum(o[i] * o[i]);
-                if (lane == 0) ss_now[t] = s;
-            }
-        }
-        // Every block of the cluster has written its sums; they stay valid for one more round (two buffers), and a block
-        // that writes that buffer again has passed the next round's barrier, behind everyone's reads of this one.
-        cluster.sync();
-        // lane t of every warp adds the cluster's sums of token t
-        float inv = 0.f;
-        if (lane < n) {
-            float s = 0.f;
-            for (int r = 0; r < n_peers; r++) s += cluster.map_shared_rank(ss_now, r)[lane];
-            inv = 1.0f / sqrtf(s / (float)p.norm_width + p.eps);
-        }
-#pragma unroll
-        for (int i = 0; i < TOK / 4; i++) {
-            const int t = warp + 4 * i;
-            const float f = __shfl_sync(0xffffffffu, inv, t);
-            if (t < n) {
-                T* dst = reinterpret_cast<T*>(p.out) + (size_t)(tok0 + blk * TOK + t) * p.out_ld + (size_t)h * p.dv + c0 + lane;
-                *dst = from_float<T>(o[i] * f * wn);
-            }
-        }
-    }
-    cp_async_wait<0>();
-    if (n_tok > 0) {
+    if (warp < kGrWarps) {
+        // ---- the recurrence
+        const int k0 = (warp * 4 + (lane >> 3)) * R, col = (lane & 7) * 4;
+        const bool fresh = pp.tp.hist[b] == 0;
+        float4* st = reinterpret_cast<float4*>(p.state + (((size_t)b * p.H + h) * dk) * p.dv + c0 + col);
+        const size_t st_row = (size_t)p.dv / 4;
+        f32x2 S[R / 2][4];
 #pragma unroll
         for (int r = 0; r < R; r += 2) {
-            float a[4], c[4];
-#pragma unroll
-            for (int j = 0; j < 4; j++) asm("mov.b64 {%0, %1}, %2;" : "=f"(a[j]), "=f"(c[j]) : "l"(S[r / 2][j]));
-            if (k0 + r < dk) st[(size_t)(k0 + r) * st_row] = make_float4(a[0], a[1], a[2], a[3]);
-            if (k0 + r + 1 < dk) st[(size_t)(k0 + r + 1) * st_row] = make_float4(c[0], c[1], c[2], c[3]);
+            float4 a = make_float4(0.f, 0.f, 0.f, 0.f), c = a;
+            if (!fresh && k0 + r < dk) a = st[(size_t)(k0 + r) * st_row];
+            if (!fresh && k0 + r + 1 < dk) c = st[(size_t)(k0 + r + 1) * st_row];
+            S[r / 2][0] = pack_f2(a.x, c.x);
+            S[r / 2][1] = pack_f2(a.y, c.y);
+            S[r / 2][2] = pack_f2(a.z, c.z);
+            S[r / 2][3] = pack_f2(a.w, c.w);
         }
+        pdl_wait();
+        pdl_launch_dependents();
+        const bool hi2 = lane & 16, hi1 = lane & 8;
+        const int my_col = col + (hi2 ? 2 : 0) + (hi1 ? 1 : 0);
+        cluster.sync();  // block 0 is prepared
+        for (int it = 0; it < n_blk + 2; it++) {
+            if (it < n_blk) {
+                const float* sg = ready + (it & 1) * BLK + k0;
+                const float* sq = sg + TOK * DKP;
+                const float* sv = ready + (it & 1) * BLK + 2 * TOK * DKP + col;
+                float* dst = part + (it & 1) * PART + warp * TOK * kGrCols + my_col;
+                const int n4 = (min(TOK, n_tok - it * TOK) + 3) & ~3;  // tokens behind the end have g = q = v = 0
+                for (int t = 0; t < n4; t += 4) {
+                    f32x2 o2[4][4];
+#pragma unroll
+                    for (int u = 0; u < 4; u++) {
+                        const float4 v4 = *reinterpret_cast<const float4*>(sv + (t + u) * kGrCols);
+                        const f32x2 vv[4] = {pack_f2(v4.x, v4.x), pack_f2(v4.y, v4.y), pack_f2(v4.z, v4.z), pack_f2(v4.w, v4.w)};
+                        f32x2 g2[R / 2], q2[R / 2];
+                        const float *gt = sg + (t + u) * DKP, *qt = sq + (t + u) * DKP;
+                        if constexpr (R >= 4) {
+#pragma unroll
+                            for (int r = 0; r < R / 2; r += 2) {
+                                *reinterpret_cast<ulonglong2*>(&g2[r]) = *reinterpret_cast<const ulonglong2*>(gt + 2 * r);
+                                *reinterpret_cast<ulonglong2*>(&q2[r]) = *reinterpret_cast<const ulonglong2*>(qt + 2 * r);
+                            }
+                        } else {
+                            g2[0] = *reinterpret_cast<const f32x2*>(gt);
+                            q2[0] = *reinterpret_cast<const f32x2*>(qt);
+                        }
+#pragma unroll
+                        for (int c = 0; c < 4; c++) o2[u][c] = 0ull;
+#pragma unroll
+                        for (int r = 0; r < R / 2; r++)
+#pragma unroll
+                            for (int c = 0; c < 4; c++) {
+                                S[r][c] = fma_f2(g2[r], sub_f2(vv[c], S[r][c]), S[r][c]);
+                                o2[u][c] = fma_f2(q2[r], S[r][c], o2[u][c]);
+                            }
+                    }
+                    // sum over the row groups of the warp; a lane keeps one column: halves first (columns 0-1 | 2-3), then
+                    // one of two
+#pragma unroll
+                    for (int u = 0; u < 4; u++) {
+                        const float o[4] = {sum_f2(o2[u][0]), sum_f2(o2[u][1]), sum_f2(o2[u][2]), sum_f2(o2[u][3])};
+                        float a0 = hi2 ? o[2] : o[0], a1 = hi2 ? o[3] : o[1];
+                        a0 += __shfl_xor_sync(0xffffffffu, hi2 ? o[0] : o[2], 16);
+                        a1 += __shfl_xor_sync(0xffffffffu, hi2 ? o[1] : o[3], 16);
+                        dst[(t + u) * kGrCols] = (hi1 ? a1 : a0) + __shfl_xor_sync(0xffffffffu, hi1 ? a0 : a1, 8);
+                    }
+                }
+            }
+            cluster.sync();
+        }
+        if (n_tok > 0) {
+#pragma unroll
+            for (int r = 0; r < R; r += 2) {
+                float a[4], c[4];
+#pragma unroll
+                for (int j = 0; j < 4; j++) asm("mov.b64 {%0, %1}, %2;" : "=f"(a[j]), "=f"(c[j]) : "l"(S[r / 2][j]));
+                if (k0 + r < dk) st[(size_t)(k0 + r) * st_row] = make_float4(a[0], a[1], a[2], a[3]);
+                if (k0 + r + 1 < dk) st[(size_t)(k0 + r + 1) * st_row] = make_float4(c[0], c[1], c[2], c[3]);
+            }
+        }
+    } else {
+        // ---- feed and drain
+        const int ft = tid - kGrWarps * 32, fw = ft >> 5;
+        const int n_peers = gridDim.x;
+        // the channels whose gates this thread makes: ft % DKP of tokens ft / DKP, + 128 / DKP, ... (two channels when there
+        // are more of them than threads)
+        constexpr int KPT = DKP > kGrFeed ? DKP / kGrFeed : 1, TSTEP = DKP > kGrFeed ? 1 : kGrFeed / DKP;
+        float zb[KPT], lower[KPT];
+#pragma unroll
+        for (int i = 0; i < KPT; i++) {
+            const int k = min(ft % DKP + i * kGrFeed, dk - 1);
+            zb[i] = p.zb[h * dk + k];
+            lower[i] = p.lower[h * dk + k];
+        }
+        const float wn = p.w[c0 + lane] * p.out_scale;
+        pdl_wait();
+        pdl_launch_dependents();
+        const T* q = reinterpret_cast<const T*>(p.q) + (size_t)h * dk;
+        const T* z = reinterpret_cast<const T*>(p.z) + (size_t)h * dk;
+        const T* v = reinterpret_cast<const T*>(p.v) + (size_t)h * p.dv + c0;
+        const int kc = dk / VEC, per_tok = 2 * kc + kGrCols / VEC;
+        const uint32_t raw_base = (uint32_t)__cvta_generic_to_shared(smem);
+        auto issue = [&](int blk) {  // a warp copies whole tokens
+            if (blk < n_blk) {
+                const int t0 = blk * TOK, n = min(TOK, n_tok - t0);
+                for (int t = fw; t < n; t += kGrFeed / 32) {
+                    const size_t row = (size_t)(tok0 + t0 + t) * p.ld;
+                    const uint32_t dst = raw_base + (uint32_t)((blk & 1) * raw) + (uint32_t)(t * per_tok) * 16u;
+                    for (int c = lane; c < per_tok; c += 32) {
+                        const T* src = c < kc ? q + row + c * VEC : c < 2 * kc ? z + row + (c - kc) * VEC : v + row + (c - 2 * kc) * VEC;
+                        cp_async16(dst + c * 16u, src, 16);
+                    }
+                }
+            }
+            cp_async_commit();
+        };
+        auto prepare = [&](int blk) {  // the copies of this block were issued one call ago
+            cp_async_wait<0>();
+            asm volatile("bar.sync 1, %0;" ::"n"(kGrFeed) : "memory");  // the feeding threads' copies of the block, and their reads of the one before
+            issue(blk + 1);
+            if (blk >= n_blk) return;
+            const int n = min(TOK, n_tok - blk * TOK), n4 = (n + 3) & ~3;
+            const T* rb = reinterpret_cast<const T*>(smem + (size_t)(blk & 1) * raw);
+            const int row_el = 2 * dk + kGrCols;
+            float* sg = ready + (blk & 1) * BLK;
+            float* sq = sg + TOK * DKP;
+            float* sv = sq + TOK * DKP;
+#pragma unroll
+            for (int i = 0; i < KPT; i++) {
+                const int k = ft % DKP + i * kGrFeed, kk = min(k, dk - 1);
+#pragma unroll 4
+                for (int t = ft / DKP; t < n4; t += TSTEP) {
+                    const T* row = rb + min(t, n - 1) * row_el + kk;
+                    float g, qs;
+                    gate<T>(to_float(row[0]), to_float(row[dk]), zb[i], lower[i], g, qs);
+                    const bool real = k < dk && t < n;
+                    sg[t * DKP + k] = real ? g : 0.f;
+                    sq[t * DKP + k] = real ? qs : 0.f;
+                }
+            }
+#pragma unroll 4
+            for (int t = fw; t < n4; t += kGrFeed / 32) {
+                const float x = to_float(rb[min(t, n - 1) * row_el + 2 * dk + lane]);
+                sv[t * kGrCols + lane] = t < n ? x : 0.f;
+            }
+        };
+        issue(0);
+        prepare(0);
+        cluster.sync();
+        float o[TOK / 4];  // outputs of token fw + 4 i, column `lane`, of the block summed last
+        for (int it = 0; it < n_blk + 2; it++) {
+            prepare(it + 1);
+            if (it >= 2) {
+                // norm and store block it - 2: every block of the cluster left its sums before the last barrier, and writes
+                // that buffer again behind the next one
+                const int blk = it - 2, n = min(TOK, n_tok - blk * TOK);
+                float inv = 0.f;
+                if (lane < TOK) {
+                    float* mine = ssq + (blk & 1) * TOK;
+                    float s[8];
+#pragma unroll
+                    for (int r = 0; r < 8; r++) s[r] = r < n_peers ? cluster.map_shared_rank(mine, r)[lane] : 0.f;
+                    inv = 1.0f / sqrtf((((s[0] + s[1]) + (s[2] + s[3])) + ((s[4] + s[5]) + (s[6] + s[7]))) / (float)p.norm_width + p.eps);
+                }
+                T* dst = reinterpret_cast<T*>(p.out) + (size_t)(tok0 + blk * TOK) * p.out_ld + (size_t)h * p.dv + c0 + lane;
+#pragma unroll
+                for (int i = 0; i < TOK / 4; i++) {
+                    const int t = fw + 4 * i;
+                    const float f = __shfl_sync(0xffffffffu, inv, t);
+                    if (t < n) dst[(size_t)t * p.out_ld] = from_float<T>(o[i] * f * wn);
+                }
+            }
+            if (it >= 1 && it <= n_blk) {
+                // add the warps' partial outputs of block it - 1 (rows behind its end are whatever was there: never stored)
+                const float* src = part + ((it - 1) & 1) * PART + lane;
+                float* mine = ssq + ((it - 1) & 1) * TOK;
+#pragma unroll
+                for (int i = 0; i < TOK / 4; i++) {
+                    o[i] = 0.f;
+#pragma unroll
+                    for (int w = 0; w < kGrWarps; w++) o[i] += src[(w * TOK + fw + 4 * i) * kGrCols];
+                }
+#pragma unroll
+                for (int i = 0; i < TOK / 4; i++) {
+                    const float s = warp_sum(o[i] * o[i]);
+                    if (lane == 0) mine[fw + 4 * i] = s;
+                }
+            }
+            cluster.sync();
+        }
+        cp_async_wait<0>();
     }
-    cluster.sync();  // peers may still be reading this block's sums
 }
 
 // One token per sequence.  A block owns `cols` value columns of one (sequence, head); cols / 4 threads share a row and
@@ -386,13 +423,13 @@ static int launch_cluster(Kernel kern, dim3 grid, int threads, size_t smem, cuda
     return ONELLM_OK;
 }
 
-template <typename T, int R>
+template <typename T, int R, int TOK>
 static int launch_gr(const GrParams& p, int B, cudaStream_t st)
 {
-    auto kern = gated_recurrence_kernel<T, R>;
+    auto kern = gated_recurrence_kernel<T, R, TOK>;
     static DeviceOnce attr;
     ONELLM_CUDA(attr.run([kern] { return cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024); }));
-    return launch_cluster(kern, dim3(p.g.dv / kGrCols, p.g.H, B), kGrThreads, gr_smem_bytes<T, R>(p.g.dk), st, p);
+    return launch_cluster(kern, dim3(p.g.dv / kGrCols, p.g.H, B), kGrThreads, gr_smem_bytes<T, R, TOK>(p.g.dk), st, p);
 }
 
 template <typename T>
@@ -405,11 +442,15 @@ static int dispatch_gr(const GrParams& p, int B, cudaStream_t st)
             if (p.g.dv % (32 * n) == 0) cols = p.g.dv / n;
         return launch_cluster(gated_recurrence_step_kernel<T>, dim3(p.g.dv / cols, p.g.H, B), kGsThreads, 0, st, p, cols);
     }
+    // token blocks of 32 where one thread block per SM is all there is, else of 16 (two thread blocks share an SM)
     const int dk = p.g.dk;
-    if (dk <= 32) return launch_gr<T, 2>(p, B, st);
-    if (dk <= 64) return launch_gr<T, 4>(p, B, st);
-    if (dk <= 128) return launch_gr<T, 8>(p, B, st);
-    return launch_gr<T, 16>(p, B, st);
+    if constexpr (sizeof(T) == 2) {
+        if (dk <= 128 && (long)B * p.g.H * (p.g.dv / kGrCols) <= num_sms())
+            return dk <= 64 ? launch_gr<T, 2, 32>(p, B, st) : launch_gr<T, 4, 32>(p, B, st);
+    }
+    if (dk <= 64) return launch_gr<T, 2, 16>(p, B, st);
+    if (dk <= 128) return launch_gr<T, 4, 16>(p, B, st);
+    return launch_gr<T, 8, 16>(p, B, st);
 }
 
 int gated_recurrence(const GatedRecurrence& g, const TokenPositions& tp, int B, cudaStream_t st)
