@@ -512,7 +512,8 @@ ONELLM_API int onellm_biased_attn_decode(const onellm_biased_attn* a, const onel
  *     f = lower + (1 - lower) * sigmoid(z + zb)     state = diag(f) state + (1 - f) v^T     o = state^T silu(q)
  *     out = o * rsqrt(sum(o^2) / norm_width + eps) * w * out_scale
  * q, z, v: token t at + t * ld, heads dk / dk / dv apart; zb, lower [H * dk]; w [dv]; state [B, H, dk, dv], taken as zero
- * for a sequence at its first position. */
+ * for a sequence at its first position.  work: scratch of a context pass, onellm_gated_recurrence_workspace bytes for its
+ * tokens, 16-byte aligned (unused by a decode step). */
 typedef struct onellm_gated_recurrence {
     int dtype;
     int H, dk, dv;
@@ -526,8 +527,11 @@ typedef struct onellm_gated_recurrence {
     void* out;
     long out_ld;
     float out_scale;
+    void* work;
 } onellm_gated_recurrence;
-ONELLM_API int onellm_gated_recurrence_run(const onellm_gated_recurrence* g, const onellm_token_positions* tp, int B, void* stream);
+ONELLM_API size_t onellm_gated_recurrence_workspace(int tokens, int H, int dk, int dv);
+/* tokens: of the whole launch (context pass: cu[B]). */
+ONELLM_API int onellm_gated_recurrence_run(const onellm_gated_recurrence* g, const onellm_token_positions* tp, int tokens, void* stream);
 
 /* RMSNorm with weights stored around zero, out of a float stream into one or two buffers (out2 may be NULL):
  *     out_i[r] = x[r or rows[r]] * rsqrt(mean(x^2) + eps) * (1 + w_i)

@@ -54,7 +54,7 @@ class GatedRecurrence(C.Structure):
     _fields_ = [("dtype", C.c_int), ("H", C.c_int), ("dk", C.c_int), ("dv", C.c_int),
                 ("q", C.c_void_p), ("z", C.c_void_p), ("v", C.c_void_p), ("ld", C.c_long), ("zb", C.c_void_p), ("lower", C.c_void_p),
                 ("w", C.c_void_p), ("eps", C.c_float), ("norm_width", C.c_int), ("state", C.c_void_p),
-                ("out", C.c_void_p), ("out_ld", C.c_long), ("out_scale", C.c_float)]
+                ("out", C.c_void_p), ("out_ld", C.c_long), ("out_scale", C.c_float), ("work", C.c_void_p)]
 
 
 def lib() -> C.CDLL:
@@ -68,7 +68,7 @@ def lib() -> C.CDLL:
         for name, restype in (("onellm_last_error", C.c_char_p), ("onellm_decode_attn_workspace_bytes", C.c_size_t),
                               ("onellm_decode_attn_static_scratch_bytes", C.c_size_t), ("onellm_llama_device_bytes", C.c_size_t),
                               ("onellm_llama_stream", C.c_void_p), ("onellm_llama_destroy", None), ("onellm_model_design", C.c_char_p),
-                              ("onellm_biased_attn_decode_workspace", C.c_size_t)):
+                              ("onellm_biased_attn_decode_workspace", C.c_size_t), ("onellm_gated_recurrence_workspace", C.c_size_t)):
             if hasattr(l, name):  # a library built for one design has its entry points only
                 getattr(l, name).restype = restype
         _lib = l
@@ -338,8 +338,12 @@ def biased_attn_decode(a, tp, step_bound, workspace, stream=None):
     _check(lib().onellm_biased_attn_decode(C.byref(a), C.byref(tp), C.c_int(step_bound), _p(workspace), _stream(stream)))
 
 
-def gated_recurrence(g, tp, B, stream=None):
-    _check(lib().onellm_gated_recurrence_run(C.byref(g), C.byref(tp), C.c_int(B), _stream(stream)))
+def gated_recurrence_workspace(tokens, H, dk, dv):
+    return int(lib().onellm_gated_recurrence_workspace(C.c_int(tokens), C.c_int(H), C.c_int(dk), C.c_int(dv)))
+
+
+def gated_recurrence(g, tp, tokens, stream=None):
+    _check(lib().onellm_gated_recurrence_run(C.byref(g), C.byref(tp), C.c_int(tokens), _stream(stream)))
 
 
 def norm_pair(dtype, x, rows, n_rows, w1, w2, out1, out2, eps, width, ld, stream=None):

@@ -155,6 +155,7 @@ struct Finuvik : Engine {
     struct Buffers {
         float* x;
         void *h1, *h2, *mix, *cat;
+        void* rec_work;  // context pass only
     };
     int layer(size_t i, const Buffers& buf, int tokens, const TokenPositions& tp, int max_new, int step_bound);
     int lm_head(const float* stream_rows, const int* rows, int n_rows, void* hn, float* padded, float* out);
@@ -290,7 +291,8 @@ int Finuvik::layer(size_t i, const Buffers& buf, int tokens, const TokenPosition
     g.out = at(buf.cat, w.cat_r);
     g.out_ld = w.n_cat;
     g.out_scale = (float)l.right_scale;
-    RC(gated_recurrence(g, tp, tp.B, stream));
+    g.work = buf.rec_work;
+    RC(gated_recurrence(g, tp, tp.B, tokens, stream));
     pj = Projection{};
     pj.dtype = dtype;
     pj.M = tokens;
@@ -328,7 +330,7 @@ int Finuvik::decode_layers(int step_bound, bool with_head)
 {
     const TokenPositions tp = {nullptr, nullptr, batch, d_step, d_step_off};
     RC(embedding_pos_launch(dtype, d_ids, x, embed, pos, batch, width, c.vocab, max_seq_len, tp, d_bad_id, stream));
-    const Buffers buf = {x, h1, h2, mix, cat};
+    const Buffers buf = {x, h1, h2, mix, cat, nullptr};
     for (size_t i = 0; i < c.layers.size(); i++) RC(layer(i, buf, batch, tp, 1, step_bound));
     return with_head ? lm_head(x, nullptr, batch, h1, logits_p, static_cast<float*>(logits)) : ONELLM_OK;
 }
@@ -346,6 +348,10 @@ int Finuvik::context_layers(const ContextBatch& cb)
         buf.h2 = cv.take_bytes(T * W * es);
         buf.mix = cv.take_bytes(T * max_mix * es);
         buf.cat = cv.take_bytes(T * max_cat * es);
+        size_t work = 0;
+        for (size_t i = 0; i < c.layers.size(); i++)
+            work = std::max(work, gated_recurrence_workspace((int)T, c.layers[i].RH, weights[i].rk, weights[i].rv));
+        buf.rec_work = cv.take_bytes(work);
         hn = cv.take_bytes((size_t)cb.n_rows * W * es);
         padded = vocab_p == c.vocab ? nullptr : cv.take<float>((size_t)cb.n_rows * vocab_p);
         if (pass == 0) {

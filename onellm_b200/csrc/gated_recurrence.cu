@@ -4,28 +4,35 @@
 //     s <- s + g (v - s)
 // which needs one multiply-add and keeps the digits of a gate near one (g comes from the complementary sigmoid).
 //
-// Context pass (gated_recurrence_kernel).  A thread block owns 32 value columns of one (sequence, head) and keeps that
-// part of the state, dk x 32 floats, in registers over all tokens of the call: columns of the state never meet, only the
-// dk rows are summed into the output.  Eight warps do nothing but the recurrence: a thread holds R rows x 4 columns as
-// pairs of rows for the packed fma.rn.f32x2; the 8 lanes of a row group cover the 32 columns, the 4 row groups of each
-// warp and the warps the dk <= 32 R rows; tokens are taken four at a time so that their sums over the row groups overlap.
-// Four more warps feed and drain them, a block of tokens ahead and behind: they copy the projections (cp.async), turn
-// them into g and silu(q), add the partial outputs of the eight warps, and norm and store the result.  The blocks of a
-// head form a cluster: the RMS norm needs all value columns, and the sums of squares of a token block are exchanged
-// through distributed shared memory.  One cluster barrier per token block orders everything.
+// Context pass, three launches:
+//   1. gated_recurrence_prepare_kernel turns the projections into g and silu(q), in float and head by head, so that the
+//      tokens of a head lie behind each other.
+//   2. gated_recurrence_scan_kernel.  A thread block owns 32 value columns of one (sequence, head) and keeps that part of
+//      the state, dk x 32 floats, in registers over all tokens of the call: columns of the state never meet, only the dk
+//      rows are summed into the output.  A thread holds R rows x 4 columns as pairs of rows for the packed fma.rn.f32x2;
+//      the 8 lanes of a row group cover the 32 columns, the 4 row groups of each of the 8 warps the dk <= 32 R rows;
+//      tokens are taken four at a time so that their sums over the row groups overlap.  Blocks of tokens arrive by bulk
+//      copies (one for g and q, one for v) in two stages; one block barrier per token block, behind which the warps add
+//      their partial outputs.
+//   3. gated_recurrence_norm_kernel: RMS norm per head, output in the element type.
+// (One launch that made the gates itself, once per value tile, and normed through a cluster spent two thirds of its time
+// outside the recurrence.)
 //
 // Decode step (gated_recurrence_step_kernel).  One token per sequence: the state is streamed once through registers,
 // HBM-bound; its first rows are requested before the dependency wait, because they do not depend on the kernel in front.
 #include <cooperative_groups.h>
 
+#include <algorithm>
+
 #include "mixers.h"
+#include "tc_common.cuh"
 
 namespace cg = cooperative_groups;
 
 namespace onellm {
 
-constexpr int kGrCols = 32, kGrWarps = 8, kGrFeed = 128;  // value columns of a block; recurrence warps; feeding threads
-constexpr int kGrThreads = kGrWarps * 32 + kGrFeed;
+constexpr int kGrCols = 32, kGrWarps = 8;  // value columns of a block; warps
+constexpr int kGrThreads = kGrWarps * 32;
 
 typedef unsigned long long f32x2;
 __device__ __forceinline__ f32x2 pack_f2(float lo, float hi)
@@ -85,229 +92,228 @@ struct GrParams {
     TokenPositions tp;
 };
 
-// bytes of one raw token block: q and z rows of dk, v rows of 32 columns
-template <typename T, int TOK>
-__host__ __device__ constexpr size_t gr_raw_bytes(int dk) { return (size_t)TOK * (2 * dk + kGrCols) * sizeof(T); }
-// floats of one prepared token block
-template <int R, int TOK>
-__host__ __device__ constexpr int gr_block_floats() { return TOK * (2 * 32 * R + kGrCols); }
-template <typename T, int R, int TOK>
-static size_t gr_smem_bytes(int dk)
+// Layout of the work space of T tokens: g and silu(q) [H][T][2 * dkp], v [H][dv / 32][T][32], outputs before the norm
+// [T][H][dv]; all float, dkp = dk padded to the rows of a block.
+static int gr_dkp(int dk) { return dk <= 64 ? 64 : dk <= 128 ? 128 : 256; }
+
+template <typename T>
+__global__ void __launch_bounds__(256) gated_recurrence_prepare_kernel(const GrParams pp, int tokens, int dkp, float* __restrict__ gq, float* __restrict__ vf)
 {
-    return 2 * gr_raw_bytes<T, TOK>(dk) + sizeof(float) * 2 * ((size_t)gr_block_floats<R, TOK>() + kGrWarps * TOK * kGrCols + TOK);
+    const GatedRecurrence& p = pp.g;
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x, dk = p.dk, dv = p.dv;
+    const T* q = reinterpret_cast<const T*>(p.q) + (size_t)t * p.ld;
+    const T* z = reinterpret_cast<const T*>(p.z) + (size_t)t * p.ld;
+    const T* v = reinterpret_cast<const T*>(p.v) + (size_t)t * p.ld;
+    auto load4 = [](const T* src, float (&f)[4]) {
+        if constexpr (sizeof(T) == 4) {
+            const float4 x = *reinterpret_cast<const float4*>(src);
+            f[0] = x.x; f[1] = x.y; f[2] = x.z; f[3] = x.w;
+        } else {
+            const uint2 x = *reinterpret_cast<const uint2*>(src);
+            const float2 a = unpack2<T>(x.x), b = unpack2<T>(x.y);
+            f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+        }
+    };
+    const int nq = p.H * (dkp / 4);
+    for (int i = threadIdx.x; i < nq; i += blockDim.x) {
+        const int h = i / (dkp / 4), k = (i % (dkp / 4)) * 4;
+        float g[4] = {0.f, 0.f, 0.f, 0.f}, qs[4] = {0.f, 0.f, 0.f, 0.f};  // rows behind dk change nothing
+        if (k < dk) {
+            const int c = h * dk + k;
+            float qv[4], zv[4];
+            load4(q + c, qv);
+            load4(z + c, zv);
+            const float4 zb = *reinterpret_cast<const float4*>(p.zb + c), lo = *reinterpret_cast<const float4*>(p.lower + c);
+            gate<T>(qv[0], zv[0], zb.x, lo.x, g[0], qs[0]);
+            gate<T>(qv[1], zv[1], zb.y, lo.y, g[1], qs[1]);
+            gate<T>(qv[2], zv[2], zb.z, lo.z, g[2], qs[2]);
+            gate<T>(qv[3], zv[3], zb.w, lo.w, g[3], qs[3]);
+        }
+        float* dst = gq + ((size_t)h * tokens + t) * 2 * dkp + k;
+        *reinterpret_cast<float4*>(dst) = make_float4(g[0], g[1], g[2], g[3]);
+        *reinterpret_cast<float4*>(dst + dkp) = make_float4(qs[0], qs[1], qs[2], qs[3]);
+    }
+    for (int i = threadIdx.x; i < p.H * (dv / 4); i += blockDim.x) {
+        const int c = i * 4, tile = c / kGrCols;  // tiles of all heads in a row: h * (dv / 32) + tile of the head
+        float x[4];
+        load4(v + c, x);
+        *reinterpret_cast<float4*>(vf + ((size_t)tile * tokens + t) * kGrCols + c % kGrCols) = make_float4(x[0], x[1], x[2], x[3]);
+    }
 }
 
-template <typename T, int R, int TOK>
-__global__ void __launch_bounds__(kGrThreads) gated_recurrence_kernel(const GrParams pp)
+__device__ __forceinline__ void bulk_load(uint32_t dst, const void* src, uint32_t bytes, uint32_t bar)
 {
-    constexpr int DKP = 32 * R;  // dk padded to whole thread tiles; the extra rows have zero gates and queries
-    constexpr int VEC = Vec16<T>::N;
-    constexpr int BLK = gr_block_floats<R, TOK>(), PART = kGrWarps * TOK * kGrCols;
-    const GatedRecurrence& p = pp.g;
-    extern __shared__ __align__(16) unsigned char smem[];
-    const int dk = p.dk, h = blockIdx.y, b = blockIdx.z, c0 = blockIdx.x * kGrCols;
-    const size_t raw = gr_raw_bytes<T, TOK>(dk);
-    float* ready = reinterpret_cast<float*>(smem + 2 * raw);  // two blocks of g [TOK][DKP], silu(q) [TOK][DKP], v [TOK][32]
-    float* part = ready + 2 * BLK;                            // two blocks of [warp][TOK][32]
-    float* ssq = part + 2 * PART;                             // [2][TOK]
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    cg::cluster_group cluster = cg::this_cluster();
+    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst), "l"(src), "r"(bytes), "r"(bar)
+                 : "memory");
+}
 
-    const int tok0 = pp.tp.cu[b], n_tok = pp.tp.cu[b + 1] - tok0;
-    const int n_blk = (n_tok + TOK - 1) / TOK;
-    if (warp < kGrWarps) {
-        // ---- the recurrence
-        const int k0 = (warp * 4 + (lane >> 3)) * R, col = (lane & 7) * 4;
-        const bool fresh = pp.tp.hist[b] == 0;
-        float4* st = reinterpret_cast<float4*>(p.state + (((size_t)b * p.H + h) * dk) * p.dv + c0 + col);
-        const size_t st_row = (size_t)p.dv / 4;
-        f32x2 S[R / 2][4];
+template <int R, int TOK>
+constexpr size_t gr_smem_bytes() { return sizeof(float) * 2 * ((size_t)TOK * (2 * 32 * R + kGrCols) + (size_t)kGrWarps * TOK * kGrCols); }
+
+template <int R, int TOK>
+__global__ void __launch_bounds__(kGrThreads)
+gated_recurrence_scan_kernel(const GrParams pp, int tokens, const float* __restrict__ gq, const float* __restrict__ vf, float* __restrict__ of)
+{
+    constexpr int DKP = 32 * R;
+    constexpr int STAGE = TOK * (2 * DKP + kGrCols), PART = kGrWarps * TOK * kGrCols;  // floats
+    const GatedRecurrence& p = pp.g;
+    extern __shared__ __align__(128) float smem_f[];
+    float* part = smem_f + 2 * STAGE;
+    __shared__ __align__(8) uint64_t bars[2];
+    const int dk = p.dk, h = blockIdx.y, b = blockIdx.z, c0 = blockIdx.x * kGrCols;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int k0 = (warp * 4 + (lane >> 3)) * R, col = (lane & 7) * 4;
+    const int tok0 = pp.tp.cu[b], n_tok = pp.tp.cu[b + 1] - tok0, n_blk = (n_tok + TOK - 1) / TOK;
+    const bool fresh = pp.tp.hist[b] == 0;
+    if (tid == 0) {
+        mbar_init(smem_u32(&bars[0]), 1);
+        mbar_init(smem_u32(&bars[1]), 1);
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    // the state was written by an earlier call: it does not depend on the kernel in front of this one
+    float4* st = reinterpret_cast<float4*>(p.state + (((size_t)b * p.H + h) * dk) * p.dv + c0 + col);
+    const size_t st_row = (size_t)p.dv / 4;
+    f32x2 S[R / 2][4];
+#pragma unroll
+    for (int r = 0; r < R; r += 2) {
+        float4 a = make_float4(0.f, 0.f, 0.f, 0.f), c = a;
+        if (!fresh && k0 + r < dk) a = st[(size_t)(k0 + r) * st_row];
+        if (!fresh && k0 + r + 1 < dk) c = st[(size_t)(k0 + r + 1) * st_row];
+        S[r / 2][0] = pack_f2(a.x, c.x);
+        S[r / 2][1] = pack_f2(a.y, c.y);
+        S[r / 2][2] = pack_f2(a.z, c.z);
+        S[r / 2][3] = pack_f2(a.w, c.w);
+    }
+    __syncthreads();
+    pdl_wait();
+    pdl_launch_dependents();
+    const float* gq_src = gq + ((size_t)h * tokens + tok0) * 2 * DKP;
+    const float* v_src = vf + ((size_t)(h * (p.dv / kGrCols) + blockIdx.x) * tokens + tok0) * kGrCols;
+    auto load = [&](int blk) {
+        const int s = blk & 1, n = min(TOK, n_tok - blk * TOK);
+        const uint32_t dst = smem_u32(smem_f + s * STAGE), bar = smem_u32(&bars[s]);
+        const uint32_t gq_bytes = (uint32_t)n * 2 * DKP * 4, v_bytes = (uint32_t)n * kGrCols * 4;
+        mbar_expect_tx(bar, gq_bytes + v_bytes);
+        bulk_load(dst, gq_src + (size_t)blk * TOK * 2 * DKP, gq_bytes, bar);
+        bulk_load(dst + TOK * 2 * DKP * 4, v_src + (size_t)blk * TOK * kGrCols, v_bytes, bar);
+    };
+    if (tid == 0) {
+        if (n_blk > 0) load(0);
+        if (n_blk > 1) load(1);
+    }
+    const bool hi2 = lane & 16, hi1 = lane & 8;
+    const int my_col = col + (hi2 ? 2 : 0) + (hi1 ? 1 : 0);
+    bool ok = true;
+    for (int blk = 0; blk < n_blk; blk++) {
+        const int s = blk & 1, n = min(TOK, n_tok - blk * TOK);
+        ok = mbar_wait(smem_u32(&bars[s]), (uint32_t)(blk >> 1) & 1u);
+        const float* sg = smem_f + s * STAGE + k0;
+        const float* sv = smem_f + s * STAGE + TOK * 2 * DKP + col;
+        float* dst = part + s * PART + warp * TOK * kGrCols + my_col;
+        if (ok) {
+            int t = 0;
+            auto token = [&](int tt, f32x2 (&o2)[4]) {
+                const float4 v4 = *reinterpret_cast<const float4*>(sv + tt * kGrCols);
+                const f32x2 vv[4] = {pack_f2(v4.x, v4.x), pack_f2(v4.y, v4.y), pack_f2(v4.z, v4.z), pack_f2(v4.w, v4.w)};
+                f32x2 g2[R / 2], q2[R / 2];
+                const float *gt = sg + tt * 2 * DKP, *qt = gt + DKP;
+                if constexpr (R >= 4) {
+#pragma unroll
+                    for (int r = 0; r < R / 2; r += 2) {
+                        *reinterpret_cast<ulonglong2*>(&g2[r]) = *reinterpret_cast<const ulonglong2*>(gt + 2 * r);
+                        *reinterpret_cast<ulonglong2*>(&q2[r]) = *reinterpret_cast<const ulonglong2*>(qt + 2 * r);
+                    }
+                } else {
+                    g2[0] = *reinterpret_cast<const f32x2*>(gt);
+                    q2[0] = *reinterpret_cast<const f32x2*>(qt);
+                }
+#pragma unroll
+                for (int c = 0; c < 4; c++) o2[c] = 0ull;
+#pragma unroll
+                for (int r = 0; r < R / 2; r++)
+#pragma unroll
+                    for (int c = 0; c < 4; c++) {
+                        S[r][c] = fma_f2(g2[r], sub_f2(vv[c], S[r][c]), S[r][c]);
+                        o2[c] = fma_f2(q2[r], S[r][c], o2[c]);
+                    }
+            };
+            // sum over the row groups of the warp; a lane keeps one column: halves first (columns 0-1 | 2-3), then one of two
+            auto reduce = [&](int tt, const f32x2 (&o2)[4]) {
+                const float o[4] = {sum_f2(o2[0]), sum_f2(o2[1]), sum_f2(o2[2]), sum_f2(o2[3])};
+                float a0 = hi2 ? o[2] : o[0], a1 = hi2 ? o[3] : o[1];
+                a0 += __shfl_xor_sync(0xffffffffu, hi2 ? o[0] : o[2], 16);
+                a1 += __shfl_xor_sync(0xffffffffu, hi2 ? o[1] : o[3], 16);
+                dst[tt * kGrCols] = (hi1 ? a1 : a0) + __shfl_xor_sync(0xffffffffu, hi1 ? a0 : a1, 8);
+            };
+            for (; t + 4 <= n; t += 4) {
+                f32x2 o2[4][4];
+#pragma unroll
+                for (int u = 0; u < 4; u++) token(t + u, o2[u]);
+#pragma unroll
+                for (int u = 0; u < 4; u++) reduce(t + u, o2[u]);
+            }
+            for (; t < n; t++) {
+                f32x2 o2[4];
+                token(t, o2);
+                reduce(t, o2);
+            }
+        }
+        // everyone is done with the stage and has left its partial outputs (two buffers of them: a warp writes this one again
+        // behind the next barrier, which everybody reaches after the sums below)
+        ok = __syncthreads_and(ok);
+        if (!ok) break;
+        if (tid == 0 && blk + 2 < n_blk) load(blk + 2);
+        float* out = of + ((size_t)(tok0 + blk * TOK) * p.H + h) * p.dv + c0 + lane;
+        const float* src = part + s * PART + lane;
+#pragma unroll
+        for (int i = 0; i < TOK / kGrWarps; i++) {
+            const int t = warp + kGrWarps * i;
+            if (t < n) {
+                float o = 0.f;
+#pragma unroll
+                for (int w = 0; w < kGrWarps; w++) o += src[(w * TOK + t) * kGrCols];
+                out[(size_t)t * p.H * p.dv] = o;
+            }
+        }
+    }
+    if (ok && n_tok > 0) {
 #pragma unroll
         for (int r = 0; r < R; r += 2) {
-            float4 a = make_float4(0.f, 0.f, 0.f, 0.f), c = a;
-            if (!fresh && k0 + r < dk) a = st[(size_t)(k0 + r) * st_row];
-            if (!fresh && k0 + r + 1 < dk) c = st[(size_t)(k0 + r + 1) * st_row];
-            S[r / 2][0] = pack_f2(a.x, c.x);
-            S[r / 2][1] = pack_f2(a.y, c.y);
-            S[r / 2][2] = pack_f2(a.z, c.z);
-            S[r / 2][3] = pack_f2(a.w, c.w);
+            float a[4], c[4];
+#pragma unroll
+            for (int j = 0; j < 4; j++) asm("mov.b64 {%0, %1}, %2;" : "=f"(a[j]), "=f"(c[j]) : "l"(S[r / 2][j]));
+            if (k0 + r < dk) st[(size_t)(k0 + r) * st_row] = make_float4(a[0], a[1], a[2], a[3]);
+            if (k0 + r + 1 < dk) st[(size_t)(k0 + r + 1) * st_row] = make_float4(c[0], c[1], c[2], c[3]);
         }
-        pdl_wait();
-        pdl_launch_dependents();
-        const bool hi2 = lane & 16, hi1 = lane & 8;
-        const int my_col = col + (hi2 ? 2 : 0) + (hi1 ? 1 : 0);
-        cluster.sync();  // block 0 is prepared
-        for (int it = 0; it < n_blk + 2; it++) {
-            if (it < n_blk) {
-                const float* sg = ready + (it & 1) * BLK + k0;
-                const float* sq = sg + TOK * DKP;
-                const float* sv = ready + (it & 1) * BLK + 2 * TOK * DKP + col;
-                float* dst = part + (it & 1) * PART + warp * TOK * kGrCols + my_col;
-                const int n4 = (min(TOK, n_tok - it * TOK) + 3) & ~3;  // tokens behind the end have g = q = v = 0
-                for (int t = 0; t < n4; t += 4) {
-                    f32x2 o2[4][4];
-#pragma unroll
-                    for (int u = 0; u < 4; u++) {
-                        const float4 v4 = *reinterpret_cast<const float4*>(sv + (t + u) * kGrCols);
-                        const f32x2 vv[4] = {pack_f2(v4.x, v4.x), pack_f2(v4.y, v4.y), pack_f2(v4.z, v4.z), pack_f2(v4.w, v4.w)};
-                        f32x2 g2[R / 2], q2[R / 2];
-                        const float *gt = sg + (t + u) * DKP, *qt = sq + (t + u) * DKP;
-                        if constexpr (R >= 4) {
-#pragma unroll
-                            for (int r = 0; r < R / 2; r += 2) {
-                                *reinterpret_cast<ulonglong2*>(&g2[r]) = *reinterpret_cast<const ulonglong2*>(gt + 2 * r);
-                                *reinterpret_cast<ulonglong2*>(&q2[r]) = *reinterpret_cast<const ulonglong2*>(qt + 2 * r);
-                            }
-                        } else {
-                            g2[0] = *reinterpret_cast<const f32x2*>(gt);
-                            q2[0] = *reinterpret_cast<const f32x2*>(qt);
-                        }
-#pragma unroll
-                        for (int c = 0; c < 4; c++) o2[u][c] = 0ull;
-#pragma unroll
-                        for (int r = 0; r < R / 2; r++)
-#pragma unroll
-                            for (int c = 0; c < 4; c++) {
-                                S[r][c] = fma_f2(g2[r], sub_f2(vv[c], S[r][c]), S[r][c]);
-                                o2[u][c] = fma_f2(q2[r], S[r][c], o2[u][c]);
-                            }
-                    }
-                    // sum over the row groups of the warp; a lane keeps one column: halves first (columns 0-1 | 2-3), then
-                    // one of two
-#pragma unroll
-                    for (int u = 0; u < 4; u++) {
-                        const float o[4] = {sum_f2(o2[u][0]), sum_f2(o2[u][1]), sum_f2(o2[u][2]), sum_f2(o2[u][3])};
-                        float a0 = hi2 ? o[2] : o[0], a1 = hi2 ? o[3] : o[1];
-                        a0 += __shfl_xor_sync(0xffffffffu, hi2 ? o[0] : o[2], 16);
-                        a1 += __shfl_xor_sync(0xffffffffu, hi2 ? o[1] : o[3], 16);
-                        dst[(t + u) * kGrCols] = (hi1 ? a1 : a0) + __shfl_xor_sync(0xffffffffu, hi1 ? a0 : a1, 8);
-                    }
-                }
-            }
-            cluster.sync();
-        }
-        if (n_tok > 0) {
-#pragma unroll
-            for (int r = 0; r < R; r += 2) {
-                float a[4], c[4];
-#pragma unroll
-                for (int j = 0; j < 4; j++) asm("mov.b64 {%0, %1}, %2;" : "=f"(a[j]), "=f"(c[j]) : "l"(S[r / 2][j]));
-                if (k0 + r < dk) st[(size_t)(k0 + r) * st_row] = make_float4(a[0], a[1], a[2], a[3]);
-                if (k0 + r + 1 < dk) st[(size_t)(k0 + r + 1) * st_row] = make_float4(c[0], c[1], c[2], c[3]);
-            }
-        }
-    } else {
-        // ---- feed and drain
-        const int ft = tid - kGrWarps * 32, fw = ft >> 5;
-        const int n_peers = gridDim.x;
-        // the channels whose gates this thread makes: ft % DKP of tokens ft / DKP, + 128 / DKP, ... (two channels when there
-        // are more of them than threads)
-        constexpr int KPT = DKP > kGrFeed ? DKP / kGrFeed : 1, TSTEP = DKP > kGrFeed ? 1 : kGrFeed / DKP;
-        float zb[KPT], lower[KPT];
-#pragma unroll
-        for (int i = 0; i < KPT; i++) {
-            const int k = min(ft % DKP + i * kGrFeed, dk - 1);
-            zb[i] = p.zb[h * dk + k];
-            lower[i] = p.lower[h * dk + k];
-        }
-        const float wn = p.w[c0 + lane] * p.out_scale;
-        pdl_wait();
-        pdl_launch_dependents();
-        const T* q = reinterpret_cast<const T*>(p.q) + (size_t)h * dk;
-        const T* z = reinterpret_cast<const T*>(p.z) + (size_t)h * dk;
-        const T* v = reinterpret_cast<const T*>(p.v) + (size_t)h * p.dv + c0;
-        const int kc = dk / VEC, per_tok = 2 * kc + kGrCols / VEC;
-        const uint32_t raw_base = (uint32_t)__cvta_generic_to_shared(smem);
-        auto issue = [&](int blk) {  // a warp copies whole tokens
-            if (blk < n_blk) {
-                const int t0 = blk * TOK, n = min(TOK, n_tok - t0);
-                for (int t = fw; t < n; t += kGrFeed / 32) {
-                    const size_t row = (size_t)(tok0 + t0 + t) * p.ld;
-                    const uint32_t dst = raw_base + (uint32_t)((blk & 1) * raw) + (uint32_t)(t * per_tok) * 16u;
-                    for (int c = lane; c < per_tok; c += 32) {
-                        const T* src = c < kc ? q + row + c * VEC : c < 2 * kc ? z + row + (c - kc) * VEC : v + row + (c - 2 * kc) * VEC;
-                        cp_async16(dst + c * 16u, src, 16);
-                    }
-                }
-            }
-            cp_async_commit();
-        };
-        auto prepare = [&](int blk) {  // the copies of this block were issued one call ago
-            cp_async_wait<0>();
-            asm volatile("bar.sync 1, %0;" ::"n"(kGrFeed) : "memory");  // the feeding threads' copies of the block, and their reads of the one before
-            issue(blk + 1);
-            if (blk >= n_blk) return;
-            const int n = min(TOK, n_tok - blk * TOK), n4 = (n + 3) & ~3;
-            const T* rb = reinterpret_cast<const T*>(smem + (size_t)(blk & 1) * raw);
-            const int row_el = 2 * dk + kGrCols;
-            float* sg = ready + (blk & 1) * BLK;
-            float* sq = sg + TOK * DKP;
-            float* sv = sq + TOK * DKP;
-#pragma unroll
-            for (int i = 0; i < KPT; i++) {
-                const int k = ft % DKP + i * kGrFeed, kk = min(k, dk - 1);
-#pragma unroll 4
-                for (int t = ft / DKP; t < n4; t += TSTEP) {
-                    const T* row = rb + min(t, n - 1) * row_el + kk;
-                    float g, qs;
-                    gate<T>(to_float(row[0]), to_float(row[dk]), zb[i], lower[i], g, qs);
-                    const bool real = k < dk && t < n;
-                    sg[t * DKP + k] = real ? g : 0.f;
-                    sq[t * DKP + k] = real ? qs : 0.f;
-                }
-            }
-#pragma unroll 4
-            for (int t = fw; t < n4; t += kGrFeed / 32) {
-                const float x = to_float(rb[min(t, n - 1) * row_el + 2 * dk + lane]);
-                sv[t * kGrCols + lane] = t < n ? x : 0.f;
-            }
-        };
-        issue(0);
-        prepare(0);
-        cluster.sync();
-        float o[TOK / 4];  // outputs of token fw + 4 i, column `lane`, of the block summed last
-        for (int it = 0; it < n_blk + 2; it++) {
-            prepare(it + 1);
-            if (it >= 2) {
-                // norm and store block it - 2: every block of the cluster left its sums before the last barrier, and writes
-                // that buffer again behind the next one
-                const int blk = it - 2, n = min(TOK, n_tok - blk * TOK);
-                float inv = 0.f;
-                if (lane < TOK) {
-                    float* mine = ssq + (blk & 1) * TOK;
-                    float s[8];
-#pragma unroll
-                    for (int r = 0; r < 8; r++) s[r] = r < n_peers ? cluster.map_shared_rank(mine, r)[lane] : 0.f;
-                    inv = 1.0f / sqrtf((((s[0] + s[1]) + (s[2] + s[3])) + ((s[4] + s[5]) + (s[6] + s[7]))) / (float)p.norm_width + p.eps);
-                }
-                T* dst = reinterpret_cast<T*>(p.out) + (size_t)(tok0 + blk * TOK) * p.out_ld + (size_t)h * p.dv + c0 + lane;
-#pragma unroll
-                for (int i = 0; i < TOK / 4; i++) {
-                    const int t = fw + 4 * i;
-                    const float f = __shfl_sync(0xffffffffu, inv, t);
-                    if (t < n) dst[(size_t)t * p.out_ld] = from_float<T>(o[i] * f * wn);
-                }
-            }
-            if (it >= 1 && it <= n_blk) {
-                // add the warps' partial outputs of block it - 1 (rows behind its end are whatever was there: never stored)
-                const float* src = part + ((it - 1) & 1) * PART + lane;
-                float* mine = ssq + ((it - 1) & 1) * TOK;
-#pragma unroll
-                for (int i = 0; i < TOK / 4; i++) {
-                    o[i] = 0.f;
-#pragma unroll
-                    for (int w = 0; w < kGrWarps; w++) o[i] += src[(w * TOK + fw + 4 * i) * kGrCols];
-                }
-#pragma unroll
-                for (int i = 0; i < TOK / 4; i++) {
-                    const float s = warp_sum(o[i] * o[i]);
-                    if (lane == 0) mine[fw + 4 * i] = s;
-                }
-            }
-            cluster.sync();
-        }
-        cp_async_wait<0>();
     }
+}
+static const TimeoutFlag timeout_flag(tc_flag_read_clear);
+
+// one warp per (token, head)
+template <typename T>
+__global__ void __launch_bounds__(256) gated_recurrence_norm_kernel(const GrParams pp, int tokens, const float* __restrict__ of)
+{
+    const GatedRecurrence& p = pp.g;
+    pdl_launch_dependents();
+    pdl_wait();
+    const long i = (long)blockIdx.x * 8 + (threadIdx.x >> 5);
+    const int lane = threadIdx.x & 31;
+    if (i >= (long)tokens * p.H) return;
+    const int t = (int)(i / p.H), h = (int)(i % p.H);
+    const float* src = of + (size_t)i * p.dv;
+    float o[8], ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < 8; j++) {
+        o[j] = lane + 32 * j < p.dv ? src[lane + 32 * j] : 0.f;
+        ss = fmaf(o[j], o[j], ss);
+    }
+    const float inv = p.out_scale / sqrtf(warp_sum(ss) / (float)p.norm_width + p.eps);
+    T* dst = reinterpret_cast<T*>(p.out) + (size_t)t * p.out_ld + (size_t)h * p.dv;
+#pragma unroll
+    for (int j = 0; j < 8; j++)
+        if (lane + 32 * j < p.dv) dst[lane + 32 * j] = from_float<T>(o[j] * inv * p.w[lane + 32 * j]);
 }
 
 // One token per sequence.  A block owns `cols` value columns of one (sequence, head); cols / 4 threads share a row and
@@ -423,17 +429,18 @@ static int launch_cluster(Kernel kern, dim3 grid, int threads, size_t smem, cuda
     return ONELLM_OK;
 }
 
-template <typename T, int R, int TOK>
-static int launch_gr(const GrParams& p, int B, cudaStream_t st)
+template <int R, int TOK>
+static int launch_scan(const GrParams& p, int B, int tokens, const float* gq, const float* vf, float* of, cudaStream_t st)
 {
-    auto kern = gated_recurrence_kernel<T, R, TOK>;
+    auto kern = gated_recurrence_scan_kernel<R, TOK>;
     static DeviceOnce attr;
-    ONELLM_CUDA(attr.run([kern] { return cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024); }));
-    return launch_cluster(kern, dim3(p.g.dv / kGrCols, p.g.H, B), kGrThreads, gr_smem_bytes<T, R, TOK>(p.g.dk), st, p);
+    ONELLM_CUDA(attr.run([kern] { return cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)gr_smem_bytes<R, TOK>()); }));
+    ONELLM_CUDA(launch_pdl(kern, dim3(p.g.dv / kGrCols, p.g.H, B), dim3(kGrThreads), gr_smem_bytes<R, TOK>(), st, p, tokens, gq, vf, of));
+    return ONELLM_OK;
 }
 
 template <typename T>
-static int dispatch_gr(const GrParams& p, int B, cudaStream_t st)
+static int dispatch_gr(const GrParams& p, int B, int tokens, cudaStream_t st)
 {
     if (!p.tp.cu) {
         // columns of a head over several blocks only while whole heads leave SMs without work
@@ -442,32 +449,45 @@ static int dispatch_gr(const GrParams& p, int B, cudaStream_t st)
             if (p.g.dv % (32 * n) == 0) cols = p.g.dv / n;
         return launch_cluster(gated_recurrence_step_kernel<T>, dim3(p.g.dv / cols, p.g.H, B), kGsThreads, 0, st, p, cols);
     }
-    // token blocks of 32 where one thread block per SM is all there is, else of 16 (two thread blocks share an SM)
-    const int dk = p.g.dk;
-    if constexpr (sizeof(T) == 2) {
-        if (dk <= 128 && (long)B * p.g.H * (p.g.dv / kGrCols) <= num_sms())
-            return dk <= 64 ? launch_gr<T, 2, 32>(p, B, st) : launch_gr<T, 4, 32>(p, B, st);
-    }
-    if (dk <= 64) return launch_gr<T, 2, 16>(p, B, st);
-    if (dk <= 128) return launch_gr<T, 4, 16>(p, B, st);
-    return launch_gr<T, 8, 16>(p, B, st);
+    if (tokens <= 0) return ONELLM_OK;
+    const int dkp = gr_dkp(p.g.dk);
+    float* gq = static_cast<float*>(p.g.work);
+    float* vf = gq + (size_t)tokens * p.g.H * 2 * dkp;
+    float* of = vf + (size_t)tokens * p.g.H * p.g.dv;
+    ONELLM_CUDA(launch_pdl(gated_recurrence_prepare_kernel<T>, dim3(tokens), dim3(256), 0, st, p, tokens, dkp, gq, vf));
+    // long token blocks where one thread block per SM is all there is, short ones (more thread blocks per SM) otherwise
+    const bool few = (long)B * p.g.H * (p.g.dv / kGrCols) <= num_sms();
+    int rc;
+    if (dkp == 64) rc = few ? launch_scan<2, 32>(p, B, tokens, gq, vf, of, st) : launch_scan<2, 16>(p, B, tokens, gq, vf, of, st);
+    else if (dkp == 128) rc = few ? launch_scan<4, 32>(p, B, tokens, gq, vf, of, st) : launch_scan<4, 16>(p, B, tokens, gq, vf, of, st);
+    else rc = launch_scan<8, 16>(p, B, tokens, gq, vf, of, st);
+    if (rc) return rc;
+    ONELLM_CUDA(launch_pdl(gated_recurrence_norm_kernel<T>, dim3((unsigned)(((long)tokens * p.g.H + 7) / 8)), dim3(256), 0, st, p, tokens, of));
+    return ONELLM_OK;
 }
 
-int gated_recurrence(const GatedRecurrence& g, const TokenPositions& tp, int B, cudaStream_t st)
+size_t gated_recurrence_workspace(int tokens, int H, int dk, int dv) { return (size_t)tokens * H * (2 * gr_dkp(dk) + 2 * dv) * sizeof(float); }
+
+int gated_recurrence(const GatedRecurrence& g, const TokenPositions& tp, int B, int tokens, cudaStream_t st)
 {
     ONELLM_REQUIRE(g.q && g.z && g.v && g.zb && g.lower && g.w && g.state && g.out, ONELLM_ERR_ARG, "gated_recurrence: null pointer");
     ONELLM_REQUIRE(g.dk > 0 && g.dk % 16 == 0 && g.dk <= 256 && g.dv > 0 && g.dv % kGrCols == 0 && g.dv <= 8 * kGrCols, ONELLM_ERR_UNSUPPORTED,
                    "gated_recurrence: key size %d must be a multiple of 16 and value size %d of 32, both at most 256", g.dk, g.dv);
-    ONELLM_REQUIRE(g.H > 0 && g.H <= 65535 && B > 0 && B <= 65535 && g.ld % 8 == 0 && (tp.cu ? tp.hist != nullptr : tp.step && tp.off),
+    ONELLM_REQUIRE(g.H > 0 && g.H <= 65535 && B > 0 && B <= 65535 && g.ld % 8 == 0 && (tp.cu ? tp.hist && g.work && aligned16(g.work) : tp.step && tp.off),
                    ONELLM_ERR_ARG, "gated_recurrence: bad argument");
     const GrParams p = {g, tp};
-    return g.dtype == ONELLM_F32 ? dispatch_gr<float>(p, B, st) : dispatch_gr<__nv_bfloat16>(p, B, st);
+    return g.dtype == ONELLM_F32 ? dispatch_gr<float>(p, B, tokens, st) : dispatch_gr<__nv_bfloat16>(p, B, tokens, st);
 }
 
 }  // namespace onellm
 
-extern "C" int onellm_gated_recurrence_run(const onellm_gated_recurrence* g, const onellm_token_positions* tp, int B, void* stream)
+extern "C" size_t onellm_gated_recurrence_workspace(int tokens, int H, int dk, int dv)
 {
-    ONELLM_REQUIRE(g && tp, ONELLM_ERR_ARG, "gated_recurrence: null pointer");
-    return onellm::gated_recurrence(*g, *tp, B, reinterpret_cast<cudaStream_t>(stream));
+    return tokens > 0 && H > 0 && dk > 0 && dv > 0 ? onellm::gated_recurrence_workspace(tokens, H, dk, dv) : 0;
+}
+
+extern "C" int onellm_gated_recurrence_run(const onellm_gated_recurrence* g, const onellm_token_positions* tp, int tokens, void* stream)
+{
+    ONELLM_REQUIRE(g && tp && tokens >= 0, ONELLM_ERR_ARG, "gated_recurrence: bad argument");
+    return onellm::gated_recurrence(*g, *tp, tp->B, tokens, reinterpret_cast<cudaStream_t>(stream));
 }

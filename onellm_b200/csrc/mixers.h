@@ -33,7 +33,8 @@ size_t biased_attn_decode_workspace(int B, int H, int dv);
 int biased_attn_decode(const BiasedAttn& a, const TokenPositions& tp, int step_bound, void* workspace, cudaStream_t st);
 int build_query_factor(float* out, int S, double scale, double coef, double every, cudaStream_t st);
 int build_distance_penalty(float* out, const float* r1, const float* r2, int H, int S, cudaStream_t st);
-int gated_recurrence(const GatedRecurrence& g, const TokenPositions& tp, int B, cudaStream_t st);
+size_t gated_recurrence_workspace(int tokens, int H, int dk, int dv);
+int gated_recurrence(const GatedRecurrence& g, const TokenPositions& tp, int B, int tokens, cudaStream_t st);
 
 // norm.cu
 int norm_pair(int dtype, const float* x, const int* rows, int n_rows, const float* w1, const float* w2, void* out1, void* out2, float eps,

@@ -140,14 +140,15 @@ def make_mechanism_case(name, torch, m, B, ctx, plain=False) -> Case:
         state = [torch.zeros(B, RH, RK, RV, **f32) for _ in range(rot)]
         zb, lower, w = torch.full((RH * RK,), 2.0, **f32), torch.full((RH * RK,), 0.5, **f32), torch.ones(RV, **f32)
         c0 = (H + G) * D + G * DV
+        work = torch.empty(ob.gated_recurrence_workspace(T, RH, RK, RV), device="cuda", dtype=torch.uint8)
         g = [ob.GatedRecurrence(BF, RH, RK, RV, p + c0 * 2, p + (c0 + RH * RK) * 2, p + (c0 + 2 * RH * RK) * 2, n_mix, zb.data_ptr(),
-                                lower.data_ptr(), w.data_ptr(), 1e-6, RV, state[i].data_ptr(), cat.data_ptr() + H * DV * 2, n_cat, 1.0)
-             for i in range(rot)]
-        fn = lambda i: ob.gated_recurrence(g[i], tp, B)
-        keep = (mix, cat, cu, hist, off, step, state, zb, lower, w)
+                                lower.data_ptr(), w.data_ptr(), 1e-6, RV, state[i].data_ptr(), cat.data_ptr() + H * DV * 2, n_cat, 1.0,
+                                work.data_ptr()) for i in range(rot)]
+        fn = lambda i: ob.gated_recurrence(g[i], tp, T)
+        keep = (mix, cat, cu, hist, off, step, state, zb, lower, w, work)
         if prefill:  # decay and write (a product and a multiply-add), read (a multiply-add) per state element and token
-            return Case(fn, rot, 5.0 * T * RH * RK * RV, "flop", "gated_recurrence_kernel", keep=keep)
-        return Case(fn, rot, 2 * B * RH * RK * RV * 4 + B * RH * (2 * RK + 2 * RV) * 2, "B", "gated_recurrence_kernel", keep=keep)
+            return Case(fn, rot, 5.0 * T * RH * RK * RV, "flop", "gated_recurrence_scan_kernel", launches=3, keep=keep)
+        return Case(fn, rot, 2 * B * RH * RK * RV * 4 + B * RH * (2 * RK + 2 * RV) * 2, "B", "gated_recurrence_step_kernel", keep=keep)
     raise ValueError(f"unknown case {name}")
 
 

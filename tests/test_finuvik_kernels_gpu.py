@@ -286,10 +286,11 @@ def run_recurrence(ob, d, H, dk, dv, q, z, v, zb, lower, w, state, tp, B, eps=1e
     row = d.up(np.concatenate([q.reshape(T, -1), z.reshape(T, -1), v.reshape(T, -1)], 1))
     es, p = row.element_size(), row.data_ptr()
     out = d.zeros(T, H * dv + 32)
+    work = d.zeros(ob.gated_recurrence_workspace(T, H, dk, dv) // 4, f32=True) + float("nan")
     g = ob.GatedRecurrence(d.dtype, H, dk, dv, p, p + H * dk * es, p + 2 * H * dk * es, row.shape[1], d.f32(zb).data_ptr(),
                            d.f32(lower).data_ptr(), d.f32(w).data_ptr(), eps, width or dv, state.data_ptr(), out.data_ptr() + 16 * es,
-                           H * dv + 32, scale_out)
-    ob.gated_recurrence(g, tp, B)
+                           H * dv + 32, scale_out, work.data_ptr())
+    ob.gated_recurrence(g, tp, T)
     o = host(out)
     assert np.all(o[:, :16] == 0) and np.all(o[:, -16:] == 0)
     return o[:, 16:-16].reshape(T, H, dv)
@@ -365,6 +366,6 @@ def test_bad_arguments_are_errors(cuda, ob):
     assert e.value.status == -2
     with pytest.raises(ob.OnellmError):
         ob.project(ob.BF16, t.row, t.row, None, t.out, 4, 12, 16)
-    g = ob.GatedRecurrence(ob.BF16, 1, 16, 48, 16, 16, 16, 16, 16, 16, 16, 1e-5, 48, 16, 16, 48, 1.0)
+    g = ob.GatedRecurrence(ob.BF16, 1, 16, 48, 16, 16, 16, 16, 16, 16, 16, 1e-5, 48, 16, 16, 48, 1.0, 16)
     with pytest.raises(ob.OnellmError):
         ob.gated_recurrence(g, tp, 1)
