@@ -632,8 +632,9 @@ ONELLM_API int onellm_llama_set_tp_exchange(onellm_llama* m, int peer_memory);
  * NULL.  Waits for the model's stream. */
 ONELLM_API int onellm_llama_last_draws(onellm_llama* m, float* host_u, int* host_step, int* table_in_use);
 /* 1: run the context phase one position at a time through the decode kernels (cross-check path);
- * 0 (default): all prompt tokens at once through the context-phase kernels; 2: the same with the norm kernels
- * kept between the projections on one GPU too (what tensor-parallel runs always do; comparison). */
+ * 0 (default): all prompt tokens at once through the context-phase kernels; 2: a design's unfused kernels instead of its
+ * fused ones, for comparison (LLaMA: the norm kernels kept between the projections on one GPU too, what tensor-parallel
+ * runs always do; Finuvik: plain attention in prompts and decode steps). */
 ONELLM_API int onellm_llama_set_prefill_by_decode(onellm_llama* m, int enabled);
 
 /* Context phase for `batch` prompts of equal length (host ids [batch, prompt_len]); resets the
@@ -652,7 +653,8 @@ ONELLM_API int onellm_llama_prefill_ragged(onellm_llama* m, const int* host_ids,
  * host_first_ids (may be NULL) receives the next generated token per sequence. */
 ONELLM_API int onellm_llama_extend(onellm_llama* m, const int* host_ids, int n_new, int* host_first_ids);
 /* Declares cur_len positions of `batch` sequences as already present in the KV cache and host_ids
- * [batch] as the next input tokens (resume on a cache filled elsewhere; profiling without prefill). */
+ * [batch] as the next input tokens (resume on a cache filled elsewhere; profiling without prefill).  Recurrent states are
+ * taken as they are: they have no positions to go back to. */
 ONELLM_API int onellm_llama_seek(onellm_llama* m, int batch, int cur_len, const int* host_ids);
 /* One generated token per sequence.  host_in_ids (may be NULL: use the previous step's samples)
  * are the tokens to feed; host_out_ids (may be NULL: stay asynchronous) receives the samples. */

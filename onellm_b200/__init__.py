@@ -475,7 +475,7 @@ class Engine:
         _check(lib().onellm_llama_set_graphs(self._h, C.c_int(1 if enabled else 0)))
 
     def set_prefill_by_decode(self, enabled):
-        """False / 0: context-phase kernels; True / 1: position by position; 2: context-phase kernels with norm kernels."""
+        """False / 0: context-phase kernels; True / 1: position by position; 2: a design's unfused kernels (comparison)."""
         _check(lib().onellm_llama_set_prefill_by_decode(self._h, C.c_int(int(enabled))))
 
     def prefill(self, ids):

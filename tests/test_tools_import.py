@@ -5,7 +5,8 @@ import re
 
 
 def test_tools_import_without_a_gpu():
-    for name in ("onellm_b200.kernel_cases", "onellm_b200.tune_plans", "onellm_b200.convert_hf"):
+    for name in ("onellm_b200.kernel_cases", "onellm_b200.tune_plans", "onellm_b200.convert_hf", "onellm_b200.generate",
+                 "onellm_b200.trace_run"):
         importlib.import_module(name)
 
 
