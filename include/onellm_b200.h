@@ -533,7 +533,7 @@ ONELLM_API size_t onellm_gated_recurrence_workspace(int tokens, int H, int dk, i
 /* tokens: of the whole launch (context pass: cu[B]). */
 ONELLM_API int onellm_gated_recurrence_run(const onellm_gated_recurrence* g, const onellm_token_positions* tp, int tokens, void* stream);
 
-/* RMSNorm with weights stored around zero, out of a float stream into one or two buffers (out2 may be NULL):
+/* RMSNorm whose weights are offsets from one, out of a float stream into one or two buffers (out2 may be NULL):
  *     out_i[r] = x[r or rows[r]] * rsqrt(mean(x^2) + eps) * (1 + w_i)
  * `width` columns count; ld is the row stride of every buffer, the columns behind width hold zeros. */
 ONELLM_API int onellm_norm_pair(int dtype, const float* x, const int* rows, int n_rows, const float* w1, const float* w2, void* out1,

@@ -1,6 +1,7 @@
-// Small HBM-bound kernels: SwiGLU on a packed [tokens, 2, I] buffer and the embedding gather.
+// Small HBM-bound kernels: SwiGLU on a packed [tokens, 2, I] buffer, the embedding gather, and the embedding with learned
+// positions of designs that keep their residual stream in float.
 //
-// Replace silu_and_mul_kernel (src/kernels/activation_kernel.cu:10-21) and embeddingFunctor
+// The first two replace silu_and_mul_kernel (src/kernels/activation_kernel.cu:10-21) and embeddingFunctor
 // (src/kernels/input_embedding.cu:7-20) of the reference with 16-byte vectorised versions.
 #include "mixers.h"
 

@@ -1,4 +1,4 @@
-// Gated outer-product recurrence (the HGRN2 form of linear attention: the forget gate also decides what is written);
+// Gated outer-product recurrence (HGRN2: what a channel forgets of its state is the share it takes of the new value);
 // gates, recurrence and the per-head RMS norm of the output are computed in float.  With g = 1 - f a state element
 // moves as
 //     s <- s + g (v - s)

@@ -171,7 +171,7 @@ extern "C" int onellm_row_sumsq(int dtype, const void* x, int rows, int cols, fl
 }
 
 namespace onellm {
-// RMSNorm with weights stored around zero, out of a float residual stream: for row r (or rows[r]) of x
+// RMSNorm whose weights are offsets from one, out of a float residual stream: for row r (or rows[r]) of x
 //     out_i[r] = x * rsqrt(mean(x^2) + eps) * (1 + w_i)          i = 1, 2 (out2 may be NULL)
 // into one or two buffers of element type T: two parallel branches that normalise the same stream with weights of their
 // own share one pass over it.  `width` columns count, `ld` is the row stride of all buffers (the columns behind `width`
