@@ -508,12 +508,18 @@ ONELLM_API size_t onellm_biased_attn_decode_workspace(int B, int H, int dv);
 ONELLM_API int onellm_biased_attn_decode(const onellm_biased_attn* a, const onellm_token_positions* tp, int step_bound, void* workspace,
                                          void* stream);
 
-/* Gated outer-product recurrence with a float state, per sequence and head (dk a multiple of 16, dv of 32, at most 256):
+/* Gated outer-product recurrence with a float state, per sequence and head (dk a multiple of 16, at most 512; dv a multiple of
+ * 32 for every 256 columns, at most 2048).
+ * kind ONELLM_GR_TIED (HGRN2: what a channel forgets is the share it takes of the new value):
  *     f = lower + (1 - lower) * sigmoid(z + zb)     state = diag(f) state + (1 - f) v^T     o = state^T silu(q)
- *     out = o * rsqrt(sum(o^2) / norm_width + eps) * w * out_scale
- * q, z, v: token t at + t * ld, heads dk / dk / dv apart; zb, lower [H * dk]; w [dv]; state [B, H, dk, dv], taken as zero
- * for a sequence at its first position.  work: scratch of a context pass, onellm_gated_recurrence_workspace bytes for its
- * tokens, 16-byte aligned (unused by a decode step). */
+ * kind ONELLM_GR_KEYED (gated linear attention: a key of its own, the gate through a low-rank projection):
+ *     f = sigmoid(A r + zb) ^ inv_tau               state = diag(f) state + k v^T           o = state^T (q * q_scale)
+ * out = o * rsqrt(sum(o^2) / norm_width + eps) * w * out_scale, times silu(g) when g is given
+ * q, z (TIED), k (KEYED), v, r (KEYED, `rank` elements), g: token t at + t * ld, heads dk / dk / dk / dv / - / dv apart;
+ * zb, lower (TIED) [H * dk]; A (KEYED) [H * dk, rank] float; w [dv]; state [B, H, dk, dv], taken as zero for a sequence at
+ * its first position.  work: scratch of a context pass, onellm_gated_recurrence_workspace bytes for its tokens, 16-byte
+ * aligned (unused by a decode step). */
+enum onellm_gr_kind { ONELLM_GR_TIED = 0, ONELLM_GR_KEYED = 1 };
 typedef struct onellm_gated_recurrence {
     int dtype;
     int H, dk, dv;
@@ -528,27 +534,178 @@ typedef struct onellm_gated_recurrence {
     long out_ld;
     float out_scale;
     void* work;
+    int kind; /* enum onellm_gr_kind */
+    const void *k, *r;
+    int rank;
+    const float* A;
+    float inv_tau, q_scale;
+    const void* g;
 } onellm_gated_recurrence;
-ONELLM_API size_t onellm_gated_recurrence_workspace(int tokens, int H, int dk, int dv);
+ONELLM_API size_t onellm_gated_recurrence_workspace(int kind, int tokens, int H, int dk, int dv);
 /* tokens: of the whole launch (context pass: cu[B]). */
 ONELLM_API int onellm_gated_recurrence_run(const onellm_gated_recurrence* g, const onellm_token_positions* tp, int tokens, void* stream);
 
-/* RMSNorm whose weights are offsets from one, out of a float stream into one or two buffers (out2 may be NULL):
- *     out_i[r] = x[r or rows[r]] * rsqrt(mean(x^2) + eps) * (1 + w_i)
- * `width` columns count; ld is the row stride of every buffer, the columns behind width hold zeros. */
-ONELLM_API int onellm_norm_pair(int dtype, const float* x, const int* rows, int n_rows, const float* w1, const float* w2, void* out1,
-                                void* out2, float eps, int width, int ld, void* stream);
+/* RMSNorm out of a float stream into one or two buffers (out2 may be NULL):
+ *     out_i[r] = x[r or rows[r]] * rsqrt(mean(x^2) + eps) * (w_base + w_i)
+ * w_base 1: weights kept as offsets from one, 0: plain weights.  `width` columns count; ld is the row stride of every
+ * buffer, the columns behind width hold zeros.  With `add` the stream takes a sum of rows first (in place):
+ *     x[r] += add_scale * sum_{k < add_n} add[add_rows[r * add_n + k]]
+ * and out1 may be NULL (the sum alone). */
+typedef struct onellm_norm_rows {
+    int dtype;
+    float* x;
+    const int* rows;
+    int n_rows;
+    const float *w1, *w2;
+    void *out1, *out2;
+    float eps, w_base;
+    int width, ld;
+    const void* add;
+    const int* add_rows;
+    int add_n;
+    float add_scale;
+} onellm_norm_rows;
+ONELLM_API int onellm_norm_rows_run(const onellm_norm_rows* n, void* stream);
 
-/* Projection of any number of tokens, W and W2 [K,N]:  y = x.W,  y = act(x.W) * (x.W2)  (W2 given),  y = resid + x.W  (resid
- * given, float, with f32).  f32: y is float.  ldy: row stride of y and resid (0: N).  BF16: K % 16 == 0, N and ldy % 8 == 0. */
-enum onellm_gate_act { ONELLM_GATE_SILU = 0, ONELLM_GATE_RELU = 1 };
-ONELLM_API int onellm_project(int dtype, const void* x, const void* W, const void* W2, void* y, long ldy, int M, int N, int K, int act, int f32,
-                              const float* resid, void* stream);
+/* Gate functions of a projection with two weights, from g = x.W and u = x.W2:
+ *     SILU  silu(g) * u        RELU  max(g, 0) * u
+ *     CLAMPED  with g' = min(g, limit), u' = min(max(u, -limit), limit):  g' * sigmoid(1.702 g') * (u' + 1) */
+enum onellm_gate_act { ONELLM_GATE_SILU = 0, ONELLM_GATE_RELU = 1, ONELLM_GATE_CLAMPED = 2 };
+
+/* Rows of a projection in groups that use weights of their own (experts, heads).  Group g uses the weight w_stride * g
+ * elements behind W (and W2), reads its columns x_stride * g elements into a row of x and writes y_stride * g elements into
+ * a row of y.
+ *   off == NULL  every group takes all M rows of x
+ *   off          device [groups + 1]: group g owns the rows off[g] .. off[g + 1] - 1 of y, at most M of them;
+ *                x_rows (or NULL: the same row): which row of x stands behind a row of y
+ *   used, n_used (or NULL): the groups that have rows at all, so that a launch needs no blocks for the others; `n` is the
+ *                number of groups, or the most that can be used
+ *   row_scale (or NULL): factor of a row of y on x.W and x.W2, in front of the gate function
+ *   tile_group, tile_row, n_tiles, max_tiles: M > 64 with off: 128-row tiles of the rows, tile_row the first row of a tile */
+typedef struct onellm_row_groups {
+    int n;
+    const int *used, *n_used, *off, *x_rows;
+    const float* row_scale;
+    long w_stride, x_stride, y_stride;
+    const int *tile_group, *tile_row, *n_tiles;
+    int max_tiles;
+    int weights; /* weights behind W, for the bounds of a tiled launch */
+    long rows;   /* rows of x, likewise */
+} onellm_row_groups;
+
+/* Projection of any number of tokens, W and W2 [K, N] with rows ldw (0: N) elements apart, x rows ldx (0: K) apart:
+ *     y = x.W        y = gate(x.W, x.W2)  (W2 given)        y = resid + scale * x.W  (resid given, float, with f32 or F32)
+ * f32: y is float.  ldy: row stride of y and resid (0: N).  BF16: K % 16 == 0, N and all strides % 8 == 0; ldw and ldx need
+ * groups. */
+typedef struct onellm_projection {
+    int dtype;
+    const void *x, *W, *W2;
+    void* y;
+    long ldy;
+    int M, N, K;
+    int act;
+    int f32;
+    const float* resid;
+    float scale, limit;
+    long ldx;
+    int ldw;
+    const onellm_row_groups* groups;
+} onellm_projection;
+ONELLM_API int onellm_project(const onellm_projection* p, void* stream);
+
+/* Routing of a mixture of experts.  logits [T, ld] float; a token's score of an expert is the sigmoid of its logit; the `top`
+ * best (the lower number on a tie) are chosen and their scores are the weights.  Rows in expert order ("slots"):
+ *     slot [T * top]: the slot of a token's k-th choice;  slot_token, slot_weight [T * top];  off [experts + 1]
+ *     used [min(experts, T * top)], n_used: experts with rows;  tile_group, tile_row, n_tiles: their 128-row tiles, at most
+ *     onellm_route_max_tiles of them;  count [experts]: scratch, zero before the first call
+ * With x and xs (T > 64) the rows of x (ld_x elements) are copied into slot order. */
+typedef struct onellm_route {
+    int T, experts, top;
+    const float* logits;
+    long ld;
+    int *slot, *slot_token;
+    float* slot_weight;
+    int *off, *used, *n_used, *tile_group, *tile_row, *n_tiles, *count, *choice;
+    float* choice_weight; /* choice, choice_weight [T * top]: scratch */
+    int dtype;
+    const void* x;
+    void* xs;
+    int ld_x;
+} onellm_route;
+ONELLM_API int onellm_route_max_tiles(int T, int experts, int top);
+ONELLM_API int onellm_route_run(const onellm_route* r, void* stream);
 
 /* out[t] = table[ids[t]] + pos_table[position of t] in float, rows of ld elements.  A bad id raises bad[0], a position
  * outside [0, max_pos) bad[1]; the row is zero then. */
 ONELLM_API int onellm_embedding_pos(int dtype, const int* ids, float* out, const void* table, const void* pos_table, int n_tokens, int ld,
                                     int vocab, int max_pos, const onellm_token_positions* tp, int* bad, void* stream);
+
+/* out[t] = norm(table[ids[t]]) in float: RMSNorm over `width` of ld columns with plain weights.  A bad id raises bad[0]; the
+ * row is zero then. */
+ONELLM_API int onellm_embedding_norm(int dtype, const int* ids, float* out, const void* table, const float* w, float eps, int n_tokens,
+                                     int width, int ld, int vocab, int* bad, void* stream);
+/* out[r, c] = cap * tanh(in[r * ld + c] / cap) for c < cols */
+ONELLM_API int onellm_softcap(const float* in, long ld, float* out, int rows, int cols, float cap, void* stream);
+
+/* Attention over latents with a sliding window: a token's keys and values for all heads are linear in one latent of `rank`
+ * elements, and only latents are cached, in a ring of R >= window rows per sequence (position p in row p % R).  A query at
+ * position p sees the positions p - window + 1 .. p.
+ *   onellm_latent_store: RMSNorm of two groups of columns of the projected rows (token t at src + t * ld): q_src (q_width
+ *       columns) -> q_out rows of q_ld, kv_src (rank columns) -> the latents.  A decode step writes them into the ring, a
+ *       context pass into rows `fresh`: with `joined` behind the positions a sequence has in the ring (its last
+ *       min(hist, window - 1), copied there), else in packed token order.  onellm_latent_keep then moves the last of them
+ *       into the ring, after the attention.
+ *   onellm_latent_attn: q [T, H, rank_p]: queries already turned into latent space; scores (q . c) * scale; the output
+ *       [T, H, rank_p] is the weighted latent of a head, times sigmoid(gate[t * gate_ld + h]) and out_scale.  Ring and (context
+ *       pass) fresh latents in packed order.  `plain`: one warp per token and head, any type; else BF16 tensor-core warps
+ *       (T <= 64).
+ * rank_p: rank padded to a multiple of 16, the padding zero. */
+typedef struct onellm_latent_attn {
+    int dtype;
+    int H, rank, window, R;
+    void* ring;   /* [B, R, rank_p] */
+    void* fresh;  /* [.., rank_p] */
+    int joined;
+    const void *q_src, *kv_src;
+    long ld;
+    const float *q_w, *kv_w;
+    int q_width, q_ld;
+    void* q_out;
+    float eps;
+    const void* q;
+    float scale;
+    const void* gate;
+    long gate_ld;
+    void* out;
+    float out_scale;
+} onellm_latent_attn;
+/* max_hist: most positions a sequence has before this pass; max_new: most new tokens of one */
+ONELLM_API int onellm_latent_store(const onellm_latent_attn* a, const onellm_token_positions* tp, int tokens, int max_hist, void* stream);
+ONELLM_API int onellm_latent_keep(const onellm_latent_attn* a, const onellm_token_positions* tp, int max_new, void* stream);
+ONELLM_API size_t onellm_latent_attn_workspace(int tokens, int H, int rank);
+/* span_bound: an upper bound of the keys a query sees (at most window) */
+ONELLM_API int onellm_latent_attn_run(const onellm_latent_attn* a, const onellm_token_positions* tp, int tokens, int span_bound, int plain,
+                                      void* workspace, void* stream);
+
+/* Causal attention of a context pass over keys and values that lie packed beside each other (BF16, tcgen05): row n of kv
+ * holds the keys of all H heads (dk columns each) and then their values (dv columns each); the rows of a sequence are its
+ * last min(hist, window - 1) earlier positions and then its new tokens, sequence after sequence.  Scores (q . k) * scale;
+ * a query sees itself and the window - 1 positions before it.  Output times sigmoid(gate) and out_scale.  dk, dv: multiples
+ * of 16, at most 256. */
+typedef struct onellm_window_attn {
+    int H, dk, dv, window;
+    const void* q;
+    long q_ld;
+    const void* kv;
+    long kv_ld, kv_rows;
+    float scale;
+    const void* gate;
+    long gate_ld;
+    void* out;
+    long out_ld;
+    float out_scale;
+} onellm_window_attn;
+ONELLM_API int onellm_window_attn_run(const onellm_window_attn* a, const onellm_token_positions* tp, int max_new, void* stream);
 
 /* ---------------------------------------------------------------------------------------
  * LLaMA model: weights, KV cache and the generation loop (host side in C++).

@@ -54,7 +54,55 @@ class GatedRecurrence(C.Structure):
     _fields_ = [("dtype", C.c_int), ("H", C.c_int), ("dk", C.c_int), ("dv", C.c_int),
                 ("q", C.c_void_p), ("z", C.c_void_p), ("v", C.c_void_p), ("ld", C.c_long), ("zb", C.c_void_p), ("lower", C.c_void_p),
                 ("w", C.c_void_p), ("eps", C.c_float), ("norm_width", C.c_int), ("state", C.c_void_p),
-                ("out", C.c_void_p), ("out_ld", C.c_long), ("out_scale", C.c_float), ("work", C.c_void_p)]
+                ("out", C.c_void_p), ("out_ld", C.c_long), ("out_scale", C.c_float), ("work", C.c_void_p),
+                ("kind", C.c_int), ("k", C.c_void_p), ("r", C.c_void_p), ("rank", C.c_int), ("A", C.c_void_p),
+                ("inv_tau", C.c_float), ("q_scale", C.c_float), ("g", C.c_void_p)]
+
+
+class NormRows(C.Structure):
+    """onellm_norm_rows (device addresses)."""
+    _fields_ = [("dtype", C.c_int), ("x", C.c_void_p), ("rows", C.c_void_p), ("n_rows", C.c_int), ("w1", C.c_void_p), ("w2", C.c_void_p),
+                ("out1", C.c_void_p), ("out2", C.c_void_p), ("eps", C.c_float), ("w_base", C.c_float), ("width", C.c_int), ("ld", C.c_int),
+                ("add", C.c_void_p), ("add_rows", C.c_void_p), ("add_n", C.c_int), ("add_scale", C.c_float)]
+
+
+class RowGroups(C.Structure):
+    """onellm_row_groups (device addresses)."""
+    _fields_ = [("n", C.c_int), ("used", C.c_void_p), ("n_used", C.c_void_p), ("off", C.c_void_p), ("x_rows", C.c_void_p),
+                ("row_scale", C.c_void_p), ("w_stride", C.c_long), ("x_stride", C.c_long), ("y_stride", C.c_long),
+                ("tile_group", C.c_void_p), ("tile_row", C.c_void_p), ("n_tiles", C.c_void_p), ("max_tiles", C.c_int),
+                ("weights", C.c_int), ("rows", C.c_long)]
+
+
+class Projection(C.Structure):
+    """onellm_projection (device addresses)."""
+    _fields_ = [("dtype", C.c_int), ("x", C.c_void_p), ("W", C.c_void_p), ("W2", C.c_void_p), ("y", C.c_void_p), ("ldy", C.c_long),
+                ("M", C.c_int), ("N", C.c_int), ("K", C.c_int), ("act", C.c_int), ("f32", C.c_int), ("resid", C.c_void_p),
+                ("scale", C.c_float), ("limit", C.c_float), ("ldx", C.c_long), ("ldw", C.c_int), ("groups", C.POINTER(RowGroups))]
+
+
+class Route(C.Structure):
+    """onellm_route (device addresses)."""
+    _fields_ = [("T", C.c_int), ("experts", C.c_int), ("top", C.c_int), ("logits", C.c_void_p), ("ld", C.c_long)] + [
+        (n, C.c_void_p) for n in ("slot", "slot_token", "slot_weight", "off", "used", "n_used", "tile_group", "tile_row", "n_tiles", "count",
+                                  "choice", "choice_weight")] + [
+        ("dtype", C.c_int), ("x", C.c_void_p), ("xs", C.c_void_p), ("ld_x", C.c_int)]
+
+
+class LatentAttn(C.Structure):
+    """onellm_latent_attn (device addresses)."""
+    _fields_ = [("dtype", C.c_int), ("H", C.c_int), ("rank", C.c_int), ("window", C.c_int), ("R", C.c_int), ("ring", C.c_void_p),
+                ("fresh", C.c_void_p), ("joined", C.c_int), ("q_src", C.c_void_p), ("kv_src", C.c_void_p), ("ld", C.c_long),
+                ("q_w", C.c_void_p), ("kv_w", C.c_void_p), ("q_width", C.c_int), ("q_ld", C.c_int), ("q_out", C.c_void_p),
+                ("eps", C.c_float), ("q", C.c_void_p), ("scale", C.c_float), ("gate", C.c_void_p), ("gate_ld", C.c_long),
+                ("out", C.c_void_p), ("out_scale", C.c_float)]
+
+
+class WindowAttn(C.Structure):
+    """onellm_window_attn (device addresses)."""
+    _fields_ = [("H", C.c_int), ("dk", C.c_int), ("dv", C.c_int), ("window", C.c_int), ("q", C.c_void_p), ("q_ld", C.c_long),
+                ("kv", C.c_void_p), ("kv_ld", C.c_long), ("kv_rows", C.c_long), ("scale", C.c_float), ("gate", C.c_void_p),
+                ("gate_ld", C.c_long), ("out", C.c_void_p), ("out_ld", C.c_long), ("out_scale", C.c_float)]
 
 
 def lib() -> C.CDLL:
@@ -68,7 +116,8 @@ def lib() -> C.CDLL:
         for name, restype in (("onellm_last_error", C.c_char_p), ("onellm_decode_attn_workspace_bytes", C.c_size_t),
                               ("onellm_decode_attn_static_scratch_bytes", C.c_size_t), ("onellm_llama_device_bytes", C.c_size_t),
                               ("onellm_llama_stream", C.c_void_p), ("onellm_llama_destroy", None), ("onellm_model_design", C.c_char_p),
-                              ("onellm_biased_attn_decode_workspace", C.c_size_t), ("onellm_gated_recurrence_workspace", C.c_size_t)):
+                              ("onellm_biased_attn_decode_workspace", C.c_size_t), ("onellm_gated_recurrence_workspace", C.c_size_t),
+                              ("onellm_latent_attn_workspace", C.c_size_t)):
             if hasattr(l, name):  # a library built for one design has its entry points only
                 getattr(l, name).restype = restype
         _lib = l
@@ -310,7 +359,8 @@ def topk_sample(topk_id, topk_val, B, K, temperature, rng_step, vocab_size, end_
                                     _p(u_out), _stream(stream)))
 
 
-GATE_SILU, GATE_RELU = 0, 1
+GATE_SILU, GATE_RELU, GATE_CLAMPED = 0, 1, 2
+GR_TIED, GR_KEYED = 0, 1
 
 
 def query_factor(out, S, scale, coef, every, stream=None):
@@ -338,22 +388,64 @@ def biased_attn_decode(a, tp, step_bound, workspace, stream=None):
     _check(lib().onellm_biased_attn_decode(C.byref(a), C.byref(tp), C.c_int(step_bound), _p(workspace), _stream(stream)))
 
 
-def gated_recurrence_workspace(tokens, H, dk, dv):
-    return int(lib().onellm_gated_recurrence_workspace(C.c_int(tokens), C.c_int(H), C.c_int(dk), C.c_int(dv)))
+def gated_recurrence_workspace(tokens, H, dk, dv, kind=GR_TIED):
+    return int(lib().onellm_gated_recurrence_workspace(C.c_int(kind), C.c_int(tokens), C.c_int(H), C.c_int(dk), C.c_int(dv)))
 
 
 def gated_recurrence(g, tp, tokens, stream=None):
     _check(lib().onellm_gated_recurrence_run(C.byref(g), C.byref(tp), C.c_int(tokens), _stream(stream)))
 
 
-def norm_pair(dtype, x, rows, n_rows, w1, w2, out1, out2, eps, width, ld, stream=None):
-    _check(lib().onellm_norm_pair(C.c_int(dtype), _p(x), _p(rows), C.c_int(n_rows), _p(w1), _p(w2), _p(out1), _p(out2), C.c_float(eps),
-                                  C.c_int(width), C.c_int(ld), _stream(stream)))
+def norm_rows(dtype, x, rows, n_rows, w1, w2, out1, out2, eps, width, ld, w_base=0.0, add=None, add_rows=None, add_n=0, add_scale=1.0,
+              stream=None):
+    n = NormRows(dtype, _p(x), _p(rows), n_rows, _p(w1), _p(w2), _p(out1), _p(out2), eps, w_base, width, ld, _p(add), _p(add_rows), add_n,
+                 add_scale)
+    _check(lib().onellm_norm_rows_run(C.byref(n), _stream(stream)))
 
 
-def project(dtype, x, W, W2, y, M, N, K, ldy=0, act=GATE_SILU, f32=False, resid=None, stream=None):
-    _check(lib().onellm_project(C.c_int(dtype), _p(x), _p(W), _p(W2), _p(y), C.c_long(ldy), C.c_int(M), C.c_int(N), C.c_int(K),
-                                C.c_int(act), C.c_int(1 if f32 else 0), _p(resid), _stream(stream)))
+def project(dtype, x, W, W2, y, M, N, K, ldy=0, act=GATE_SILU, f32=False, resid=None, scale=1.0, limit=0.0, ldx=0, ldw=0, groups=None,
+            stream=None):
+    p = Projection(dtype, _p(x), _p(W), _p(W2), _p(y), ldy, M, N, K, act, 1 if f32 else 0, _p(resid), scale, limit, ldx, ldw,
+                   C.pointer(groups) if groups is not None else None)
+    _check(lib().onellm_project(C.byref(p), _stream(stream)))
+
+
+def route_max_tiles(T, experts, top):
+    return int(lib().onellm_route_max_tiles(C.c_int(T), C.c_int(experts), C.c_int(top)))
+
+
+def route(r, stream=None):
+    _check(lib().onellm_route_run(C.byref(r), _stream(stream)))
+
+
+def latent_store(a, tp, tokens, max_hist=0, stream=None):
+    _check(lib().onellm_latent_store(C.byref(a), C.byref(tp), C.c_int(tokens), C.c_int(max_hist), _stream(stream)))
+
+
+def latent_keep(a, tp, max_new, stream=None):
+    _check(lib().onellm_latent_keep(C.byref(a), C.byref(tp), C.c_int(max_new), _stream(stream)))
+
+
+def latent_attn_workspace(tokens, H, rank):
+    return int(lib().onellm_latent_attn_workspace(C.c_int(tokens), C.c_int(H), C.c_int(rank)))
+
+
+def latent_attn(a, tp, tokens, span_bound, workspace, plain=False, stream=None):
+    _check(lib().onellm_latent_attn_run(C.byref(a), C.byref(tp), C.c_int(tokens), C.c_int(span_bound), C.c_int(1 if plain else 0),
+                                        _p(workspace), _stream(stream)))
+
+
+def window_attn(a, tp, max_new, stream=None):
+    _check(lib().onellm_window_attn_run(C.byref(a), C.byref(tp), C.c_int(max_new), _stream(stream)))
+
+
+def embedding_norm(dtype, ids, out, table, w, eps, n_tokens, width, ld, vocab, bad, stream=None):
+    _check(lib().onellm_embedding_norm(C.c_int(dtype), _p(ids), _p(out), _p(table), _p(w), C.c_float(eps), C.c_int(n_tokens), C.c_int(width),
+                                       C.c_int(ld), C.c_int(vocab), _p(bad), _stream(stream)))
+
+
+def softcap(x, ld, out, rows, cols, cap, stream=None):
+    _check(lib().onellm_softcap(_p(x), C.c_long(ld), _p(out), C.c_int(rows), C.c_int(cols), C.c_float(cap), _stream(stream)))
 
 
 def embedding_pos(dtype, ids, out, table, pos_table, n_tokens, ld, vocab, max_pos, tp, bad, stream=None):

@@ -24,9 +24,10 @@ NVCC_FLAGS = [
 
 # What a design opened with onellm_model_open is linked from: the engine, the projections, sampling, and its own files.
 ENGINE_SOURCES = ["elementwise.cu", "engine.cu", "errors.cpp", "gemm_tc.cu", "model_files.cpp", "norm.cu", "sampling.cu",
-                  "skinny_gemm.cu", "skinny_gemm_staged.cu", "skinny_gemm_tc.cu"]
+                  "skinny_gemm.cu", "skinny_gemm_staged.cu", "skinny_gemm_tc.cu", "weight_placer.cu"]
 DESIGN_SOURCES = {
     "Finuvik": ["biased_attn.cu", "biased_attn_tc.cu", "finuvik.cu", "gated_recurrence.cu"],
+    "Fuposun": ["biased_attn_tc.cu", "fuposun.cu", "gated_recurrence.cu", "latent_attn.cu", "route.cu"],
 }
 
 

@@ -1,5 +1,6 @@
-// Context pass of BiasedAttn (mixers.h) on the 5th-generation tensor cores: bfloat16, key and value sizes of their own,
-// a score factor per query position and a penalty per head and distance.
+// Context pass of BiasedAttn and WindowAttn (mixers.h) on the 5th-generation tensor cores: bfloat16, key and value sizes of
+// their own; the scores of the one take a factor per query position and a penalty per head and distance, those of the other
+// a constant scale and a sliding window.
 //
 // The schedule is the one of context_attn_tc_kernel (context_attn_tc.cu): a block owns 128 query rows of one
 // (sequence, head) and walks the cache in 64-row tiles; S = Q.K^T and O += P.V by tcgen05.mma with S, P and O in tensor
@@ -8,7 +9,10 @@
 //     a multiple of 64 is zero-filled by TMA and by the threads that write Q);
 //   - the scores of a row are turned into log2 units by the factor of its position and lose the penalty of their
 //     distance before the maximum is taken.  A tile of scores spans 191 distances: the threads read the table of the
-//     head directly, consecutive rows at consecutive addresses.
+//     head directly, consecutive rows at consecutive addresses;
+//   - WINDOWED: keys and values of all heads lie beside each other in one buffer that a sequence's rows are packed into, so
+//     a head is a range of columns; the tiles of a block start at the first key its first query sees, masks apply on both
+//     sides, a row may see nothing in its block's first tiles, and the output takes the gate of its token and head.
 // Every mbarrier wait is bounded; on expiry the block raises the time-out flag, stops, frees its tensor memory and
 // returns.
 #include <math.h>
@@ -30,6 +34,10 @@ struct BaParams {
     const int *cu, *hist;
     int kch, vch;         // 64-column chunks of a key / value
     uint32_t tmem_cols;   // 256 or 512
+    int window;           // WINDOWED from here on
+    float scale_log2;
+    const void* gate;
+    long gate_ld;
 };
 
 __device__ __forceinline__ void ba_umma_ta(uint32_t tmem_d, uint32_t tmem_a, uint64_t bdesc, uint32_t idesc, uint32_t accumulate)
@@ -40,6 +48,7 @@ __device__ __forceinline__ void ba_umma_ta(uint32_t tmem_d, uint32_t tmem_a, uin
         : "memory");
 }
 
+template <bool WINDOWED>
 __global__ void __launch_bounds__(kBaThreads, 2)
 biased_attn_tc_kernel(const BaParams p, const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v)
 {
@@ -87,11 +96,20 @@ biased_attn_tc_kernel(const BaParams p, const __grid_constant__ CUtensorMap map_
     pdl_wait();
     const int tok0 = p.cu[b], q_len = p.cu[b + 1] - tok0, hist = p.hist[b];
     const int q0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * kBaQ;  // the blocks with the most cache tiles first
-    const bool active = q0 < q_len && hist + q_len <= p.a.S;
+    const bool active = q0 < q_len && (WINDOWED || hist + q_len <= p.a.S);
     const int q_rows = active ? min(kBaQ, q_len - q0) : 0;
     const int kv_end = hist + q0 + q_rows;
-    const int n_tiles = active ? (kv_end + kBaKV - 1) / kBaKV : 0;
-    const int cache_row0 = (b * p.a.G + hk) * p.a.S;
+    const int key0 = WINDOWED ? max(0, hist + q0 - p.window + 1) : 0;  // first key of the first tile
+    const int n_tiles = active ? (kv_end - key0 + kBaKV - 1) / kBaKV : 0;
+    // row of key0 and columns of the head
+    int cache_row0 = (b * p.a.G + hk) * p.a.S, k_col = 0, v_col = 0;
+    if (WINDOWED) {
+        int base = tok0;
+        for (int i = 0; i < b; i++) base += min(p.hist[i], p.window - 1);
+        cache_row0 = base + key0 - (hist - min(hist, p.window - 1));
+        k_col = h * p.a.dk;
+        v_col = p.a.H * p.a.dk + h * p.a.dv;
+    }
 
     if (warp == 4 && active) {
         // ---- control: the whole warp runs this code, one elected lane issues (warp-uniform control flow keeps the
@@ -99,16 +117,16 @@ biased_attn_tc_kernel(const BaParams p, const __grid_constant__ CUtensorMap map_
         uint32_t leader;
         asm volatile("{\n .reg .pred p;\n elect.sync _|p, 0xffffffff;\n selp.u32 %0, 1, 0, p;\n}" : "=r"(leader));
         bool ok = true;
-        auto load = [&](const CUtensorMap* map, unsigned char* base, int tile_bytes, int chunks, uint32_t full0, int j) {
+        auto load = [&](const CUtensorMap* map, unsigned char* base, int tile_bytes, int chunks, uint32_t full0, int j, int col) {
             const int s = j & 1;
             if (leader) {
                 mbar_expect_tx(full0 + 8 * s, tile_bytes);
                 for (int c = 0; c < chunks; c++)
-                    tma_load_2d(smem_u32(base + s * tile_bytes + c * kBaKVChunk), map, 64 * c, cache_row0 + j * kBaKV, full0 + 8 * s);
+                    tma_load_2d(smem_u32(base + s * tile_bytes + c * kBaKVChunk), map, col + 64 * c, cache_row0 + j * kBaKV, full0 + 8 * s);
             }
         };
-        auto load_k = [&](int j) { load(&map_k, sK, k_tile, kch, k_full0, j); };
-        auto load_v = [&](int j) { load(&map_v, sV, v_tile, vch, v_full0, j); };
+        auto load_k = [&](int j) { load(&map_k, sK, k_tile, kch, k_full0, j, k_col); };
+        auto load_v = [&](int j) { load(&map_v, sV, v_tile, vch, v_full0, j, v_col); };
         auto wait_all = [&](uint32_t bar, uint32_t parity) { return __all_sync(0xffffffffu, mbar_wait(bar, parity)); };
         const uint32_t types = (1u << 4) | umma_operand_bits<bf16>() | ((uint32_t)(kBaQ >> 4) << 24);
         const uint32_t idesc_s = types | ((uint32_t)(kBaKV >> 3) << 17);
@@ -169,8 +187,8 @@ biased_attn_tc_kernel(const BaParams p, const __grid_constant__ CUtensorMap map_
         const uint32_t t_lane = tmem_base + ((uint32_t)(warp * 32) << 16);
         const uint32_t t_o = t_lane + kBaO;
         const uint32_t row_off = (r >> 3) * 1024 + (r & 7) * 128;
-        const float factor = row_ok ? p.a.q_factor[pos] : 0.f;
-        const float* pen = p.a.penalty + (size_t)h * p.a.S;
+        const float factor = WINDOWED ? p.scale_log2 : row_ok ? p.a.q_factor[pos] : 0.f;
+        const float* pen = WINDOWED ? nullptr : p.a.penalty + (size_t)h * p.a.S;
         const int pos_c = row_ok ? pos : hist + q0;  // rows behind the end of the sequence read the penalties of its first row
         float m_ref = -INFINITY, l_run = 0.f;
         bool ok = true;
@@ -188,15 +206,24 @@ biased_attn_tc_kernel(const BaParams p, const __grid_constant__ CUtensorMap map_
             ok = __all_sync(0xffffffffu, ok);
             if (!ok) break;
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-            const int kv0 = j * kBaKV;
-            const bool need_mask = kv0 + kBaKV - 1 > hist + q0;
+            const int kv0 = key0 + j * kBaKV;
+            const bool need_mask = kv0 + kBaKV - 1 > hist + q0 || (WINDOWED && kv0 <= hist + q0 + q_rows - 1 - p.window);
             uint32_t sv[64];
             tmem_ld32(t_lane + (uint32_t)((j & 1) * kBaKV), *reinterpret_cast<uint32_t(*)[32]>(&sv[0]));
             tmem_ld32(t_lane + (uint32_t)((j & 1) * kBaKV + 32), *reinterpret_cast<uint32_t(*)[32]>(&sv[32]));
             asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
             float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
             const float* pd = pen + (pos_c - kv0);  // penalty of the tile's first key; key i: pd[-i]
-            if (need_mask) {
+            if constexpr (WINDOWED) {
+                if (need_mask) {
+                    const int last = pos_c - kv0, before = last - p.window;  // visible: before < i <= last
+#pragma unroll
+                    for (int i = 0; i < 64; i++)
+                        if (i > last || i <= before) sv[i] = __float_as_uint(-INFINITY);
+                }
+#pragma unroll
+                for (int i = 0; i < 64; i++) mx4[i & 3] = fmaxf(mx4[i & 3], __uint_as_float(sv[i]));
+            } else if (need_mask) {
 #pragma unroll
                 for (int i = 0; i < 64; i++) {
                     float s = -INFINITY;
@@ -212,8 +239,9 @@ biased_attn_tc_kernel(const BaParams p, const __grid_constant__ CUtensorMap map_
                     mx4[i & 3] = fmaxf(mx4[i & 3], s);
                 }
             }
-            const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
-            const bool grow = mx > m_ref + 8.f;  // always on the first tile: every row sees cache row 0
+            float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
+            if (WINDOWED) mx *= factor;  // a positive scale commutes with the maximum
+            const bool grow = mx > m_ref + 8.f;  // always on the first tile with a key the row sees
             float alpha = 1.f;
             if (grow) {
                 alpha = fast_exp2(m_ref - mx);
@@ -221,9 +249,10 @@ biased_attn_tc_kernel(const BaParams p, const __grid_constant__ CUtensorMap map_
                 l_run *= alpha;
             }
             float sum4[4] = {0.f, 0.f, 0.f, 0.f};
+            const float ref = WINDOWED && m_ref == -INFINITY ? 0.f : m_ref;  // nothing seen so far: all weights zero
 #pragma unroll
             for (int i = 0; i < 64; i++) {
-                const float pv = fast_exp2(__uint_as_float(sv[i]) - m_ref);
+                const float pv = fast_exp2(WINDOWED ? fmaf(__uint_as_float(sv[i]), factor, -ref) : __uint_as_float(sv[i]) - ref);
                 sum4[i & 3] += pv;
                 sv[i] = __float_as_uint(pv);
             }
@@ -268,7 +297,9 @@ biased_attn_tc_kernel(const BaParams p, const __grid_constant__ CUtensorMap map_
         ok = __all_sync(0xffffffffu, ok);
         if (ok) {
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-            const float inv = l_run > 0.f ? p.a.out_scale / l_run : 0.f;
+            float inv = l_run > 0.f ? p.a.out_scale / l_run : 0.f;
+            if (WINDOWED && p.gate && row_ok)
+                inv *= 1.f / (1.f + expf(-__bfloat162float(static_cast<const bf16*>(p.gate)[(size_t)(tok0 + q0 + r) * p.gate_ld + h])));
             bf16* dst = reinterpret_cast<bf16*>(p.a.out) + (size_t)(tok0 + q0 + r) * p.a.out_ld + (size_t)h * p.a.dv;
 #pragma unroll 1
             for (int c0 = 0; c0 < vch * 64; c0 += 32) {
@@ -296,9 +327,19 @@ biased_attn_tc_kernel(const BaParams p, const __grid_constant__ CUtensorMap map_
 
 static const TimeoutFlag timeout_flag(tc_flag_read_clear);
 
+template <bool WINDOWED>
+static int ba_launch(const BaParams& p, int B, int max_new, const CUtensorMap& map_k, const CUtensorMap& map_v, cudaStream_t st)
+{
+    const int smem = p.kch * kBaQChunk + 2 * (p.kch + p.vch) * kBaKVChunk + 256;
+    static DeviceOnce attr;
+    ONELLM_CUDA(attr.run([] { return cudaFuncSetAttribute(biased_attn_tc_kernel<WINDOWED>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); }));
+    ONELLM_CUDA(launch_pdl(biased_attn_tc_kernel<WINDOWED>, dim3((max_new + kBaQ - 1) / kBaQ, p.a.H, B), dim3(kBaThreads), smem, st, p, map_k, map_v));
+    return ONELLM_OK;
+}
+
 int biased_attn_tc_launch(const BiasedAttn& a, const TokenPositions& tp, int max_new, cudaStream_t st)
 {
-    BaParams p = {a, tp.cu, tp.hist, (a.dk + 63) / 64, (a.dv + 63) / 64, 256u};
+    BaParams p = {a, tp.cu, tp.hist, (a.dk + 63) / 64, (a.dv + 63) / 64, 256u, 0, 0.f, nullptr, 0};
     if (p.vch > 2) p.tmem_cols = 512u;
     const uint64_t rows = (uint64_t)tp.B * a.G * a.S;
     ONELLM_REQUIRE(rows < (1ull << 31), ONELLM_ERR_UNSUPPORTED, "biased_attn: cache of %llu rows", (unsigned long long)rows);
@@ -306,11 +347,38 @@ int biased_attn_tc_launch(const BiasedAttn& a, const TokenPositions& tp, int max
     int rc = make_map(&map_k, a.k_cache, (uint64_t)a.dk, rows, kBaKV);
     if (!rc) rc = make_map(&map_v, a.v_cache, (uint64_t)a.dv, rows, kBaKV);
     if (rc) return rc;
-    const int smem = p.kch * kBaQChunk + 2 * (p.kch + p.vch) * kBaKVChunk + 256;
-    static DeviceOnce attr;
-    ONELLM_CUDA(attr.run([] { return cudaFuncSetAttribute(biased_attn_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); }));
-    ONELLM_CUDA(launch_pdl(biased_attn_tc_kernel, dim3((max_new + kBaQ - 1) / kBaQ, a.H, tp.B), dim3(kBaThreads), smem, st, p, map_k, map_v));
-    return ONELLM_OK;
+    return ba_launch<false>(p, tp.B, max_new, map_k, map_v, st);
+}
+
+int window_attn(const WindowAttn& a, const TokenPositions& tp, int max_new, cudaStream_t st)
+{
+    ONELLM_REQUIRE(a.q && a.kv && a.out && tp.cu && tp.hist && tp.B > 0, ONELLM_ERR_ARG, "window_attn: null pointer");
+    ONELLM_REQUIRE(a.H > 0 && a.dk > 0 && a.dv > 0 && a.dk % 16 == 0 && a.dv % 16 == 0 && a.dk <= 256 && a.dv <= 256, ONELLM_ERR_UNSUPPORTED,
+                   "window_attn: key size %d and value size %d must be multiples of 16, at most 256", a.dk, a.dv);
+    ONELLM_REQUIRE(a.window > 0 && a.scale > 0.f && a.q_ld % 8 == 0 && a.out_ld % 8 == 0 && a.kv_ld % 8 == 0 && a.kv_ld >= (long)a.H * (a.dk + a.dv) &&
+                       a.kv_rows > 0 && a.kv_rows < (1l << 31),
+                   ONELLM_ERR_ARG, "window_attn: bad argument");
+    if (max_new <= 0) return ONELLM_OK;
+    BiasedAttn base = {};
+    base.H = base.G = a.H;
+    base.dk = a.dk;
+    base.dv = a.dv;
+    base.q = a.q;
+    base.ld = a.q_ld;
+    base.out = a.out;
+    base.out_ld = a.out_ld;
+    base.out_scale = a.out_scale;
+    BaParams p = {base, tp.cu, tp.hist, (a.dk + 63) / 64, (a.dv + 63) / 64, 256u, a.window, a.scale * 1.4426950408889634f, a.gate, a.gate_ld};
+    if (p.vch > 2) p.tmem_cols = 512u;
+    CUtensorMap map;
+    RC(make_map(&map, a.kv, (uint64_t)a.kv_ld, (uint64_t)a.kv_rows, kBaKV));
+    return ba_launch<true>(p, tp.B, max_new, map, map, st);
 }
 
 }  // namespace onellm
+
+extern "C" int onellm_window_attn_run(const onellm_window_attn* a, const onellm_token_positions* tp, int max_new, void* stream)
+{
+    ONELLM_REQUIRE(a && tp, ONELLM_ERR_ARG, "window_attn: null pointer");
+    return onellm::window_attn(*a, *tp, max_new, reinterpret_cast<cudaStream_t>(stream));
+}

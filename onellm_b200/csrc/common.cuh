@@ -33,6 +33,13 @@ struct TimeoutFlag {
         }                                        \
     } while (0)
 
+// Passes the status of a call on when it failed.
+#define RC(call)               \
+    do {                       \
+        int rc__ = (call);     \
+        if (rc__) return rc__; \
+    } while (0)
+
 #define ONELLM_CUDA(call)                                                                    \
     do {                                                                                     \
         cudaError_t e__ = (call);                                                            \
@@ -369,8 +376,19 @@ struct TpEpilogue {
 // element size of the types every entry point of the C interface takes (bfloat16 is known to a subset of them)
 inline size_t dtype_size(int dtype) { return dtype == ONELLM_F16 ? 2 : (dtype == ONELLM_F32 ? 4 : 0); }
 
-// Gate function of a gated projection, act(x.W) * (x.W2)
-enum GateAct { GATE_SILU = 0, GATE_RELU = 1 };
-__device__ __forceinline__ float gate_act(float g, int act) { return act == GATE_RELU ? fmaxf(g, 0.f) : g / (1.0f + __expf(-g)); }
+// Gate function of a gated projection, from g = x.W and u = x.W2 (onellm_gate_act).  PRECISE: without the fast exponential.
+enum GateAct { GATE_SILU = ONELLM_GATE_SILU, GATE_RELU = ONELLM_GATE_RELU, GATE_CLAMPED = ONELLM_GATE_CLAMPED };
+template <bool PRECISE = false>
+__device__ __forceinline__ float gate_pair(float g, float u, int act, float limit)
+{
+    if (act == GATE_RELU) return fmaxf(g, 0.f) * u;
+    float s = g;
+    if (act == GATE_CLAMPED) {
+        g = fminf(g, limit);
+        u = fminf(fmaxf(u, -limit), limit) + 1.0f;
+        s = 1.702f * g;
+    }
+    return g / (1.0f + (PRECISE ? expf(-s) : __expf(-s))) * u;
+}
 
 }  // namespace onellm

@@ -180,3 +180,96 @@ extern "C" int onellm_embedding_pos(int dtype, const int* ids, float* out, const
     ONELLM_REQUIRE(dtype == ONELLM_BF16 || dtype == ONELLM_F32, ONELLM_ERR_UNSUPPORTED, "embedding_pos: dtype %d", dtype);
     return embedding_pos_launch(dtype, ids, out, table, pos_table, n_tokens, ld, vocab, max_pos, *tp, bad, reinterpret_cast<cudaStream_t>(stream));
 }
+
+namespace onellm {
+// Token embedding through an RMSNorm into a float residual stream: out[t] = norm(table[id]) * w over `width` of ld columns.
+template <typename T>
+__global__ void __launch_bounds__(256)
+embedding_norm_kernel(const int* __restrict__ ids, float* __restrict__ out, const T* __restrict__ table, const float* __restrict__ w, float eps,
+                      int width, int ld, int vocab, int* __restrict__ bad)
+{
+    constexpr int VEC = Vec16<T>::N;
+    __shared__ float part[8];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x, id = ids[t];
+    const bool ok = id >= 0 && id < vocab;
+    if (threadIdx.x == 0 && !ok) atomicExch(bad, 1);
+    const T* src = table + (size_t)(ok ? id : 0) * ld;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < ld / VEC; i += blockDim.x) {
+        float a[VEC];
+        Vec16<T>::load(src + (size_t)i * VEC, a);
+#pragma unroll
+        for (int e = 0; e < VEC; e++) ss = fmaf(a[e], a[e], ss);
+    }
+    ss = warp_sum(ss);
+    if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = ss;
+    __syncthreads();
+    float total = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; i++) total += part[i];
+    const float inv = ok ? 1.0f / sqrtf(total / (float)width + eps) : 0.f;
+    for (int i = threadIdx.x; i < ld / VEC; i += blockDim.x) {
+        float a[VEC];
+        Vec16<T>::load(src + (size_t)i * VEC, a);
+        const float4* g = reinterpret_cast<const float4*>(w + (size_t)i * VEC);
+        float4* dst = reinterpret_cast<float4*>(out + (size_t)t * ld + (size_t)i * VEC);
+#pragma unroll
+        for (int e = 0; e < VEC; e += 4) {
+            const float4 k = g[e / 4];
+            dst[e / 4] = make_float4(a[e] * inv * k.x, a[e + 1] * inv * k.y, a[e + 2] * inv * k.z, a[e + 3] * inv * k.w);
+        }
+    }
+}
+
+// Launched with a full stream dependency, as embedding_pos_launch.
+int embedding_norm_launch(int dtype, const int* ids, float* out, const void* table, const float* w, float eps, int n_tokens, int width, int ld,
+                          int vocab, int* bad, cudaStream_t st)
+{
+    ONELLM_REQUIRE(ids && out && table && w && bad && ld % 8 == 0 && width > 0 && width <= ld, ONELLM_ERR_ARG, "embedding_norm: bad argument");
+    ONELLM_REQUIRE(dtype == ONELLM_BF16 || dtype == ONELLM_F32, ONELLM_ERR_UNSUPPORTED, "embedding_norm: dtype %d", dtype);
+    if (n_tokens <= 0) return ONELLM_OK;
+    note_launch();
+    if (dtype == ONELLM_F32) {
+        (void)prefer_max_shared((const void*)embedding_norm_kernel<float>);
+        embedding_norm_kernel<float><<<n_tokens, 256, 0, st>>>(ids, out, (const float*)table, w, eps, width, ld, vocab, bad);
+    } else {
+        (void)prefer_max_shared((const void*)embedding_norm_kernel<__nv_bfloat16>);
+        embedding_norm_kernel<__nv_bfloat16><<<n_tokens, 256, 0, st>>>(ids, out, (const __nv_bfloat16*)table, w, eps, width, ld, vocab, bad);
+    }
+    ONELLM_CHECK_LAUNCH();
+    return ONELLM_OK;
+}
+
+// out[r, c] = cap * tanh(in[r, c] / cap), rows of ld elements into dense rows
+__global__ void __launch_bounds__(256) softcap_kernel(const float* __restrict__ in, long ld, float* __restrict__ out, int cols, float cap)
+{
+    pdl_launch_dependents();
+    pdl_wait();
+    const float* src = in + (size_t)blockIdx.y * ld;
+    float* dst = out + (size_t)blockIdx.y * cols;
+    for (int c = blockIdx.x * blockDim.x + threadIdx.x; c < cols; c += gridDim.x * blockDim.x) dst[c] = cap * tanhf(src[c] / cap);
+}
+
+int softcap(const float* in, long ld, float* out, int rows, int cols, float cap, cudaStream_t st)
+{
+    ONELLM_REQUIRE(in && out && ld >= cols && cols > 0 && cap > 0.f, ONELLM_ERR_ARG, "softcap: bad argument");
+    for (int r = 0; r < rows; r += 65535) {
+        const int n = rows - r < 65535 ? rows - r : 65535;
+        ONELLM_CUDA(launch_pdl(softcap_kernel, dim3((cols + 1023) / 1024, n), dim3(256), 0, st, in + (size_t)r * ld, ld, out + (size_t)r * cols, cols, cap));
+    }
+    return ONELLM_OK;
+}
+}  // namespace onellm
+
+extern "C" int onellm_embedding_norm(int dtype, const int* ids, float* out, const void* table, const float* w, float eps, int n_tokens, int width,
+                                     int ld, int vocab, int* bad, void* stream)
+{
+    return embedding_norm_launch(dtype, ids, out, table, w, eps, n_tokens, width, ld, vocab, bad, reinterpret_cast<cudaStream_t>(stream));
+}
+
+extern "C" int onellm_softcap(const float* in, long ld, float* out, int rows, int cols, float cap, void* stream)
+{
+    return softcap(in, ld, out, rows, cols, cap, reinterpret_cast<cudaStream_t>(stream));
+}

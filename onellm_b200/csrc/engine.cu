@@ -179,7 +179,7 @@ int Engine::run_step(int mode, int prompt_len)
     ONELLM_REQUIRE(step <= max_seq_len, ONELLM_ERR_STATE, "decode: sequence length %d exceeds max_seq_len %d", step,
                    max_seq_len);
     int bound = (step + 255) / 256 * 256;
-    if (bound > max_seq_len) bound = max_seq_len;
+    bound = std::min({bound, max_seq_len, span_cap});
     if (!use_graphs) {
         const long before = launches_noted();
         RC(enqueue_step(mode, bound, prompt_len));
@@ -269,6 +269,7 @@ int Engine::prefill_context(int B, const int* lens)
     last_logits = c.logits;
     c.cu = d_cu;
     c.hist = d_hist;
+    c.host_hist = hist.data();
     c.rows = d_rows;
     ONELLM_CUDA(cudaMemcpyAsync(d_step_off, off.data(), B * sizeof(int), cudaMemcpyHostToDevice, stream));
     ONELLM_CUDA(cudaMemcpyAsync(d_cu, cu.data(), (B + 1) * sizeof(int), cudaMemcpyHostToDevice, stream));

@@ -10,12 +10,6 @@
 
 namespace onellm {
 
-#define RC(call)              \
-    do {                      \
-        int rc__ = (call);    \
-        if (rc__) return rc__; \
-    } while (0)
-
 inline size_t align_up(size_t x, size_t a) { return (x + a - 1) / a * a; }
 inline int blocks_for(size_t n) { return (int)((n + 255) / 256 < 4096 ? (n + 255) / 256 : 4096); }
 
@@ -42,6 +36,7 @@ struct ContextBatch {
     size_t T = 0;              // tokens
     const int* cu = nullptr;   // device [B + 1]: token offsets of the sequences
     const int* hist = nullptr; // device [B]: positions a sequence has cached
+    const int* host_hist = nullptr;  // the same on the host
     const int* rows = nullptr; // device [n_rows]: packed token rows whose logits are wanted, the last one of every
     int n_rows = 0;            // sequence first (those B rows are sampled from)
     void* logits = nullptr;    // device [n_rows, vocab] of Engine::logits_dtype
@@ -50,6 +45,7 @@ struct ContextBatch {
 struct Engine {
     // capacity and vocabulary, set by the design's constructor
     int vocab = 0, max_seq_len = 0, max_batch = 0, eos_id = 2;
+    int span_cap = 0x7fffffff;  // most positions a launch of a decode step depends on (the longest window of a windowed design)
     int logits_dtype = ONELLM_F16;
     // memory
     char* arena = nullptr;
@@ -95,7 +91,8 @@ struct Engine {
     virtual const char* design() const = 0;
     virtual void carve(Carver& cv) = 0;
     // From the batch ids in d_ids (and, for every sequence b, its position *d_step - 1 + d_step_off[b]) through all
-    // layers; with_head also the logits of every sequence into `logits`.  `step_bound` is an upper bound of *d_step.
+    // layers; with_head also the logits of every sequence into `logits`.  `step_bound` is an upper bound of
+    // min(*d_step, span_cap).
     virtual int decode_layers(int step_bound, bool with_head) = 0;
     // All tokens of a context pass through all layers, and the logits of c.rows into c.logits.
     virtual int context_layers(const ContextBatch& c) = 0;

@@ -5,7 +5,7 @@
 // logarithmic distance penalty instead of a rotation, an HGRN2 recurrence and a ReLU-gated feed-forward (a layer may
 // have none).  Layers may share the weights of another layer; every layer run has its own cache and state.
 //
-// The parallel form sets the launches of a layer.  All branch inputs come from one pass over the stream (norm_pair), all
+// The parallel form sets the launches of a layer.  All branch inputs come from one pass over the stream (norm_rows), all
 // mixer projections are one matrix [width, q | k | v | q' | f | v'], and all branch outputs are columns of one buffer
 //     cat = [ left_scale * attention | right_scale * recurrence | relu(gate) * up ]
 // whose product with the stacked output weights [W_o ; W_o' ; W_down] is added to the float residual stream in the
@@ -23,10 +23,9 @@
 #include "mixers.h"
 #include "model_files.h"
 #include "project.h"
+#include "weight_placer.h"
 
 namespace onellm {
-
-static int pad_to(int x, int m) { return (x + m - 1) / m * m; }
 
 struct FinuvikLayerConfig {
     int weights_of = -1;  // the layer whose tensors are used (itself, or the one named)
@@ -158,7 +157,8 @@ struct Finuvik : Engine {
         void* rec_work;  // context pass only
     };
     int layer(size_t i, const Buffers& buf, int tokens, const TokenPositions& tp, int max_new, int step_bound);
-    int lm_head(const float* stream_rows, const int* rows, int n_rows, void* hn, float* padded, float* out);
+    int norm(float* stream_rows, const int* rows, int n_rows, const float* w1, const float* w2, void* out1, void* out2);
+    int lm_head(float* stream_rows, const int* rows, int n_rows, void* hn, float* padded, float* out);
     int load(const std::string& folder);
     int finalize();
     bool own(size_t i) const { return c.layers[i].weights_of == (int)i; }
@@ -222,6 +222,11 @@ void Finuvik::carve(Carver& cv)
     ws = cv.take_bytes(biased_attn_decode_workspace((int)B, max_ws_heads, max_ws_dv));
 }
 
+int Finuvik::norm(float* stream_rows, const int* rows, int n_rows, const float* w1, const float* w2, void* out1, void* out2)
+{
+    return norm_rows({dtype, stream_rows, rows, n_rows, w1, w2, out1, out2, (float)c.eps, 1.f, c.width, width, nullptr, nullptr, 0, 0.f}, stream);
+}
+
 // One layer over `tokens` tokens: a context pass (tp.cu) or a decode step.
 int Finuvik::layer(size_t i, const Buffers& buf, int tokens, const TokenPositions& tp, int max_new, int step_bound)
 {
@@ -229,8 +234,8 @@ int Finuvik::layer(size_t i, const Buffers& buf, int tokens, const TokenPosition
     const FinuvikWeights& w = weights[l.weights_of];
     const size_t es = esize();
     auto at = [es](void* base, int col) { return static_cast<void*>(static_cast<char*>(base) + (size_t)col * es); };
-    RC(norm_pair(dtype, buf.x, nullptr, tokens, w.norm1, w.norm2, buf.h1, w.ff ? buf.h2 : nullptr, (float)c.eps, c.width, width, stream));
-    Projection pj = {};
+    RC(norm(buf.x, nullptr, tokens, w.norm1, w.norm2, buf.h1, w.ff ? buf.h2 : nullptr));
+    Projection pj;
     pj.dtype = dtype;
     pj.M = tokens;
     pj.x = buf.h1;
@@ -307,10 +312,10 @@ int Finuvik::layer(size_t i, const Buffers& buf, int tokens, const TokenPosition
 }
 
 // Final norm and head of some rows of the stream; logits in float, [n_rows, vocab].
-int Finuvik::lm_head(const float* stream_rows, const int* rows, int n_rows, void* hn, float* padded, float* out)
+int Finuvik::lm_head(float* stream_rows, const int* rows, int n_rows, void* hn, float* padded, float* out)
 {
-    RC(norm_pair(dtype, stream_rows, rows, n_rows, final_norm, nullptr, hn, nullptr, (float)c.eps, c.width, width, stream));
-    Projection pj = {};
+    RC(norm(stream_rows, rows, n_rows, final_norm, nullptr, hn, nullptr));
+    Projection pj;
     pj.dtype = dtype;
     pj.M = n_rows;
     pj.x = hn;
@@ -350,7 +355,7 @@ int Finuvik::context_layers(const ContextBatch& cb)
         buf.cat = cv.take_bytes(T * max_cat * es);
         size_t work = 0;
         for (size_t i = 0; i < c.layers.size(); i++)
-            work = std::max(work, gated_recurrence_workspace((int)T, c.layers[i].RH, weights[i].rk, weights[i].rv));
+            work = std::max(work, gated_recurrence_workspace(ONELLM_GR_TIED, (int)T, c.layers[i].RH, weights[i].rk, weights[i].rv));
         buf.rec_work = cv.take_bytes(work);
         hn = cv.take_bytes((size_t)cb.n_rows * W * es);
         padded = vocab_p == c.vocab ? nullptr : cv.take<float>((size_t)cb.n_rows * vocab_p);
@@ -368,81 +373,9 @@ int Finuvik::context_layers(const ContextBatch& cb)
 }
 
 // ---- weights -----------------------------------------------------------------------------------------------
-// src [out, in] (bfloat16) -> dst [.., ld] of type T, transposed: element (o, i) goes to row (i / in_d) * in_p + i % in_d,
-// column (o / out_d) * out_p + o % out_d: heads of in_d / out_d elements padded to in_p / out_p.  The rest stays zero.
-template <typename T>
-__global__ void place_kernel(T* __restrict__ dst, int ld, const __nv_bfloat16* __restrict__ src, int out, int in, int out_d, int out_p, int in_d,
-                             int in_p, int transposed)
-{
-    const size_t n = (size_t)out * in;
-    for (size_t e = blockIdx.x * (size_t)blockDim.x + threadIdx.x; e < n; e += (size_t)gridDim.x * blockDim.x) {
-        const int o = (int)(e / in), i = (int)(e % in);
-        const size_t r = (size_t)(i / in_d) * in_p + i % in_d, col = (size_t)(o / out_d) * out_p + o % out_d;
-        dst[transposed ? r * ld + col : col * ld + r] = from_float<T>(__bfloat162float(src[e]));
-    }
-}
-
-// Places tensors of a file; one staging buffer on the device.
-struct FinuvikLoader {
-    Finuvik& m;
-    SafeTensors file;
-    __nv_bfloat16* stage = nullptr;
-    size_t stage_bytes = 0;
-
-    explicit FinuvikLoader(Finuvik& model) : m(model) {}
-    ~FinuvikLoader()
-    {
-        if (stage) cudaFree(stage);
-    }
-    // the tensor's raw bfloat16 data in `stage`
-    int fetch(const std::string& name, int64_t rows, int64_t cols)
-    {
-        const SafeTensor* t = file.find(name);
-        ONELLM_REQUIRE(t, ONELLM_ERR_IO, "no tensor %s", name.c_str());
-        const std::vector<int64_t> want = cols > 0 ? std::vector<int64_t>{rows, cols} : std::vector<int64_t>{rows};
-        ONELLM_REQUIRE(t->shape == want && t->dtype == "BF16", ONELLM_ERR_IO, "tensor %s: expected bfloat16 [%lld%s%s]", name.c_str(), (long long)rows,
-                       cols > 0 ? ", " : "", cols > 0 ? std::to_string(cols).c_str() : "");
-        std::vector<char> raw;
-        RC(file.read(*t, &raw));
-        ONELLM_REQUIRE(raw.size() == (size_t)rows * (cols > 0 ? cols : 1) * 2, ONELLM_ERR_IO, "tensor %s: wrong number of bytes", name.c_str());
-        if (raw.size() > stage_bytes) {
-            if (stage) cudaFree(stage);
-            stage = nullptr;
-            stage_bytes = 0;
-            ONELLM_CUDA(cudaMalloc(&stage, raw.size()));
-            stage_bytes = raw.size();
-        }
-        ONELLM_CUDA(cudaMemcpyAsync(stage, raw.data(), raw.size(), cudaMemcpyHostToDevice, m.stream));
-        ONELLM_CUDA(cudaStreamSynchronize(m.stream));  // `raw` goes away, the stage is used again
-        return ONELLM_OK;
-    }
-    int place(const std::string& name, void* dst, int ld, int row, int col, int out, int out_d, int out_p, int in, int in_d, int in_p, bool transposed = true)
-    {
-        RC(fetch(name, out, in));
-        const size_t at = transposed ? (size_t)row * ld + col : (size_t)col * ld + row;
-        const int nb = blocks_for((size_t)out * in);
-        if (m.dtype == ONELLM_F32)
-            place_kernel<float><<<nb, 256, 0, m.stream>>>(static_cast<float*>(dst) + at, ld, stage, out, in, out_d, out_p, in_d, in_p, transposed);
-        else
-            place_kernel<__nv_bfloat16><<<nb, 256, 0, m.stream>>>(static_cast<__nv_bfloat16*>(dst) + at, ld, stage, out, in, out_d, out_p, in_d, in_p, transposed);
-        ONELLM_CHECK_LAUNCH();
-        ONELLM_CUDA(cudaStreamSynchronize(m.stream));
-        return ONELLM_OK;
-    }
-    // a vector kept in float, heads of d padded to p
-    int vec(const std::string& name, float* dst, int n, int d, int p)
-    {
-        RC(fetch(name, n, 0));
-        place_kernel<float><<<blocks_for(n), 256, 0, m.stream>>>(dst, 1, stage, n, 1, d, p, 1, 1, 0);
-        ONELLM_CHECK_LAUNCH();
-        ONELLM_CUDA(cudaStreamSynchronize(m.stream));
-        return ONELLM_OK;
-    }
-};
-
 int Finuvik::load(const std::string& folder)
 {
-    FinuvikLoader f(*this);
+    WeightPlacer f(dtype, stream);
     RC(f.file.open(folder + "/model.safetensors"));
     const int D = c.width;
     // plain [rows, width] tables keep their orientation

@@ -20,6 +20,7 @@
 #include <algorithm>
 #include <mutex>
 
+#include "project.h"
 #include "tc_common.cuh"
 
 namespace onellm {
@@ -54,6 +55,12 @@ constexpr int kTcSmemBytes = kTcStages * kTcStageBytes + 1024 /* alignment slack
 //   act:     gate function of MODE 2
 //   ldy:     row stride of y (and of resid); 0: N
 //   f32:     y and resid are float instead of the element type (no ss_out then)
+//   scale:   with f32, factor on the result in front of the residual
+//   limit:   bound of the clamped gate function
+// GROUPED: the rows of x and y lie in groups with weights of their own (onellm_row_groups: the experts of a mixture).  The
+// row tiles come from a table, 128 rows of one group each; the weights are stacked, so that a tile reads K rows of W from
+// row group * K on.  Columns of x behind K are zero-filled, so that a last K slice that reaches into the next weight adds
+// nothing.
 struct TcEpilogue {
     const float* row_ss;
     int ss_parts;
@@ -64,12 +71,13 @@ struct TcEpilogue {
     int act;
     long ldy;
     int f32;
+    float scale = 1.f, limit = 0.f;
 };
 
-template <typename T, int MODE>
+template <typename T, int MODE, bool GROUPED = false>
 __global__ void __launch_bounds__(kTcThreads)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
-               const __grid_constant__ CUtensorMap map_b2, T* y, int M, int N, int K, const TcEpilogue epi)
+               const __grid_constant__ CUtensorMap map_b2, T* y, int M, int N, int K, const TcEpilogue epi, const RowGroups grp)
 {
     constexpr bool W_NK = MODE == 1;
     constexpr bool DUAL = MODE == 2;
@@ -86,14 +94,26 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
     // tile to the right, so the tiles in flight at one time (one per SM) cover a near-square patch
     // of the output and share their A row blocks and B column blocks in L2.  (Row-major order made every
     // wave touch all column tiles of B: operands were read from DRAM seven times over.)
-    const int tiles_m = (M + kTcBM - 1) / kTcBM, tiles_n = (N + kOutN - 1) / kOutN;
-    const int n_tiles = tiles_m * tiles_n;
-    auto tile_origin = [&](int t, int& m0, int& n0) {
+    int tiles_m = (M + kTcBM - 1) / kTcBM;
+    const int tiles_n = (N + kOutN - 1) / kOutN;
+    int n_tiles = tiles_m * tiles_n;
+    // first row and column of a tile, the row of the stacked weights it starts at, the end of its rows
+    auto tile_origin = [&](int t, int& m0, int& n0, int& k0, int& m_end) {
         const int per_band = kTcBand * tiles_n;
         const int band = t / per_band, in_band = t % per_band;
         const int band_rows = min(kTcBand, tiles_m - band * kTcBand);
-        m0 = (band * kTcBand + in_band % band_rows) * kTcBM;
+        const int mt = band * kTcBand + in_band % band_rows;
         n0 = (in_band / band_rows) * kOutN;
+        if constexpr (GROUPED) {
+            const int g = grp.tile_group[mt];
+            m0 = grp.tile_row[mt];
+            k0 = g * K;
+            m_end = grp.off[g + 1];
+        } else {
+            m0 = mt * kTcBM;
+            k0 = 0;
+            m_end = M;
+        }
     };
     const int k_steps = (K + kTcBK - 1) / kTcBK;
 
@@ -119,14 +139,18 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
     const uint32_t tmem_base = *tmem_slot;
 
     pdl_wait();  // x comes from the previous kernel in the stream
+    if constexpr (GROUPED) {
+        tiles_m = *grp.n_tiles;
+        n_tiles = tiles_m * tiles_n;
+    }
 
     if (warp == 0 && lane == 0) {
         // producer: one 64-deep slice of A and of B per stage, tile after tile
         int it = 0;
         bool ok = true;
         for (int t = blockIdx.x; t < n_tiles && ok; t += gridDim.x) {
-            int m0, n0;
-            tile_origin(t, m0, n0);
+            int m0, n0, k0, m_end;
+            tile_origin(t, m0, n0, k0, m_end);
             for (int ks = 0; ks < k_steps; ks++, it++) {
                 const int s = it % kTcStages;
                 if (it >= kTcStages) ok = mbar_wait(empty0 + 8 * s, ((it / kTcStages) - 1) & 1);
@@ -139,13 +163,13 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                 } else if (DUAL) {
 #pragma unroll
                     for (int c = 0; c < 2; c++) {
-                        tma_load_2d(b_dst + c * kTcBChunk, &map_b, n0 + 64 * c, ks * kTcBK, full0 + 8 * s);
-                        tma_load_2d(b_dst + (2 + c) * kTcBChunk, &map_b2, n0 + 64 * c, ks * kTcBK, full0 + 8 * s);
+                        tma_load_2d(b_dst + c * kTcBChunk, &map_b, n0 + 64 * c, k0 + ks * kTcBK, full0 + 8 * s);
+                        tma_load_2d(b_dst + (2 + c) * kTcBChunk, &map_b2, n0 + 64 * c, k0 + ks * kTcBK, full0 + 8 * s);
                     }
                 } else {
 #pragma unroll
                     for (int c = 0; c < kTcBN / 64; c++)
-                        tma_load_2d(b_dst + c * kTcBChunk, &map_b, n0 + 64 * c, ks * kTcBK, full0 + 8 * s);
+                        tma_load_2d(b_dst + c * kTcBChunk, &map_b, n0 + 64 * c, k0 + ks * kTcBK, full0 + 8 * s);
                 }
             }
         }
@@ -189,15 +213,18 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
         bool ok = true;
         for (int t = blockIdx.x; t < n_tiles && ok; t += gridDim.x, lt++) {
             const int acc = lt & 1, use = lt >> 1;
-            int m0, n0;
-            tile_origin(t, m0, n0);
+            int m0, n0, k0, m_end;
+            tile_origin(t, m0, n0, k0, m_end);
             ok = mbar_wait(acc_full0 + 8 * acc, use & 1);
             ok = __all_sync(0xffffffffu, ok);
             if (!ok) break;
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
             const int row = m0 + q * 32 + lane;
+            const bool row_ok = row < m_end;
             float inv = 1.f, sq = 0.f;
-            if (epi.row_ss && row < M) {
+            const bool scaled = GROUPED ? grp.row_scale != nullptr : epi.row_ss != nullptr;
+            if (GROUPED && scaled && row_ok) inv = grp.row_scale[row];
+            if (epi.row_ss && row_ok) {
                 float ssum = 0.f;
                 for (int pp = 0; pp < epi.ss_parts; pp++) ssum += epi.row_ss[(size_t)row * epi.ss_parts + pp];
                 inv = rsqrtf(ssum / (float)K + epi.eps);
@@ -213,16 +240,16 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
 #pragma unroll
                     for (int i = 0; i < 32; i++) {
                         const float g = __uint_as_float(r[i]) * inv;
-                        r[i] = __float_as_uint(gate_act(g, epi.act) * (__uint_as_float(u[i]) * inv));
+                        r[i] = __float_as_uint(gate_pair(g, __uint_as_float(u[i]) * inv, epi.act, epi.limit));
                     }
                 } else {
                     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-                    if (epi.row_ss) {
+                    if (scaled) {
 #pragma unroll
                         for (int i = 0; i < 32; i++) r[i] = __float_as_uint(__uint_as_float(r[i]) * inv);
                     }
                 }
-                if (row < M) {
+                if (row_ok) {
                     const size_t at = (size_t)row * ldy + n0 + c0;
 #pragma unroll
                     for (int j = 0; j < 4; j++) {
@@ -241,8 +268,9 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                                 if (epi.resid) {
                                     const float4* rs = reinterpret_cast<const float4*>(static_cast<const float*>(epi.resid) + at + 8 * j);
                                     const float4 r0 = rs[0], r1 = rs[1];
-                                    v[0] += r0.x; v[1] += r0.y; v[2] += r0.z; v[3] += r0.w;
-                                    v[4] += r1.x; v[5] += r1.y; v[6] += r1.z; v[7] += r1.w;
+                                    const float sc = epi.scale;
+                                    v[0] = fmaf(v[0], sc, r0.x); v[1] = fmaf(v[1], sc, r0.y); v[2] = fmaf(v[2], sc, r0.z); v[3] = fmaf(v[3], sc, r0.w);
+                                    v[4] = fmaf(v[4], sc, r1.x); v[5] = fmaf(v[5], sc, r1.y); v[6] = fmaf(v[6], sc, r1.z); v[7] = fmaf(v[7], sc, r1.w);
                                 }
                                 dst[0] = make_float4(v[0], v[1], v[2], v[3]);
                                 dst[1] = make_float4(v[4], v[5], v[6], v[7]);
@@ -264,7 +292,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                     }
                 }
             }
-            if (epi.ss_out && row < M) epi.ss_out[(size_t)row * tiles_n + n0 / kOutN] = sq;
+            if (epi.ss_out && row_ok) epi.ss_out[(size_t)row * tiles_n + n0 / kOutN] = sq;
             // this thread's reads of the accumulator are over: hand it back to the MMA warp
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
             mbar_arrive(acc_empty0 + 8 * acc);
@@ -342,11 +370,39 @@ static int gemm_tc_launch(const T* x, const T* W, const T* W2, T* y, int M, int 
     ONELLM_REQUIRE(tiles <= 0x7fffffffL, ONELLM_ERR_UNSUPPORTED, "gemm: too many tiles");
     const dim3 grid((unsigned)std::min<long>(tiles, num_sms()));  // persistent: one block per SM (shared memory allows no more)
     if (mode == 0)
-        ONELLM_CUDA(launch_pdl(gemm_tc_kernel<T, 0>, grid, dim3(kTcThreads), kTcSmemBytes, st, map_a, map_b, map_b2, y, M, N, K, epi));
+        ONELLM_CUDA(launch_pdl(gemm_tc_kernel<T, 0>, grid, dim3(kTcThreads), kTcSmemBytes, st, map_a, map_b, map_b2, y, M, N, K, epi, RowGroups{}));
     else if (mode == 1)
-        ONELLM_CUDA(launch_pdl(gemm_tc_kernel<T, 1>, grid, dim3(kTcThreads), kTcSmemBytes, st, map_a, map_b, map_b2, y, M, N, K, epi));
+        ONELLM_CUDA(launch_pdl(gemm_tc_kernel<T, 1>, grid, dim3(kTcThreads), kTcSmemBytes, st, map_a, map_b, map_b2, y, M, N, K, epi, RowGroups{}));
     else
-        ONELLM_CUDA(launch_pdl(gemm_tc_kernel<T, 2>, grid, dim3(kTcThreads), kTcSmemBytes, st, map_a, map_b, map_b2, y, M, N, K, epi));
+        ONELLM_CUDA(launch_pdl(gemm_tc_kernel<T, 2>, grid, dim3(kTcThreads), kTcSmemBytes, st, map_a, map_b, map_b2, y, M, N, K, epi, RowGroups{}));
+    return ONELLM_OK;
+}
+
+// Row groups (bfloat16): x has g.rows rows in group order, the weights are stacked.
+static int gemm_tc_grouped(const onellm_projection& p, const TcEpilogue& epi, cudaStream_t st)
+{
+    typedef __nv_bfloat16 T;
+    const RowGroups& g = *p.groups;
+    ONELLM_REQUIRE(g.off && g.tile_group && g.tile_row && g.n_tiles && g.max_tiles > 0 && g.rows > 0 && g.weights > 0 && !g.x_rows && !g.x_stride &&
+                       !g.y_stride && g.w_stride == (long)p.K * p.N && !p.ldw && !p.ldx && !p.resid,
+                   ONELLM_ERR_UNSUPPORTED, "project: more than 64 rows per group need a tile table, rows in group order and stacked weights");
+    CUtensorMap map_a, map_b, map_b2;
+    int rc = make_map(&map_a, p.x, (uint64_t)p.K, (uint64_t)g.rows, kTcBM);
+    if (!rc) rc = make_map(&map_b, p.W, (uint64_t)p.N, (uint64_t)p.K * g.weights, kTcBK);
+    map_b2 = map_b;
+    if (!rc && p.W2) rc = make_map(&map_b2, p.W2, (uint64_t)p.N, (uint64_t)p.K * g.weights, kTcBK);
+    if (rc) return rc;
+    const void* fn = p.W2 ? (const void*)gemm_tc_kernel<T, 2, true> : (const void*)gemm_tc_kernel<T, 0, true>;
+    static DeviceOnce attr[2];
+    ONELLM_CUDA(attr[p.W2 ? 1 : 0].run([fn] { return cudaFuncSetAttribute(fn, cudaFuncAttributeMaxDynamicSharedMemorySize, kTcSmemBytes); }));
+    const int out_n = p.W2 ? kTcBN / 2 : kTcBN;
+    const long tiles = (long)((p.N + out_n - 1) / out_n) * g.max_tiles;
+    ONELLM_REQUIRE(tiles <= 0x7fffffffL, ONELLM_ERR_UNSUPPORTED, "gemm: too many tiles");
+    const dim3 grid((unsigned)std::min<long>(tiles, num_sms()));
+    if (p.W2)
+        ONELLM_CUDA(launch_pdl(gemm_tc_kernel<T, 2, true>, grid, dim3(kTcThreads), kTcSmemBytes, st, map_a, map_b, map_b2, (T*)p.y, p.M, p.N, p.K, epi, g));
+    else
+        ONELLM_CUDA(launch_pdl(gemm_tc_kernel<T, 0, true>, grid, dim3(kTcThreads), kTcSmemBytes, st, map_a, map_b, map_b2, (T*)p.y, p.M, p.N, p.K, epi, g));
     return ONELLM_OK;
 }
 
@@ -383,17 +439,19 @@ int gemm_rows_f16(const __half* x, const __half* W, const __half* W2, __half* y,
     return gemm_tc_launch<__half>(x, W, W2, y, M, N, K, W2 ? 2 : 0, st, epi);
 }
 
-// The bfloat16 form (more than 64 tokens) for the model classes: W and W2 [K,N] (W2: gate form, act(x.W) * (x.W2)); y in
-// bfloat16 or, with f32, in float with an optional float residual; ldy is the row stride of y and resid.
-int gemm_bf16_large(const __nv_bfloat16* x, const __nv_bfloat16* W, const __nv_bfloat16* W2, void* y, long ldy, int M, int N, int K, int act,
-                    int f32, const float* resid, cudaStream_t st)
+// The bfloat16 form (more than 64 tokens, or rows in one group) behind project().
+int gemm_bf16_large(const onellm_projection& p, cudaStream_t st)
 {
+    typedef __nv_bfloat16 bf16;
     TcEpilogue epi = {};
-    epi.resid = resid;
-    epi.act = act;
-    epi.ldy = ldy;
-    epi.f32 = f32;
-    return gemm_tc_launch<__nv_bfloat16>(x, W, W2, static_cast<__nv_bfloat16*>(y), M, N, K, W2 ? 2 : 0, st, epi);
+    epi.resid = p.resid;
+    epi.act = p.act;
+    epi.limit = p.limit;
+    epi.scale = p.scale;
+    epi.ldy = p.ldy;
+    epi.f32 = p.f32;
+    if (p.groups) return gemm_tc_grouped(p, epi, st);
+    return gemm_tc_launch<bf16>((const bf16*)p.x, (const bf16*)p.W, (const bf16*)p.W2, static_cast<bf16*>(p.y), p.M, p.N, p.K, p.W2 ? 2 : 0, st, epi);
 }
 
 static const TimeoutFlag timeout_flag(tc_flag_read_clear);

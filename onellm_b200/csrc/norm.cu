@@ -8,7 +8,7 @@
 // thread owns up to kMaxVec 16-byte vectors of the row and keeps them in registers between
 // the sum-of-squares reduction and the scaling, so a row is read once and written once.
 // Rows too long for the register budget are re-read from L2 in the second phase.
-#include "common.cuh"
+#include "mixers.h"
 
 namespace onellm {
 
@@ -171,46 +171,69 @@ extern "C" int onellm_row_sumsq(int dtype, const void* x, int rows, int cols, fl
 }
 
 namespace onellm {
-// RMSNorm whose weights are offsets from one, out of a float residual stream: for row r (or rows[r]) of x
-//     out_i[r] = x * rsqrt(mean(x^2) + eps) * (1 + w_i)          i = 1, 2 (out2 may be NULL)
+// RMSNorm of a float residual stream: for row r (or rows[r]) of x
+//     out_i[r] = x * rsqrt(mean(x^2) + eps) * (w_base + w_i)          i = 1, 2 (out2 may be NULL)
 // into one or two buffers of element type T: two parallel branches that normalise the same stream with weights of their
 // own share one pass over it.  `width` columns count, `ld` is the row stride of all buffers (the columns behind `width`
 // hold zeros and get zeros).
+// ADD: the stream first takes add_scale times the sum of add_n rows of `add` (what the experts of a token made of it), so
+// that a feed-forward's last step and the next norm are one pass; out1 may be NULL then.
 constexpr int kPairVec = 8;  // float4 per thread kept in registers
-template <typename T>
-__global__ void __launch_bounds__(kNormThreads)
-norm_pair_kernel(const float* __restrict__ x, const int* __restrict__ rows, const float* __restrict__ w1, const float* __restrict__ w2,
-                 T* __restrict__ out1, T* __restrict__ out2, float eps, int width, int ld)
+template <typename T, bool ADD>
+__global__ void __launch_bounds__(kNormThreads) norm_rows_kernel(const NormRows p)
 {
     pdl_launch_dependents();
     pdl_wait();
-    const float4* xr = reinterpret_cast<const float4*>(x + (size_t)(rows ? rows[blockIdx.x] : blockIdx.x) * ld);
-    const int nvec = ld / 4;
+    float4* xr = reinterpret_cast<float4*>(p.x + (size_t)(p.rows ? p.rows[blockIdx.x] : blockIdx.x) * p.ld);
+    const int nvec = p.ld / 4;
+    const int* add_rows = ADD ? p.add_rows + (size_t)blockIdx.x * p.add_n : nullptr;
+    auto fetch = [&](int i) {
+        float4 v = xr[i];
+        if constexpr (ADD) {
+            float a[4] = {0.f, 0.f, 0.f, 0.f};
+            for (int k = 0; k < p.add_n; k++) {
+                const T* src = static_cast<const T*>(p.add) + (size_t)add_rows[k] * p.ld + 4 * i;
+                if constexpr (std::is_same<T, float>::value) {
+                    const float4 f = *reinterpret_cast<const float4*>(src);
+                    a[0] += f.x; a[1] += f.y; a[2] += f.z; a[3] += f.w;
+                } else {
+                    const uint2 w = *reinterpret_cast<const uint2*>(src);
+                    const float2 lo = unpack2<T>(w.x), hi = unpack2<T>(w.y);
+                    a[0] += lo.x; a[1] += lo.y; a[2] += hi.x; a[3] += hi.y;
+                }
+            }
+            v = make_float4(fmaf(p.add_scale, a[0], v.x), fmaf(p.add_scale, a[1], v.y), fmaf(p.add_scale, a[2], v.z), fmaf(p.add_scale, a[3], v.w));
+            xr[i] = v;
+        }
+        return v;
+    };
     float4 keep[kPairVec];
     float ss = 0.f;
 #pragma unroll
     for (int j = 0; j < kPairVec; j++) {
         const int i = threadIdx.x + j * kNormThreads;
         if (i < nvec) {
-            keep[j] = xr[i];
+            keep[j] = fetch(i);
             ss = fmaf(keep[j].x, keep[j].x, fmaf(keep[j].y, keep[j].y, fmaf(keep[j].z, keep[j].z, fmaf(keep[j].w, keep[j].w, ss))));
         }
     }
     for (int i = threadIdx.x + kPairVec * kNormThreads; i < nvec; i += kNormThreads) {
-        const float4 v = xr[i];
+        const float4 v = fetch(i);
         ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
     }
-    const float inv = 1.0f / sqrtf(block_sum_256(ss) / (float)width + eps);
+    if (ADD && !p.out1) return;
+    const float inv = 1.0f / sqrtf(block_sum_256(ss) / (float)p.width + p.eps);
     auto emit = [&](int i, const float4& v) {
-        auto one = [&](const float* w, T* out) {
+        auto one = [&](const float* w, void* out) {
             const float4 g = reinterpret_cast<const float4*>(w)[i];
-            const float o[4] = {v.x * inv * (1.f + g.x), v.y * inv * (1.f + g.y), v.z * inv * (1.f + g.z), v.w * inv * (1.f + g.w)};
-            T* dst = out + (size_t)blockIdx.x * ld + 4 * i;
+            const float b = p.w_base;
+            const float o[4] = {v.x * inv * (b + g.x), v.y * inv * (b + g.y), v.z * inv * (b + g.z), v.w * inv * (b + g.w)};
+            T* dst = static_cast<T*>(out) + (size_t)blockIdx.x * p.ld + 4 * i;
             if constexpr (std::is_same<T, float>::value) *reinterpret_cast<float4*>(dst) = make_float4(o[0], o[1], o[2], o[3]);
             else *reinterpret_cast<uint2*>(dst) = make_uint2(pack2<T>(o[0], o[1]), pack2<T>(o[2], o[3]));
         };
-        one(w1, out1);
-        if (out2) one(w2, out2);
+        one(p.w1, p.out1);
+        if (p.out2) one(p.w2, p.out2);
     };
 #pragma unroll
     for (int j = 0; j < kPairVec; j++) {
@@ -220,17 +243,21 @@ norm_pair_kernel(const float* __restrict__ x, const int* __restrict__ rows, cons
     for (int i = threadIdx.x + kPairVec * kNormThreads; i < nvec; i += kNormThreads) emit(i, xr[i]);
 }
 
-int norm_pair(int dtype, const float* x, const int* rows, int n_rows, const float* w1, const float* w2, void* out1, void* out2, float eps,
-              int width, int ld, cudaStream_t st)
+int norm_rows(const NormRows& n, cudaStream_t st)
 {
-    ONELLM_REQUIRE(x && w1 && out1 && ld % 4 == 0 && width > 0 && width <= ld, ONELLM_ERR_ARG, "norm_pair: bad argument");
-    if (n_rows <= 0) return ONELLM_OK;
-    if (dtype == ONELLM_F32)
-        ONELLM_CUDA(launch_pdl(norm_pair_kernel<float>, dim3(n_rows), dim3(kNormThreads), 0, st, x, rows, w1, w2, (float*)out1, (float*)out2,
-                               eps, width, ld));
-    else
-        ONELLM_CUDA(launch_pdl(norm_pair_kernel<__nv_bfloat16>, dim3(n_rows), dim3(kNormThreads), 0, st, x, rows, w1, w2, (__nv_bfloat16*)out1,
-                               (__nv_bfloat16*)out2, eps, width, ld));
+    ONELLM_REQUIRE(n.x && (n.out1 ? n.w1 != nullptr : n.add != nullptr) && (!n.out2 || (n.out1 && n.w2)) && (!n.add || n.add_rows), ONELLM_ERR_ARG,
+                   "norm_rows: null pointer");
+    ONELLM_REQUIRE(n.ld % 4 == 0 && n.width > 0 && n.width <= n.ld && n.add_n >= 0, ONELLM_ERR_ARG, "norm_rows: bad size");
+    ONELLM_REQUIRE(n.dtype == ONELLM_BF16 || n.dtype == ONELLM_F32, ONELLM_ERR_UNSUPPORTED, "norm_rows: dtype %d", n.dtype);
+    if (n.n_rows <= 0) return ONELLM_OK;
+    const dim3 grid(n.n_rows), block(kNormThreads);
+    if (n.dtype == ONELLM_F32) {
+        if (n.add) ONELLM_CUDA(launch_pdl(norm_rows_kernel<float, true>, grid, block, 0, st, n));
+        else ONELLM_CUDA(launch_pdl(norm_rows_kernel<float, false>, grid, block, 0, st, n));
+    } else {
+        if (n.add) ONELLM_CUDA(launch_pdl(norm_rows_kernel<__nv_bfloat16, true>, grid, block, 0, st, n));
+        else ONELLM_CUDA(launch_pdl(norm_rows_kernel<__nv_bfloat16, false>, grid, block, 0, st, n));
+    }
     return ONELLM_OK;
 }
 }  // namespace onellm
@@ -268,9 +295,8 @@ extern "C" int onellm_add_residual_rmsnorm(int dtype, void* residual, void* deco
     return ONELLM_OK;
 }
 
-extern "C" int onellm_norm_pair(int dtype, const float* x, const int* rows, int n_rows, const float* w1, const float* w2, void* out1,
-                                void* out2, float eps, int width, int ld, void* stream)
+extern "C" int onellm_norm_rows_run(const onellm_norm_rows* n, void* stream)
 {
-    ONELLM_REQUIRE(dtype == ONELLM_BF16 || dtype == ONELLM_F32, ONELLM_ERR_UNSUPPORTED, "norm_pair: dtype %d", dtype);
-    return norm_pair(dtype, x, rows, n_rows, w1, w2, out1, out2, eps, width, ld, reinterpret_cast<cudaStream_t>(stream));
+    ONELLM_REQUIRE(n, ONELLM_ERR_ARG, "norm_rows: null pointer");
+    return norm_rows(*n, reinterpret_cast<cudaStream_t>(stream));
 }

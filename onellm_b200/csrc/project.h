@@ -4,20 +4,11 @@
 
 namespace onellm {
 
-//   y[M,N] = x[M,K] . W                        W, W2 [K,N] of element type dtype (ONELLM_BF16 or ONELLM_F32)
-//   y      = act(x . W) * (x . W2)             W2 given
-//   y      = resid + x . W                     resid given (float, row stride ldy; may be y; with f32 or dtype F32)
-// f32: y is float although x and W are bfloat16.  ldy 0: N.  bfloat16: K % 16 == 0, N and ldy % 8 == 0.
-struct Projection {
-    int dtype;
-    const void *x, *W, *W2;
-    void* y;
-    long ldy;
-    int M, N, K;
-    int act;  // GateAct
-    int f32;
-    const float* resid;
+using RowGroups = onellm_row_groups;
+// The parameters are described in onellm_b200.h; everything not set is zero, the scale of the product one.
+struct Projection : onellm_projection {
+    Projection() : onellm_projection() { scale = 1.f; }
 };
-int project(const Projection& p, cudaStream_t st);
+int project(const onellm_projection& p, cudaStream_t st);
 
 }  // namespace onellm

@@ -23,6 +23,9 @@ constexpr int kRedLd = kBN + 1;   // row stride of the partial tile in shared me
 //   act:   gate function of the two-weight form.
 //   ldy:   row stride of y (and of resid); 0: N.
 //   f32:   y and resid are float instead of the element type (a residual stream or logits kept in 32 bits).
+//   scale: with f32, factor on the result in front of the residual.
+//   limit: bound of the clamped gate function.
+//   row_scale: factor of a token on the products, in front of the gate function.
 struct EpilogueArgs {
     const void* resid;  // [M, N] or NULL
     const void* bias;   // [N] or NULL
@@ -33,6 +36,8 @@ struct EpilogueArgs {
     int act;
     long ldy;
     int f32;
+    float scale = 1.f, limit = 0.f;
+    const float* row_scale = nullptr;
 };
 
 // `red` holds this block's partial tile as [NW][MP][kRedLd] floats followed by MP partial sums of squares (used
@@ -99,8 +104,15 @@ __device__ __forceinline__ void splitk_epilogue(float* red, cg::cluster_group& c
             s1.x *= inv;
             s1.y *= inv;
         }
-        v0 = DUAL ? gate_act(s0.x, ep.act) * s1.x : s0.x;
-        v1 = DUAL ? gate_act(s0.y, ep.act) * s1.y : s0.y;
+        if (!FUSED && ep.row_scale) {
+            const float rs = ep.row_scale[tok];
+            s0.x *= rs;
+            s0.y *= rs;
+            s1.x *= rs;
+            s1.y *= rs;
+        }
+        v0 = DUAL ? gate_pair(s0.x, s1.x, ep.act, ep.limit) : s0.x;
+        v1 = DUAL ? gate_pair(s0.y, s1.y, ep.act, ep.limit) : s0.y;
         w0 = s1.x;  // WIDE: the same pair 128 columns further
         w1 = s1.y;
         return true;
@@ -145,8 +157,8 @@ __device__ __forceinline__ void splitk_epilogue(float* red, cg::cluster_group& c
         if (!FUSED && ep.f32) {
             if (ep.resid) {
                 const float2 rr = *reinterpret_cast<const float2*>(static_cast<const float*>(ep.resid) + at);
-                v0 += rr.x;
-                v1 += rr.y;
+                v0 = fmaf(v0, ep.scale, rr.x);
+                v1 = fmaf(v1, ep.scale, rr.y);
             }
             *reinterpret_cast<float2*>(reinterpret_cast<float*>(y) + at) = make_float2(v0, v1);
             return 0u;

@@ -86,30 +86,51 @@ skinny_nk_kernel(const __half* __restrict__ x, const __half* __restrict__ W, __h
 
 // Plain fp32 projection for the reference's own dtype: 64x64 tiles, 16x16 threads, 4x4 outputs
 // per thread.  Correctness path for fp32 callers, not a tuned kernel.
-// resid (row stride ldy, may be y): y = resid + result.  gate >= 0: y holds the gate product of a gated pair and becomes
-// act(y) * result.
-template <bool W_NK>
+// resid (row stride ldy, may be y): y = resid + scale * result.  gate >= 0: y holds the gate product of a gated pair and
+// becomes gate_pair(y, result).  GROUPED: blockIdx.z is a group of rows with a weight of its own (onellm_row_groups).
+template <bool W_NK, bool GROUPED = false>
 __global__ void __launch_bounds__(256)
-sgemm_kernel(const float* __restrict__ x, const float* __restrict__ W, float* y, int M, int N, int K, long ldy, const float* resid, int gate)
+sgemm_kernel(const float* __restrict__ x, const float* __restrict__ W, float* y, int M, int N, int K, long ldx, int ldw, long ldy, const float* resid,
+             float scale, int gate, float limit, const RowGroups grp)
 {
     __shared__ float xs[16][64 + 1];
     __shared__ float ws[16][64 + 1];
     pdl_wait();
+    int r0 = 0;
+    if constexpr (GROUPED) {
+        int g = blockIdx.z;
+        if (grp.off) {
+            if (grp.n_used && g >= *grp.n_used) return;
+            if (grp.used) g = grp.used[g];
+            r0 = grp.off[g];
+            M = grp.off[g + 1] - r0;
+        }
+        if ((int)blockIdx.y * 64 >= M) return;
+        W += (size_t)g * grp.w_stride;
+        x += (size_t)g * grp.x_stride;
+        y += (size_t)g * grp.y_stride + (size_t)r0 * ldy;
+    }
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
     const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64;
     float acc[4][4] = {};
     for (int k0 = 0; k0 < K; k0 += 16) {
         for (int i = threadIdx.x; i < 16 * 64; i += 256) {
             const int kk = i & 15, mm = i >> 4;
-            xs[kk][mm] = (m0 + mm < M && k0 + kk < K) ? x[(size_t)(m0 + mm) * K + k0 + kk] : 0.f;
+            float v = 0.f;
+            if (m0 + mm < M && k0 + kk < K) {
+                size_t row = r0 + m0 + mm;
+                if (GROUPED && grp.off && grp.x_rows) row = grp.x_rows[row];
+                v = x[row * ldx + k0 + kk];
+            }
+            xs[kk][mm] = v;
         }
         for (int i = threadIdx.x; i < 16 * 64; i += 256) {
             if (W_NK) {
                 const int kk = i & 15, nn = i >> 4;
-                ws[kk][nn] = (n0 + nn < N && k0 + kk < K) ? W[(size_t)(n0 + nn) * K + k0 + kk] : 0.f;
+                ws[kk][nn] = (n0 + nn < N && k0 + kk < K) ? W[(size_t)(n0 + nn) * ldw + k0 + kk] : 0.f;
             } else {
                 const int nn = i & 63, kk = i >> 6;
-                ws[kk][nn] = (n0 + nn < N && k0 + kk < K) ? W[(size_t)(k0 + kk) * N + n0 + nn] : 0.f;
+                ws[kk][nn] = (n0 + nn < N && k0 + kk < K) ? W[(size_t)(k0 + kk) * ldw + n0 + nn] : 0.f;
             }
         }
         __syncthreads();
@@ -135,9 +156,9 @@ sgemm_kernel(const float* __restrict__ x, const float* __restrict__ W, float* y,
             if (m < M && n < N) {
                 const size_t at = (size_t)m * ldy + n;
                 float v = acc[i][j];
-                if (resid) v += resid[at];
-                if (gate == GATE_RELU) v *= fmaxf(y[at], 0.f);
-                else if (gate == GATE_SILU) v *= y[at] / (1.0f + expf(-y[at]));
+                if (GROUPED && grp.row_scale) v *= grp.row_scale[r0 + m];
+                if (resid) v = fmaf(v, scale, resid[at]);
+                if (gate >= 0) v = gate_pair<true>(y[at], v, gate, limit);
                 y[at] = v;
             }
         }
@@ -239,9 +260,9 @@ extern "C" int onellm_gemm_ld(int dtype, const void* x, const void* W, void* y, 
         ONELLM_REQUIRE(grid.y <= 65535, ONELLM_ERR_UNSUPPORTED, "gemm: M too large for the fp32 path");
         note_launch();
         if (w_layout == ONELLM_W_NK)
-            sgemm_kernel<true><<<grid, 256, 0, st>>>((const float*)x, (const float*)W, (float*)y, M, N, K, ldy, nullptr, -1);
+            sgemm_kernel<true><<<grid, 256, 0, st>>>((const float*)x, (const float*)W, (float*)y, M, N, K, K, K, ldy, nullptr, 1.f, -1, 0.f, RowGroups{});
         else
-            sgemm_kernel<false><<<grid, 256, 0, st>>>((const float*)x, (const float*)W, (float*)y, M, N, K, ldy, nullptr, -1);
+            sgemm_kernel<false><<<grid, 256, 0, st>>>((const float*)x, (const float*)W, (float*)y, M, N, K, K, N, ldy, nullptr, 1.f, -1, 0.f, RowGroups{});
         ONELLM_CHECK_LAUNCH();
         return ONELLM_OK;
     }
@@ -268,35 +289,69 @@ template <typename T>
 cudaError_t skinny_kn_project(const T* x, const T* W0, const T* W1, T* y, int M, int N, int K, const EpilogueArgs& ep, cudaStream_t st);
 extern template cudaError_t skinny_kn_project<__nv_bfloat16>(const __nv_bfloat16*, const __nv_bfloat16*, const __nv_bfloat16*,
                                                              __nv_bfloat16*, int, int, int, const EpilogueArgs&, cudaStream_t);
-int gemm_bf16_large(const __nv_bfloat16* x, const __nv_bfloat16* W, const __nv_bfloat16* W2, void* y, long ldy, int M, int N, int K, int act,
-                    int f32, const float* resid, cudaStream_t st);
+cudaError_t skinny_kn_grouped(const onellm_projection& p, cudaStream_t st);
+int gemm_bf16_large(const onellm_projection& p, cudaStream_t st);
 
-int project(const Projection& p, cudaStream_t st)
+static int project_f32(const onellm_projection& p, long ldy, cudaStream_t st)
+{
+    const RowGroups none = {};
+    const RowGroups& g = p.groups ? *p.groups : none;
+    const dim3 grid((p.N + 63) / 64, (p.M + 63) / 64, p.groups ? g.n : 1);
+    ONELLM_REQUIRE(grid.y <= 65535 && grid.z <= 65535, ONELLM_ERR_UNSUPPORTED, "project: too many rows for the fp32 path");
+    const long ldx = p.ldx ? p.ldx : p.K;
+    const int ldw = p.ldw ? p.ldw : p.N;
+    auto run = [&](const void* W, const float* resid, int gate) {
+        if (p.groups)
+            return launch_pdl(sgemm_kernel<false, true>, grid, dim3(256), 0, st, (const float*)p.x, (const float*)W, (float*)p.y, p.M, p.N, p.K, ldx,
+                              ldw, ldy, resid, p.scale, gate, p.limit, g);
+        return launch_pdl(sgemm_kernel<false>, grid, dim3(256), 0, st, (const float*)p.x, (const float*)W, (float*)p.y, p.M, p.N, p.K, ldx, ldw, ldy,
+                          resid, p.scale, gate, p.limit, g);
+    };
+    ONELLM_CUDA(run(p.W, p.W2 ? nullptr : p.resid, -1));
+    if (p.W2) ONELLM_CUDA(run(p.W2, nullptr, p.act));
+    return ONELLM_OK;
+}
+
+int project(const onellm_projection& p, cudaStream_t st)
 {
     ONELLM_REQUIRE(p.x && p.W && p.y && p.N > 0 && p.K > 0 && p.M >= 0, ONELLM_ERR_ARG, "project: bad argument");
+    ONELLM_REQUIRE(!p.resid || p.f32 || p.dtype == ONELLM_F32, ONELLM_ERR_ARG, "project: a residual needs a float output");
+    ONELLM_REQUIRE(p.groups ? p.groups->n > 0 && !p.resid : !p.ldx && !p.ldw, ONELLM_ERR_ARG, "project: strides and groups");
     const long ldy = p.ldy ? p.ldy : p.N;
     if (p.M == 0) return ONELLM_OK;
-    if (p.dtype == ONELLM_F32) {
-        const dim3 grid((p.N + 63) / 64, (p.M + 63) / 64);
-        ONELLM_REQUIRE(grid.y <= 65535, ONELLM_ERR_UNSUPPORTED, "project: too many rows for the fp32 path");
-        ONELLM_CUDA(launch_pdl(sgemm_kernel<false>, grid, dim3(256), 0, st, (const float*)p.x, (const float*)p.W, (float*)p.y, p.M, p.N, p.K,
-                               ldy, p.W2 ? nullptr : p.resid, -1));
-        if (p.W2)
-            ONELLM_CUDA(launch_pdl(sgemm_kernel<false>, grid, dim3(256), 0, st, (const float*)p.x, (const float*)p.W2, (float*)p.y, p.M, p.N,
-                                   p.K, ldy, (const float*)nullptr, p.act));
-        return ONELLM_OK;
-    }
+    if (p.dtype == ONELLM_F32) return project_f32(p, ldy, st);
     ONELLM_REQUIRE(p.dtype == ONELLM_BF16, ONELLM_ERR_UNSUPPORTED, "project: dtype %d", p.dtype);
-    ONELLM_REQUIRE(p.K % 16 == 0 && p.N % 8 == 0 && ldy % 8 == 0, ONELLM_ERR_UNSUPPORTED, "project: need K %% 16 == 0, N and ldy %% 8 == 0");
+    ONELLM_REQUIRE(p.K % 16 == 0 && p.N % 8 == 0 && ldy % 8 == 0 && p.ldx % 8 == 0 && p.ldw % 8 == 0, ONELLM_ERR_UNSUPPORTED,
+                   "project: need K %% 16 == 0, N and the strides %% 8 == 0");
     ONELLM_REQUIRE(aligned16(p.x) && aligned16(p.W) && aligned16(p.W2) && aligned16(p.y) && aligned16(p.resid), ONELLM_ERR_ARG,
                    "project: pointers must be 16-byte aligned");
     typedef __nv_bfloat16 bf16;
-    if (p.M > 64)
-        return gemm_bf16_large((const bf16*)p.x, (const bf16*)p.W, (const bf16*)p.W2, p.y, ldy, p.M, p.N, p.K, p.act, p.f32, p.resid, st);
+    if (p.groups) {
+        const RowGroups& g = *p.groups;
+        ONELLM_REQUIRE(g.n <= 65535 && g.w_stride % 8 == 0 && g.x_stride % 8 == 0 && g.y_stride % 8 == 0 && !p.f32, ONELLM_ERR_UNSUPPORTED,
+                       "project: at most 65535 groups, strides %% 8 == 0, output in the element type");
+        if (p.M <= 64) {
+            ONELLM_CUDA(skinny_kn_grouped(p, st));
+            return ONELLM_OK;
+        }
+        if (g.off) return gemm_bf16_large(p, st);
+        // every group takes all rows: 64 at a time
+        for (int m = 0; m < p.M; m += 64) {
+            onellm_projection part = p;
+            part.M = p.M - m < 64 ? p.M - m : 64;
+            part.x = static_cast<const bf16*>(p.x) + (size_t)m * (p.ldx ? p.ldx : p.K);
+            part.y = static_cast<bf16*>(p.y) + (size_t)m * ldy;
+            ONELLM_CUDA(skinny_kn_grouped(part, st));
+        }
+        return ONELLM_OK;
+    }
+    if (p.M > 64) return gemm_bf16_large(p, st);
     EpilogueArgs ep = {};
     ep.resid = p.resid;
     ep.early_dependents = 1;
     ep.act = p.act;
+    ep.limit = p.limit;
+    ep.scale = p.scale;
     ep.ldy = ldy;
     ep.f32 = p.f32;
     ONELLM_CUDA(skinny_kn_project<bf16>((const bf16*)p.x, (const bf16*)p.W, (const bf16*)p.W2, (bf16*)p.y, p.M, p.N, p.K, ep, st));
@@ -385,10 +440,8 @@ extern "C" int onellm_gemm_swiglu(int dtype, const void* x, const void* Wg, cons
     return ONELLM_OK;
 }
 
-extern "C" int onellm_project(int dtype, const void* x, const void* W, const void* W2, void* y, long ldy, int M, int N, int K, int act, int f32,
-                              const float* resid, void* stream)
+extern "C" int onellm_project(const onellm_projection* p, void* stream)
 {
-    ONELLM_REQUIRE(!resid || f32 || dtype == ONELLM_F32, ONELLM_ERR_ARG, "project: a residual needs a float output");
-    const Projection p = {dtype, x, W, W2, y, ldy, M, N, K, act, f32, resid};
-    return project(p, reinterpret_cast<cudaStream_t>(stream));
+    ONELLM_REQUIRE(p, ONELLM_ERR_ARG, "project: null pointer");
+    return project(*p, reinterpret_cast<cudaStream_t>(stream));
 }

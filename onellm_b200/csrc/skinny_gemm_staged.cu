@@ -26,6 +26,7 @@
 #include <tuple>
 #include <utility>
 
+#include "project.h"
 #include "skinny_common.cuh"
 
 namespace onellm {
@@ -60,12 +61,21 @@ struct FusedNormArgs {
     float eps;
 };
 
-template <typename T, int MB, bool DUAL, bool FUSED>
+// GROUPED: blockIdx.z is a group of rows with a weight of its own (onellm_row_groups: the experts of a mixture, the heads of
+// a per-head projection); M is the most rows a group has, and the 8-token rows behind a group's last one are skipped.
+struct GroupArgs {
+    RowGroups g;
+    int ldw;   // row stride of a weight
+    long ldx;  // row stride of x
+};
+
+template <typename T, int MB, bool DUAL, bool FUSED, bool GROUPED = false>
 __global__ void __launch_bounds__(kStThreads)
 skinny_kn_staged_kernel(const T* __restrict__ x, const T* __restrict__ W0, const T* __restrict__ W1,
                         T* y, int M, int N, int K, int stages_per_block, int nst,
-                        const FusedNormArgs<T> fn, const EpilogueArgs ep)
+                        const FusedNormArgs<T> fn, EpilogueArgs ep, const GroupArgs ga)
 {
+    static_assert(!(FUSED && GROUPED), "groups take their rows as they are");
     constexpr int NW = DUAL ? 2 : 1;
     constexpr int MP = 8 * MB;
     // a stage holds the weights and (not FUSED) the activations of the same 32 rows
@@ -80,6 +90,27 @@ skinny_kn_staged_kernel(const T* __restrict__ x, const T* __restrict__ W0, const
     const int k_end = min(k_begin + stages_per_block * kKC, K);
     const int n_stages = k_end > k_begin ? (k_end - k_begin + kKC - 1) / kKC : 0;
     const uint32_t smem_base = (uint32_t)__cvta_generic_to_shared(smem);
+    const int ldw = GROUPED ? ga.ldw : N;
+    const T* x_row = nullptr;  // GROUPED: the row this thread copies
+    if constexpr (GROUPED) {
+        int g = blockIdx.z, r0 = 0;
+        if (ga.g.off) {  // which rows and weights: known once the routing in front of this kernel is done
+            if (ep.early_dependents) pdl_launch_dependents();
+            pdl_wait();
+            if (ga.g.n_used && g >= *ga.g.n_used) return;  // all blocks of the cluster
+            if (ga.g.used) g = ga.g.used[g];
+            r0 = ga.g.off[g];
+            M = min(ga.g.off[g + 1] - r0, MP);
+            if (M <= 0) return;
+        }
+        const int i = r0 + min(tid >> 2, M - 1);
+        x_row = x + (size_t)(ga.g.off && ga.g.x_rows ? ga.g.x_rows[i] : i) * ga.ldx + (size_t)g * ga.g.x_stride;
+        W0 += (size_t)g * ga.g.w_stride;
+        if (DUAL) W1 += (size_t)g * ga.g.w_stride;
+        y += (size_t)g * ga.g.y_stride + (size_t)r0 * (ep.ldy ? ep.ldy : N);
+        ep.row_scale = ga.g.row_scale ? ga.g.row_scale + r0 : nullptr;
+    }
+    const int mb_used = GROUPED ? (M + 7) / 8 : MB;
 
     // Copy assignments, fixed for the whole kernel: chunk c = tid + 256*i is row c/16 of the stage,
     // 16-byte column c%16.  Source pointers advance by 32 rows per stage; destinations are offsets
@@ -96,15 +127,15 @@ skinny_kn_staged_kernel(const T* __restrict__ x, const T* __restrict__ W0, const
         wrow[i] = row;
         wcol_ok[i] = col < N;
         wdst[i] = row * (kBN * 2) + ((c16 ^ (row & 7)) << 4);
-        const size_t off = (size_t)(k_begin + row) * N + (wcol_ok[i] ? col : 0);
+        const size_t off = (size_t)(k_begin + row) * ldw + (wcol_ok[i] ? col : 0);
         wsrc[0][i] = W0 + off;
         if (DUAL) wsrc[NW - 1][i] = W1 + off;
     }
-    const size_t wstep = (size_t)kKC * N;
+    const size_t wstep = (size_t)kKC * ldw;
     // activations: thread tid < 4*MP copies 16 bytes of row tid/4
     const bool x_thread = !FUSED && tid < MP * 4;
     const int x_part = tid & 3;
-    const T* xsrc = FUSED ? x : x + (size_t)min(tid >> 2, M - 1) * K + k_begin + x_part * 8;
+    const T* xsrc = FUSED ? x : (GROUPED ? x_row : x + (size_t)min(tid >> 2, M - 1) * K) + k_begin + x_part * 8;
     const uint32_t xdst = NW * kStageBytes + (tid >> 2) * kXRowBytes + x_part * 16;
 
     int w_issued = 0, x_issued = 0;  // stages whose copies have been issued
@@ -269,6 +300,7 @@ skinny_kn_staged_kernel(const T* __restrict__ x, const T* __restrict__ W0, const
             uint32_t xb[MB][2];
 #pragma unroll
             for (int mb = 0; mb < MB; mb++) {
+                if (GROUPED && mb >= mb_used) break;
                 const unsigned char* p = xs + 8 * mb * x_row_bytes + 32 * kk;
                 xb[mb][0] = *reinterpret_cast<const uint32_t*>(p);
                 xb[mb][1] = *reinterpret_cast<const uint32_t*>(p + 16);
@@ -289,7 +321,10 @@ skinny_kn_staged_kernel(const T* __restrict__ x, const T* __restrict__ W0, const
                 // ldmatrix order is (n 0-7, k 0-7), (n 8-15, k 0-7), (n 0-7, k 8-15), (n 8-15, k 8-15)
                 // = a0, a1, a2, a3 of the mma "row" operand
 #pragma unroll
-                for (int mb = 0; mb < MB; mb++) mma_16b<T>(acc[w][mb], a[0], a[1], a[2], a[3], xb[mb][0], xb[mb][1]);
+                for (int mb = 0; mb < MB; mb++) {
+                    if (GROUPED && mb >= mb_used) break;
+                    mma_16b<T>(acc[w][mb], a[0], a[1], a[2], a[3], xb[mb][0], xb[mb][1]);
+                }
             }
         }
     }
@@ -511,7 +546,72 @@ static cudaError_t launch_staged(const T* x, const T* W0, const T* W1, T* y, int
     cfg.attrs = attr;
     cfg.numAttrs = 2;
     note_launch();
-    return cudaLaunchKernelEx(&cfg, kern, x, W0, W1, y, M, N, K, plan.per_block, plan.nst, fn, ep);
+    return cudaLaunchKernelEx(&cfg, kern, x, W0, W1, y, M, N, K, plan.per_block, plan.nst, fn, ep, GroupArgs{});
+}
+
+// Row groups: two blocks per SM, K split while that leaves whole waves of them to fill.
+template <int MB, bool DUAL>
+static cudaError_t launch_grouped(const onellm_projection& p, const EpilogueArgs& ep, const GroupArgs& ga, cudaStream_t st)
+{
+    typedef __nv_bfloat16 T;
+    auto kern = skinny_kn_staged_kernel<T, MB, DUAL, false, true>;
+    constexpr int NW = DUAL ? 2 : 1;
+    constexpr size_t stage = (size_t)NW * kStageBytes + 8 * MB * kXRowBytes;
+    constexpr size_t red = ((size_t)NW * 8 * MB * kRedLd + 8 * MB) * sizeof(float);
+    constexpr size_t cap = 110 * 1024, most = cap > red ? cap : red;
+    static DeviceOnce attr;
+    const cudaError_t e = attr.run([kern] {
+        const cudaError_t r = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)most);
+        return r != cudaSuccess ? r : prefer_max_shared((const void*)kern);
+    });
+    if (e != cudaSuccess) return e;
+    const int cols = (p.N + kBN - 1) / kBN, total = (p.K + kKC - 1) / kKC;
+    const long blocks = (long)cols * ga.g.n;
+    int ks = 1;
+    while (ks < 8 && blocks * (ks + 1) <= 2L * num_sms() && (total + ks) / (ks + 1) >= 4) ks++;
+    int per = (total + ks - 1) / ks;
+    while (ks > 1 && per * (ks - 1) >= total) per = (total + --ks - 1) / ks;
+    const int nst = std::max(3, std::min({12, per + 1, (int)(cap / stage)}));
+    cudaLaunchConfig_t cfg = {};
+    cudaLaunchAttribute at[2];
+    at[0].id = cudaLaunchAttributeClusterDimension;
+    at[0].val.clusterDim.x = 1;
+    at[0].val.clusterDim.y = ks;
+    at[0].val.clusterDim.z = 1;
+    at[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    at[1].val.programmaticStreamSerializationAllowed = 1;
+    cfg.gridDim = dim3(cols, ks, ga.g.n);
+    cfg.blockDim = dim3(kStThreads);
+    cfg.dynamicSmemBytes = std::max(stage * nst, red);
+    cfg.stream = st;
+    cfg.attrs = at;
+    cfg.numAttrs = 2;
+    note_launch();
+    return cudaLaunchKernelEx(&cfg, kern, (const T*)p.x, (const T*)p.W, (const T*)p.W2, (T*)p.y, p.M, p.N, p.K, per, nst, FusedNormArgs<T>{}, ep, ga);
+}
+
+// At most 64 rows per group, bfloat16.  Called from skinny_gemm.cu.
+cudaError_t skinny_kn_grouped(const onellm_projection& p, cudaStream_t st)
+{
+    EpilogueArgs ep = {};
+    ep.resid = p.resid;
+    ep.early_dependents = 1;
+    ep.act = p.act;
+    ep.limit = p.limit;
+    ep.scale = p.scale;
+    ep.ldy = p.ldy;
+    ep.f32 = p.f32;
+    const GroupArgs ga = {*p.groups, p.ldw ? p.ldw : p.N, p.ldx ? p.ldx : p.K};
+    if (p.W2) {
+        if (p.M <= 8) return launch_grouped<1, true>(p, ep, ga, st);
+        if (p.M <= 16) return launch_grouped<2, true>(p, ep, ga, st);
+        if (p.M <= 32) return launch_grouped<4, true>(p, ep, ga, st);
+        return launch_grouped<8, true>(p, ep, ga, st);
+    }
+    if (p.M <= 8) return launch_grouped<1, false>(p, ep, ga, st);
+    if (p.M <= 16) return launch_grouped<2, false>(p, ep, ga, st);
+    if (p.M <= 32) return launch_grouped<4, false>(p, ep, ga, st);
+    return launch_grouped<8, false>(p, ep, ga, st);
 }
 
 template <int MB>

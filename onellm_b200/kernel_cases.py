@@ -109,8 +109,8 @@ def make_mechanism_case(name, torch, m, B, ctx, plain=False) -> Case:
         rows = 4096
         xs = [torch.randn(rows, W, **f32) for _ in range(4)]
         w1, w2, o1, o2 = torch.zeros(W, **f32), torch.zeros(W, **f32), torch.empty(rows, W, **bf), torch.empty(rows, W, **bf)
-        fn = lambda i: ob.norm_pair(BF, xs[i], None, rows, w1, w2, o1, o2, 1e-6, W, W)
-        return Case(fn, 4, rows * W * 8, "B", "norm_pair_kernel", keep=(xs, w1, w2, o1, o2))
+        fn = lambda i: ob.norm_rows(BF, xs[i], None, rows, w1, w2, o1, o2, 1e-6, W, W, w_base=1.0)
+        return Case(fn, 4, rows * W * 8, "B", "norm_rows_kernel", keep=(xs, w1, w2, o1, o2))
     mix, cat = torch.randn(T, n_mix, **bf), torch.zeros(T, n_cat, **bf)
     cu = torch.arange(0, B + 1, device="cuda", dtype=torch.int32) * ctx
     hist, off = torch.zeros(B, device="cuda", dtype=torch.int32), torch.zeros(B, device="cuda", dtype=torch.int32)

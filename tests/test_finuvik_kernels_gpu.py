@@ -50,7 +50,7 @@ def rounded(a, kind):
 
 @pytest.mark.parametrize("kind", ["f32", "bf16"])
 @pytest.mark.parametrize("width,ld", [(88, 96), (1024, 1024), (9000, 9008)])
-def test_norm_pair(cuda, ob, kind, width, ld):
+def test_two_zero_centred_norms(cuda, ob, kind, width, ld):
     d = Dev(cuda, ob, kind)
     rng = np.random.default_rng(0)
     x = np.zeros((5, ld), np.float32)
@@ -59,7 +59,7 @@ def test_norm_pair(cuda, ob, kind, width, ld):
     w[:, :width] = 0.5 * rng.standard_normal((2, width))
     rows = [3, 0, 4, 2]
     o1, o2 = d.zeros(4, ld), d.zeros(4, ld)
-    ob.norm_pair(d.dtype, d.f32(x), d.i32(rows), 4, d.f32(w[0]), d.f32(w[1]), o1, o2, 1e-5, width, ld)
+    ob.norm_rows(d.dtype, d.f32(x), d.i32(rows), 4, d.f32(w[0]), d.f32(w[1]), o1, o2, 1e-5, width, ld, w_base=1.0)
     for o, wi in ((o1, w[0]), (o2, w[1])):
         ref = fr.zero_centred_rms_norm(x[rows, :width].astype(np.float64), wi[:width], 1e-5)
         assert rel_err(host(o)[:, :width], ref) < TOL[kind]
