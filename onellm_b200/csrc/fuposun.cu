@@ -103,7 +103,8 @@ static int read_feed_forward(const Json& m, const std::string& where, FuposunLay
     RC(json_object(m, "shared", w, &shared));
     RC(json_int(*shared, "ff", (where + ".shared").c_str(), &l->shared));
     RC(json_float(*shared, "limit", (where + ".shared").c_str(), &l->shared_limit));
-    ONELLM_REQUIRE(l->experts > 0 && l->top > 0 && l->top <= l->experts && l->eff > 0 && l->shared > 0, ONELLM_ERR_IO, "config: sizes of %s", w);
+    ONELLM_REQUIRE(l->experts > 0 && l->top > 0 && l->top <= l->experts && l->eff > 0 && l->shared > 0 && l->limit >= 0.0 && l->shared_limit >= 0.0,
+                   ONELLM_ERR_IO, "config: sizes of %s", w);
     ONELLM_REQUIRE(l->experts <= 1024 && l->top <= 64, ONELLM_ERR_UNSUPPORTED, "config: %s: at most 64 of 1024 experts", w);
     return ONELLM_OK;
 }

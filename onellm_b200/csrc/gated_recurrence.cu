@@ -3,12 +3,13 @@
 //   TIED (HGRN2): what a channel forgets of its state is the share it takes of the new value.  With g = 1 - f
 //         s <- s + g (v - s)
 //     which needs one multiply-add and keeps the digits of a gate near one (g comes from the complementary sigmoid).
-//   KEYED (gated linear attention): the new value comes in through a key of its own,
-//         s <- f s + k v
-//     and the gate's logit through a low-rank projection, whose second matrix is applied in float here.
+//   KEYED (gated linear attention): the new value comes in through a key of its own.  With g = f - 1
+//         s <- s + k v + g s
+//     which keeps the digits of a gate near one as well; the gate's logit comes through a low-rank projection, whose
+//     second matrix is applied in float here.
 //
 // Context pass, three launches:
-//   1. the prepare kernel turns the projections into the vectors of the recurrence (g and silu(q); or f, k and q), in
+//   1. the prepare kernel turns the projections into the vectors of the recurrence (g and silu(q); or g, k and q), in
 //      float and head by head, so that the tokens of a head lie behind each other.
 //   2. gated_recurrence_scan_kernel.  A thread block owns 32 value columns of one (sequence, head) and keeps that part of
 //      the state, dk x 32 floats, in registers over all tokens of the call: columns of the state never meet, only the dk
@@ -56,12 +57,6 @@ __device__ __forceinline__ f32x2 fma_f2(f32x2 a, f32x2 b, f32x2 c)
     asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
     return r;
 }
-__device__ __forceinline__ f32x2 mul_f2(f32x2 a, f32x2 b)
-{
-    f32x2 r;
-    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
-    return r;
-}
 __device__ __forceinline__ f32x2 sub_f2(f32x2 a, f32x2 b)
 {
     f32x2 r;
@@ -103,15 +98,15 @@ __device__ __forceinline__ void gate(float q, float z, float zb, float lower, fl
     qs = q * s;
 }
 
-// sigmoid(z) ^ inv_tau from the logarithm of the sigmoid
-__device__ __forceinline__ float decay(float z, float inv_tau) { return expf(inv_tau * (fminf(z, 0.f) - log1pf(expf(-fabsf(z))))); }
+// sigmoid(z) ^ inv_tau - 1 from the logarithm of the sigmoid
+__device__ __forceinline__ float decay(float z, float inv_tau) { return expm1f(inv_tau * (fminf(z, 0.f) - log1pf(expf(-fabsf(z))))); }
 
 struct GrParams {
     GatedRecurrence g;
     TokenPositions tp;
 };
 
-// Layout of the work space of T tokens: the vectors of a head [H][T][n * dkp] (TIED n = 2: g, silu(q); KEYED n = 3: f, q, k),
+// Layout of the work space of T tokens: the vectors of a head [H][T][n * dkp] (TIED n = 2: g, silu(q); KEYED n = 3: g, q, k),
 // v [H][dv / 32][T][32], outputs before the norm [T][H][dv]; all float, dkp = dk padded to the rows of a block.
 static int gr_dkp(int dk) { return dk <= 64 ? 64 : dk <= 128 ? 128 : dk <= 256 ? 256 : 512; }
 static int gr_vectors(int kind) { return kind == ONELLM_GR_KEYED ? 3 : 2; }
@@ -329,7 +324,7 @@ gated_recurrence_scan_kernel(const GrParams pp, int tokens, const float* __restr
                 for (int r = 0; r < R / 2; r++)
 #pragma unroll
                     for (int c = 0; c < 4; c++) {
-                        if constexpr (KEYED) S[r][c] = fma_f2(g2[r], S[r][c], mul_f2(k2[r], vv[c]));
+                        if constexpr (KEYED) S[r][c] = fma_f2(g2[r], S[r][c], fma_f2(k2[r], vv[c], S[r][c]));
                         else S[r][c] = fma_f2(g2[r], sub_f2(vv[c], S[r][c]), S[r][c]);
                         o2[c] = fma_f2(q2[r], S[r][c], o2[c]);
                     }
@@ -479,10 +474,10 @@ __global__ void __launch_bounds__(kGsThreads) gated_recurrence_step_kernel(const
                 const float g = sg[r], q = sq[r];
                 if constexpr (KEYED) {
                     const float k = sk[r];
-                    s[i].x = fmaf(g, s[i].x, k * v[0]);
-                    s[i].y = fmaf(g, s[i].y, k * v[1]);
-                    s[i].z = fmaf(g, s[i].z, k * v[2]);
-                    s[i].w = fmaf(g, s[i].w, k * v[3]);
+                    s[i].x = fmaf(g, s[i].x, fmaf(k, v[0], s[i].x));
+                    s[i].y = fmaf(g, s[i].y, fmaf(k, v[1], s[i].y));
+                    s[i].z = fmaf(g, s[i].z, fmaf(k, v[2], s[i].z));
+                    s[i].w = fmaf(g, s[i].w, fmaf(k, v[3], s[i].w));
                 } else {
                     s[i].x = fmaf(g, v[0] - s[i].x, s[i].x);
                     s[i].y = fmaf(g, v[1] - s[i].y, s[i].y);

@@ -100,6 +100,7 @@ class FuposunRef:
         self.reset()
 
     def reset(self):
+        self.margins = []  # per forward call and token: how close the closest choice of experts was, in logits
         self.pos = 0
         self.mem = [dict() for _ in self.c["layers"]]
 
@@ -131,6 +132,9 @@ class FuposunRef:
         if m["kind"] == "dense":
             return swiglu(h, *parts(""))
         r = m["router"]
+        if r["top"] < r["experts"]:
+            z = -np.sort(-(h @ w[p + "router"].T), 1)
+            self.margins[-1] = np.minimum(self.margins[-1], z[:, r["top"] - 1] - z[:, r["top"]])
         y = mixture(h, w[p + "router"], r["top"], [parts(f"e{n}.") for n in range(r["experts"])], m["expert"]["limit"])
         return y + expert(h, *parts("shared."), m["shared"]["limit"])
 
@@ -140,6 +144,7 @@ class FuposunRef:
         tokens = np.asarray(tokens)
         pos = self.pos + np.arange(len(tokens))
         self.pos += len(tokens)
+        self.margins.append(np.full(len(tokens), np.inf))
         x = plain_rms_norm(w["embed"][tokens], w["embed.norm"], eps)
         seen = []
         for i, layer in enumerate(self.c["layers"]):
