@@ -643,12 +643,15 @@ def run_ours(args, workload):
 
 
 # ---------------------------------------------------------------------------------------------
-# --design finuvik: the Finuvik design beside the LLaMA design at equal width, depth, heads and feed-forward
+# --design finuvik | fuposun: a further design beside the LLaMA design at equal width, depth, heads and feed-forward
 # ---------------------------------------------------------------------------------------------
 DESIGN_SIZES = {
-    # width, layers, heads, kv_heads, head size, ff, recurrence heads x (key, value), vocabulary
-    "w2048": dict(hidden=2048, num_layers=16, head_num=16, kv_head_num=4, head_size=128, inter_size=5632, rec=(16, 128, 128), vocab_size=32000),
-    "w4096": dict(hidden=4096, num_layers=8, head_num=32, kv_head_num=8, head_size=128, inter_size=11008, rec=(32, 128, 128), vocab_size=32000),
+    # width, layers, heads, kv_heads, head size, ff, recurrence heads x (key, value), vocabulary; window and latents of the
+    # latent attention, gla heads x (key, value), experts (of which `top` with ff / top columns each are the LLaMA feed-forward)
+    "w2048": dict(hidden=2048, num_layers=16, head_num=16, kv_head_num=4, head_size=128, inter_size=5632, rec=(16, 128, 128), vocab_size=32000,
+                  q_rank=1536, kv_rank=512, window=1024, gla=(4, 256, 512), experts=32, top=4),
+    "w4096": dict(hidden=4096, num_layers=8, head_num=32, kv_head_num=8, head_size=128, inter_size=11008, rec=(32, 128, 128), vocab_size=32000,
+                  q_rank=1536, kv_rank=512, window=1024, gla=(8, 256, 512), experts=32, top=4),
 }
 
 
@@ -663,6 +666,41 @@ def finuvik_config(s, max_positions):
             "norm": {"eps": 1e-6}, "layers": [layer] * s["num_layers"]}
 
 
+def fuposun_config(s, max_positions):
+    """Recurrent layers with a dense feed-forward and attention layers with experts in turn."""
+    D, (RH, RK, RV) = s["head_size"], s["gla"]
+    eff = s["inter_size"] // s["top"]
+    rec = {"type": "gla", "mixer": {"heads": RH, "dim": RK, "vdim": RV, "tau": 16.0}, "mlp": {"kind": "dense", "ff": s["inter_size"]}}
+    attn = {"type": "latent_attention",
+            "mixer": {"heads": s["head_num"], "dim": D, "vdim": D, "q_rank": s["q_rank"], "kv_rank": s["kv_rank"], "scale": D ** -0.5,
+                      "mask": {"size": s["window"]}},
+            "mlp": {"kind": "moe", "router": {"experts": s["experts"], "top": s["top"]}, "expert": {"ff": eff, "limit": 7.0},
+                    "shared": {"ff": eff, "limit": 7.0}}}
+    return {"architecture": "Fuposun", "vocab": s["vocab_size"], "width": s["hidden"], "norm": {"eps": 1e-6}, "residual_mult": 0.5,
+            "logit_softcap": 30.0, "layers": [rec, attn] * (s["num_layers"] // 2)}
+
+
+def design_weights(kind, s, tokens):
+    """(projection weights a token is multiplied with, weights that `tokens` tokens read at the least, state bytes of a
+    sequence, cached bytes of a sequence per visible position), all layers together; experts are chosen at random."""
+    W, L, H, G, D, I = (s[k] for k in ("hidden", "num_layers", "head_num", "kv_head_num", "head_size", "inter_size"))
+    llama = W * (H + 2 * G) * D + H * D * W + 3 * W * I
+    if kind == "llama":
+        return llama * L, llama * L, 0, L * 2 * G * D * 2
+    if kind == "finuvik":
+        RH, RK, RV = s["rec"]
+        w = llama + W * RH * (2 * RK + 2 * RV)
+        return w * L, w * L, L * RH * RK * RV * 8, L * 2 * G * D * 2
+    RH, RK, RV = s["gla"]
+    Q, K, E, top = s["q_rank"], s["kv_rank"], s["experts"], s["top"]
+    rec = W * RH * (2 * RK + 3 * RV) + 3 * W * I
+    attn = W * (Q + K) + Q * H * D + 2 * K * H * D + H * D * W + W * E
+    one = 3 * W * (I // top)
+    read = E * (1 - (1 - top / E) ** tokens)
+    half = L // 2
+    return half * (rec + attn + one * (top + 1)), half * (rec + attn + one * (read + 1)), half * RH * RK * RV * 8, half * K * 2
+
+
 def run_design(args):
     """Prefill and decode throughput of both designs and their like kernels side by side; one JSON line."""
     import torch
@@ -671,7 +709,8 @@ def run_design(args):
     torch.cuda.set_device(0)
     hbm_peak, tf_peak, peak_kind = peaks()
     smax = 4096
-    out = {"design": "finuvik", "beside": "llama", "data": "synthetic", "peak_kind": peak_kind, "hbm_gbs": hbm_peak, "bf16_tflops": tf_peak,
+    config = {"finuvik": finuvik_config, "fuposun": fuposun_config}[args.design]
+    out = {"design": args.design, "beside": "llama", "data": "synthetic", "peak_kind": peak_kind, "hbm_gbs": hbm_peak, "bf16_tflops": tf_peak,
            "models": {}, "kernels": {}}
 
     def timed(m, fn, n, warm):
@@ -689,11 +728,11 @@ def run_design(args):
         return float(np.median(ts))
 
     def open_design(kind, s, batch):
-        if kind == "finuvik":
-            m = ob.Model(finuvik_config(s, smax), ob.BF16, batch, smax)
-        else:
+        if kind == "llama":
             m = ob.Llama(max_seq_len=smax, max_batch=batch, **{k: s[k] for k in ("num_layers", "hidden", "head_num", "kv_head_num", "head_size",
                                                                                  "inter_size", "vocab_size")})
+        else:
+            m = ob.Model(config(s, smax), ob.BF16, batch, smax)
         m.init_random(seed=1, std=0.02)
         m.set_sampling(top_k=1)
         return m
@@ -703,21 +742,16 @@ def run_design(args):
         clk.wait_first(3.0)
         clk.mark_start()
         for size, s in DESIGN_SIZES.items():
-            W, L, H, G, D, I, V = (s[k] for k in ("hidden", "num_layers", "head_num", "kv_head_num", "head_size", "inter_size", "vocab_size"))
-            RH, RK, RV = s["rec"]
+            W, V = s["hidden"], s["vocab_size"]
             res = out["models"][size] = {"shape": {k: v for k, v in s.items()}}
-            for kind in ("llama", "finuvik"):
-                proj = W * (H + 2 * G) * D + H * D * W + 3 * W * I
-                state = 0
-                if kind == "finuvik":
-                    proj += W * RH * (2 * RK + 2 * RV)
-                    state = RH * RK * RV * 4 * 2
-                r = res[kind] = {"projection_weights": proj * L, "prefill": {}, "decode": {}}
+            for kind in ("llama", args.design):
+                proj = design_weights(kind, s, 1)[0]
+                r = res[kind] = {"projection_weights": proj, "prefill": {}, "decode": {}}
                 m = open_design(kind, s, 8)
                 for b, n in ((1, 2048), (8, 512)):
                     ids = rng.integers(0, V, (b, n)).astype(np.int32)
                     t = timed(m, lambda: m.prefill(ids), 5, 2)
-                    r["prefill"][f"{b}x{n}"] = {"tokens_per_s": b * n / t, "ms": t * 1e3, "projection_tflops": 2.0 * proj * L * b * n / t / 1e12}
+                    r["prefill"][f"{b}x{n}"] = {"tokens_per_s": b * n / t, "ms": t * 1e3, "projection_tflops": 2.0 * proj * b * n / t / 1e12}
                 m.close()
                 for b in (1, 8, 32):
                     m = open_design(kind, s, b)
@@ -727,29 +761,45 @@ def run_design(args):
                     def block():
                         for _ in range(16):
                             m.decode_step(None, None)
-                    m.seek(b, ctx, first)
-                    block()
-                    m.seek(b, ctx, first)
-                    t = timed(m, block, 5, 1) / 16
-                    nbytes = proj * L * 2 + V * W * 2 + L * b * (2 * (ctx + 64) * G * D * 2 + state)
+                    if kind == "fuposun":  # real states and latents, unlike tokens: what the router does depends on them
+                        m.prefill(rng.integers(0, V, (b, ctx)).astype(np.int32))
+                        warm = 3  # every step's tokens follow from the one before: go on from here
+                    else:
+                        m.seek(b, ctx, first)
+                        block()
+                        m.seek(b, ctx, first)
+                        warm = 1
+                    t = timed(m, block, 5, warm) / 16
+                    _, read, state, per_pos = design_weights(kind, s, b)
+                    span = min(ctx + 64, s["window"]) if kind == "fuposun" else ctx + 64
+                    nbytes = read * 2 + V * W * 2 + b * (span * per_pos + state)
                     r["decode"][f"b{b}_ctx{ctx}"] = {"tokens_per_s": b / t, "ms_per_step": t * 1e3, "bytes_per_step": nbytes,
                                                      "frac_of_hbm": nbytes / t / 1e9 / hbm_peak}
                     m.close()
                 torch.cuda.empty_cache()
-        pairs = [("fv_mix", "qkv"), ("fv_gate_up", "gate_up"), ("fv_out", "down"), ("fv_attn", "attn"), ("fv_rec", "attn"), ("fv_norm", "norm"),
-                 ("prefill_fv_mix", "prefill_qkv"), ("prefill_fv_gate", "prefill_gate"), ("prefill_fv_out", "prefill_down"),
-                 ("prefill_fv_attn", "prefill_attn"), ("prefill_fv_rec", None)]
-        fp32_peak = 148 * 128 * 2 * 1.965e9 / 1e12  # nominal: the recurrence runs on the fp32 pipes
+        if args.design == "finuvik":
+            pairs = [("fv_mix", "qkv"), ("fv_gate_up", "gate_up"), ("fv_out", "down"), ("fv_attn", "attn"), ("fv_rec", "attn"), ("fv_norm", "norm"),
+                     ("prefill_fv_mix", "prefill_qkv"), ("prefill_fv_gate", "prefill_gate"), ("prefill_fv_out", "prefill_down"),
+                     ("prefill_fv_attn", "prefill_attn"), ("prefill_fv_rec", None)]
+        else:
+            pairs = [("fu_in", "qkv"), ("fu_uq", "o_proj"), ("fu_absorb", "o_proj"), ("fu_uv", "o_proj"), ("fu_out", "o_proj"), ("fu_egate", "gate_up"),
+                     ("fu_edown", "down"), ("fu_route", None), ("fu_attn", "attn"), ("fu_rec", "fv_rec"), ("fu_norm", "fv_norm"),
+                     ("prefill_fu_in", "prefill_qkv"), ("prefill_fu_kv", "prefill_qkv"), ("prefill_fu_egate", "prefill_gate"),
+                     ("prefill_fu_edown", "prefill_down"), ("prefill_fu_route", None), ("prefill_fu_attn", "prefill_attn"),
+                     ("prefill_fu_rec", "prefill_fv_rec")]
+        fp32_peak = 148 * 128 * 2 * 1.965e9 / 1e12  # nominal: the recurrences run on the fp32 pipes
         done = {}
         for mine, like in pairs:
             for name in (mine, like):
                 if name is None or name in done:
                     continue
                 prefill = name.startswith("prefill_")
-                for b, ctx in (((1, 2048), (8, 512)) if prefill else ((8, 2040), (32, 2040)) if name in ("fv_attn", "attn", "fv_rec") else ((8, 2040),)):
+                decode = ((8, 2040), (32, 2040)) if name in ("fv_attn", "attn", "fv_rec", "fu_rec") else \
+                    ((8, 1024), (32, 1024), (32, 4096)) if name == "fu_attn" else ((8, 2040),)
+                for b, ctx in ((1, 2048), (8, 512)) if prefill else decode:
                     case = kc.make_case(name, torch, "7b", b, ctx, 1)
                     t = kc.time_case(case, torch, iters=20, warm=5, graph=not prefill)
-                    peak = fp32_peak * 1e12 if name == "prefill_fv_rec" else tf_peak * 1e12 if case.unit == "flop" else hbm_peak * 1e9
+                    peak = fp32_peak * 1e12 if name in ("prefill_fv_rec", "prefill_fu_rec") else tf_peak * 1e12 if case.unit == "flop" else hbm_peak * 1e9
                     done[name] = True
                     out["kernels"][f"{name}_b{b}_{ctx}"] = {"us": t * 1e6, "amount": case.amount, "unit": case.unit, "frac": case.amount / t / peak,
                                                            "beside": like if name == mine else None}
@@ -765,8 +815,8 @@ def run_design(args):
 
 def main():
     ap = argparse.ArgumentParser()
-    ap.add_argument("--design", default="llama", choices=["llama", "finuvik"],
-                    help="finuvik: throughput of the Finuvik design and its kernels beside the LLaMA design at equal size (one GPU; other "
+    ap.add_argument("--design", default="llama", choices=["llama", "finuvik", "fuposun"],
+                    help="finuvik, fuposun: throughput of that design and its kernels beside the LLaMA design at equal size (one GPU; other "
                          "options do not apply)")
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=128)
@@ -784,7 +834,7 @@ def main():
     args = ap.parse_args()
     if args.warmup < 3 and args.impl == "ours":
         args.warmup = 3
-    if args.design == "finuvik":
+    if args.design != "llama":
         run_design(args)
     elif args.impl == "reference":
         run_reference(args, args.workload)

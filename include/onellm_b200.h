@@ -659,7 +659,7 @@ ONELLM_API int onellm_softcap(const float* in, long ld, float* out, int rows, in
  *       [T, H, rank_p] is the weighted latent of a head, times sigmoid(gate[t * gate_ld + h]) and out_scale.  Ring and (context
  *       pass) fresh latents in packed order.  `plain`: one warp per token and head, any type; else BF16 tensor-core warps
  *       (T <= 64).
- * rank_p: rank padded to a multiple of 16, the padding zero. */
+ * rank_p: rank padded to a multiple of 64, the padding zero. */
 typedef struct onellm_latent_attn {
     int dtype;
     int H, rank, window, R;

@@ -27,7 +27,7 @@ ENGINE_SOURCES = ["elementwise.cu", "engine.cu", "errors.cpp", "gemm_tc.cu", "mo
                   "skinny_gemm.cu", "skinny_gemm_staged.cu", "skinny_gemm_tc.cu", "weight_placer.cu"]
 DESIGN_SOURCES = {
     "Finuvik": ["biased_attn.cu", "biased_attn_tc.cu", "finuvik.cu", "gated_recurrence.cu"],
-    "Fuposun": ["biased_attn_tc.cu", "fuposun.cu", "gated_recurrence.cu", "latent_attn.cu", "route.cu"],
+    "Fuposun": ["biased_attn_tc.cu", "fuposun.cu", "gated_recurrence.cu", "latent_attn.cu", "latent_attn_tc.cu", "route.cu"],
 }
 
 

@@ -20,7 +20,7 @@
 //                      added to the stream directly
 //
 // Sizes that the kernels do not take as they are get padded in memory with zero weights, which leaves every result as it
-// is: rows and heads to multiples of 16, recurrence value heads to multiples of 32.
+// is: rows and heads to multiples of 16, latents to 64, recurrence value heads to multiples of 32.
 #include <math.h>
 #include <string.h>
 
@@ -308,7 +308,7 @@ void Fuposun::carve(Carver& cv)
         } else {
             w.dv = pad_to(l.dv, 16);
             w.q_rank = pad_to(l.q_rank, 16);
-            w.kv_rank = pad_to(l.kv_rank, 16);
+            w.kv_rank = latent_pad(l.kv_rank);
             w.col_c = w.q_rank;
             w.col_g = w.col_c + w.kv_rank;
             w.n_in = w.col_g + pad_to(l.H, 16);

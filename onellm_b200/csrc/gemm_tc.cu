@@ -341,6 +341,20 @@ int make_map(CUtensorMap* map, const void* base, uint64_t inner, uint64_t outer,
     return ONELLM_OK;
 }
 
+int make_chunk_map(CUtensorMap* map, const void* base, uint64_t inner, uint64_t outer, uint32_t box_rows, uint32_t box_chunks)
+{
+    EncodeTiledFn enc = encode_tiled();
+    ONELLM_REQUIRE(enc, ONELLM_ERR_CUDA, "cuTensorMapEncodeTiled is not available from the driver");
+    const cuuint64_t dims[3] = {64, outer, inner / 64};
+    const cuuint64_t strides[2] = {inner * 2, 128};
+    const cuuint32_t box[3] = {64, box_rows, box_chunks};
+    const cuuint32_t estr[3] = {1, 1, 1};
+    const CUresult r = enc(map, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 3, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                           CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    ONELLM_REQUIRE(r == CUDA_SUCCESS, ONELLM_ERR_CUDA, "cuTensorMapEncodeTiled failed with %d", (int)r);
+    return ONELLM_OK;
+}
+
 int gemm_f16_skinny(const __half* x, const __half* W, __half* y, int M, int N, int K, int w_layout, cudaStream_t st);
 
 // mode 0: W [K,N]; 1: W [N,K]; 2: W and W2 [K,N], y = silu(x.W) * (x.W2)

@@ -6,8 +6,9 @@
 // every head reads the same rows and only those are cached.  They lie in a ring as long as the window, so a sequence's
 // memory does not grow with its length.
 //
-// The tensor-core kernel (at most 64 tokens: decode steps and short portions) owns up to 16 heads of one token and one
-// range of its keys: 16 is the row operand of mma.m16n8k16, so heads beyond the first are free.  Tiles of 32 latents go
+// Decode steps run on tcgen05 (latent_attn_tc.cu).  The kernel here (short portions of a prompt, at most 64 tokens, and
+// decode steps with latents above 512) owns up to 16 heads of one token and one range of its keys: 16 is the row operand of
+// mma.m16n8k16, so heads beyond the first are free.  Tiles of 32 latents go
 // through a cp.async ring; the eight warps first share the scores out by keys and halves of the rank, then the outputs by
 // 16-column groups of the same tile, which is key and value at once.  Tiles that hold no token of this very pass are
 // requested before the dependency wait.  Whole prompts are cheaper with the keys and values formed once per token
@@ -19,8 +20,6 @@
 #include "mixers.h"
 
 namespace onellm {
-
-static int latent_pad(int rank) { return (rank + 15) / 16 * 16; }
 
 // positions a sequence brings along from its ring into a joined buffer
 __device__ __forceinline__ int kept_rows(const LatentAttn& a, int hist) { return min(hist, a.window - 1); }
@@ -437,8 +436,15 @@ __global__ void __launch_bounds__(128) latent_attn_merge_kernel(const LaParams p
 }
 
 constexpr int kLaMaxSplits = 16;
+// latent_attn_tc.cu: decode steps
+bool latent_attn_tc_takes(const LatentAttn& a, const TokenPositions& tp);
+size_t latent_attn_tc_workspace(int tokens, int H, int rank);
+int latent_attn_tc(const LatentAttn& a, const TokenPositions& tp, int tokens, int span_bound, void* workspace, cudaStream_t st);
 
-size_t latent_attn_workspace(int tokens, int H, int rank) { return (size_t)std::min(tokens, 64) * H * kLaMaxSplits * (latent_pad(rank) + 2) * sizeof(float); }
+size_t latent_attn_workspace(int tokens, int H, int rank)
+{
+    return std::max((size_t)std::min(tokens, 64) * H * kLaMaxSplits * (latent_pad(rank) + 2) * sizeof(float), latent_attn_tc_workspace(tokens, H, rank));
+}
 
 template <int NP>
 static int launch_la(const LaParams& p, dim3 grid, size_t smem, cudaStream_t st)
@@ -462,7 +468,9 @@ int latent_attn(const LatentAttn& a, const TokenPositions& tp, int tokens, int s
         else ONELLM_CUDA(launch_pdl(latent_attn_plain_kernel<__nv_bfloat16>, grid, dim3(128), 0, st, a, tp, rank_p));
         return ONELLM_OK;
     }
-    ONELLM_REQUIRE(tokens <= 64 && workspace, ONELLM_ERR_UNSUPPORTED, "latent_attn: %d tokens, at most 64 in latent space", tokens);
+    ONELLM_REQUIRE(workspace, ONELLM_ERR_ARG, "latent_attn: no workspace");
+    if (latent_attn_tc_takes(a, tp)) return latent_attn_tc(a, tp, tokens, span_bound, workspace, st);
+    ONELLM_REQUIRE(tokens <= 64, ONELLM_ERR_UNSUPPORTED, "latent_attn: %d tokens, at most 64 in latent space", tokens);
     const size_t tile = la_tile_bytes(rank_p), fixed = la_fixed_bytes(rank_p);
     const int nst = (int)std::max<size_t>(2, std::min<size_t>(6, (108 * 1024 - std::min<size_t>(fixed, 64 * 1024)) / tile));
     // ranges: enough blocks for the SMs, of at least four tiles each

@@ -49,6 +49,7 @@ size_t gated_recurrence_workspace(int kind, int tokens, int H, int dk, int dv);
 int gated_recurrence(const GatedRecurrence& g, const TokenPositions& tp, int B, int tokens, cudaStream_t st);
 
 // max_hist: most positions a sequence has before this pass; max_new: most new tokens of one
+inline int latent_pad(int rank) { return (rank + 63) / 64 * 64; }
 int latent_store(const LatentAttn& a, const TokenPositions& tp, int tokens, int max_hist, cudaStream_t st);
 int latent_keep(const LatentAttn& a, const TokenPositions& tp, int max_new, cudaStream_t st);
 size_t latent_attn_workspace(int tokens, int H, int rank);

@@ -29,6 +29,13 @@ many recurrence heads as attention heads), each beside the like case above:
                                    stream of 4096 rows
     prefill_fv_mix, prefill_fv_gate, prefill_fv_out, prefill_fv_attn, prefill_fv_rec       the same in the context phase
 
+    fu_in, fu_uq, fu_out           decode: mixer inputs of a gla layer, queries out of their latent, output added to the float stream
+    fu_absorb, fu_attn, fu_uv      queries into latent space per head, attention over a window of --ctx latents, values out of it
+    fu_rec, fu_norm                one step of the gla recurrence; norm of 4096 rows that takes the experts' rows first
+    fu_route, fu_egate, fu_edown   router and choice; gate/up and down of the chosen experts
+    prefill_fu_in, prefill_fu_kv, prefill_fu_attn, prefill_fu_rec, prefill_fu_route, prefill_fu_egate, prefill_fu_edown
+                                   the same in the context phase (window: 1024 positions)
+
 Every case holds a few hundred MB on the device (more than the 126 MB L2, far less than a model) and runs on
 rotating buffers.  `--tp T` uses the per-rank shapes of T-way tensor parallelism; `--graph` times the launches as
 one CUDA graph, i.e. back to back on the device without the host's launch cost (what a decode step sees).
@@ -47,9 +54,11 @@ MODELS = {
 }
 
 DECODE_CASES = ["qkv", "o_proj", "gate_up", "down", "lm_head_kn", "lm_head", "attn", "attn_c1", "norm", "rmsnorm", "norm8",
-                "topk", "sample", "decode_layer", "fv_mix", "fv_gate_up", "fv_out", "fv_attn", "fv_rec", "fv_norm"]
+                "topk", "sample", "decode_layer", "fv_mix", "fv_gate_up", "fv_out", "fv_attn", "fv_rec", "fv_norm", "fu_in", "fu_uq", "fu_out",
+                "fu_absorb", "fu_attn", "fu_uv", "fu_rec", "fu_norm", "fu_route", "fu_egate", "fu_edown"]
 PREFILL_CASES = ["prefill_qkv", "prefill_o", "prefill_gate", "prefill_down", "prefill_lm", "prefill_attn", "prefill_rope",
-                 "prefill_layer", "prefill_fv_mix", "prefill_fv_gate", "prefill_fv_out", "prefill_fv_attn", "prefill_fv_rec"]
+                 "prefill_layer", "prefill_fv_mix", "prefill_fv_gate", "prefill_fv_out", "prefill_fv_attn", "prefill_fv_rec", "prefill_fu_in",
+                 "prefill_fu_kv", "prefill_fu_attn", "prefill_fu_rec", "prefill_fu_route", "prefill_fu_egate", "prefill_fu_edown"]
 
 
 @dataclass
@@ -152,8 +161,131 @@ def make_mechanism_case(name, torch, m, B, ctx, plain=False) -> Case:
     raise ValueError(f"unknown case {name}")
 
 
+def make_latent_case(name, torch, m, B, ctx, plain=False) -> Case:
+    """The fu_ cases: m as in MODELS, optionally with q_rank, kv_rank, window, gla (heads, key, value), gate_rank, experts, top, eff."""
+    prefill = name.startswith("prefill_")
+    what = name[name.index("fu_") + 3:]
+    W, H, D = m["hidden"], m["head_num"], m["head_size"]
+    DV, QR, KR = m.get("value_size", D), m.get("q_rank", 1536), m.get("kv_rank", 512)
+    RH, RK, RV = m.get("gla", (W // 512, 256, 512))
+    E, TOP, EF, rank = m.get("experts", 32), m.get("top", 4), m.get("eff", m["inter_size"] // 4), m.get("gate_rank", 16)
+    window = min(m.get("window", 1024), ctx) if prefill else ctx
+    T = B * ctx if prefill else B
+    bf, f32, i32 = (dict(device="cuda", dtype=t) for t in (torch.bfloat16, torch.float32, torch.int32))
+    rnd = lambda *s: 0.02 * torch.randn(*s, **bf)
+    n_rot = lambda nbytes, target=400e6: 2 if prefill else max(2, int(target // nbytes) + 1)
+    BF = ob.BF16
+    n_gla = RH * (2 * RK + 2 * RV) + 16
+    plain_shapes = {"in": (W, n_gla), "uq": (QR, H * D), "out": (H * DV, W), "kv": (KR, H * (D + DV))}
+    if what in plain_shapes:
+        K, N = plain_shapes[what]
+        rot = n_rot(K * N * 2)
+        x, w = torch.randn(T, K, **bf), [rnd(K, N) for _ in range(rot)]
+        stream = what == "out"
+        y = torch.zeros(T, N, **(f32 if stream else bf))
+        fn = lambda i: ob.project(BF, x, w[i], None, y, T, N, K, f32=stream, resid=y if stream else None, scale=0.3)
+        if prefill:
+            return Case(fn, rot, 2.0 * T * N * K, "flop", "gemm_tc_kernel (bf16)", keep=(x, w, y))
+        return Case(fn, rot, K * N * 2 + T * K * 2 + T * N * (8 if stream else 2), "B", _projection_kernel(T, False) + " (bf16)", keep=(x, w, y))
+    if what in ("absorb", "uv"):
+        K, N = (D, KR) if what == "absorb" else (KR, DV)
+        rot = n_rot(H * K * N * 2)
+        x, w, y = torch.randn(T, H * K, **bf), [rnd(H, K, N) for _ in range(rot)], torch.zeros(T, H * N, **bf)
+        g = ob.RowGroups(n=H, w_stride=K * N, x_stride=K, y_stride=N)
+        fn = lambda i: ob.project(BF, x, w[i], None, y, T, N, K, ldx=H * K, ldy=H * N, ldw=N, groups=g)
+        return Case(fn, rot, H * K * N * 2 + T * H * (K + N) * 2, "B", "skinny_kn_staged_kernel (row groups)", keep=(x, w, y, g))
+    if what == "norm":
+        rows = 4096
+        xs = [torch.randn(rows, W, **f32) for _ in range(3)]
+        add = [torch.randn(rows * TOP, W, **bf) for _ in range(3)]
+        pick = torch.randperm(rows * TOP, device="cuda").to(torch.int32)
+        w1, o1 = torch.ones(W, **f32), torch.empty(rows, W, **bf)
+        fn = lambda i: ob.norm_rows(BF, xs[i], None, rows, w1, None, o1, None, 1e-6, W, W, add=add[i], add_rows=pick, add_n=TOP, add_scale=0.3)
+        return Case(fn, 3, rows * W * (8 + 2 + 2 * TOP), "B", "norm_rows_kernel", keep=(xs, add, pick, w1, o1))
+    if what in ("route", "egate", "edown"):
+        n = T * TOP
+        h, router = torch.randn(T, W, **bf), rnd(W, E)
+        z = torch.zeros(T, E, **f32)
+        tiles = ob.route_max_tiles(T, E, TOP)
+        a = {k: torch.zeros(s, **i32) for k, s in (("slot", n), ("slot_token", n), ("off", E + 1), ("used", E), ("n_used", 1), ("tile_group", tiles),
+                                                   ("tile_row", tiles), ("n_tiles", 1), ("choice", n), ("count", E))}
+        a.update(slot_weight=torch.zeros(n, **f32), choice_weight=torch.zeros(n, **f32))
+        p = {k: v.data_ptr() for k, v in a.items()}
+        xs = torch.zeros(n, W, **bf) if T > 64 else None
+        r = ob.Route(T, E, TOP, z.data_ptr(), E, dtype=BF, **p)
+        if xs is not None:
+            r.x, r.xs, r.ld_x = h.data_ptr(), xs.data_ptr(), W
+
+        def choose(i):
+            ob.project(BF, h, router, None, z, T, E, W, f32=True)
+            ob.route(r)
+        keep = (h, router, z, a, xs, r)
+        if what == "route":
+            nbytes = T * W * 2 + W * E * 2 + T * E * 8 + (T * W * 2 + n * W * 2 if prefill else 0)
+            return Case(choose, 2, nbytes, "B", "router projection, route kernels", launches=5 if T > 64 else 2, keep=keep)
+        choose(0)
+        used = int(a["n_used"].item())
+        K, N = (W, EF) if what == "egate" else (EF, W)
+        dual = what == "egate"
+        rot = n_rot(used * K * N * 2 * (2 if dual else 1))
+        w = [rnd(E, K, N) for _ in range(rot)]
+        wu = [rnd(E, K, N) for _ in range(rot)] if dual else [None] * rot
+        tiled = T > 64
+        x = (xs if tiled else h) if dual else torch.randn(n, K, **bf)
+        y = torch.zeros(n, N, **bf)
+        g = ob.RowGroups(n=E if tiled else min(E, n), used=None if tiled else p["used"], n_used=None if tiled else p["n_used"], off=p["off"],
+                         x_rows=p["slot_token"] if dual and not tiled else None, row_scale=p["slot_weight"] if dual else None, w_stride=K * N,
+                         tile_group=p["tile_group"], tile_row=p["tile_row"], n_tiles=p["n_tiles"], max_tiles=tiles, weights=E, rows=n)
+        fn = lambda i: ob.project(BF, x, w[i], wu[i], y, T, N, K, act=ob.GATE_CLAMPED, limit=7.0, groups=g)
+        keep += (w, wu, x, y, g)
+        if prefill:
+            return Case(fn, rot, 2.0 * n * N * K * (2 if dual else 1), "flop", "gemm_tc_kernel (row groups)", keep=keep)
+        return Case(fn, rot, used * K * N * 2 * (2 if dual else 1) + n * (K + N) * 2, "B", "skinny_kn_staged_kernel (row groups)", keep=keep)
+    cu = torch.arange(0, B + 1, **i32) * ctx
+    hist, off = torch.zeros(B, **i32), torch.zeros(B, **i32)
+    step = torch.full((1,), ctx + 1, **i32)
+    tp = ob.TokenPositions(cu.data_ptr(), hist.data_ptr(), B, None, None) if prefill else \
+        ob.TokenPositions(None, None, B, step.data_ptr(), off.data_ptr())
+    if what == "attn" and prefill:
+        q, gate, out = torch.randn(T, H * D, **bf), torch.randn(T, H, **bf), torch.zeros(T, H * DV, **bf)
+        kv = [torch.randn(T, H * (D + DV), **bf) for _ in range(2)]
+        a = [ob.WindowAttn(H, D, DV, window, q.data_ptr(), H * D, kv[i].data_ptr(), H * (D + DV), T, D ** -0.5, gate.data_ptr(), H, out.data_ptr(),
+                           H * DV, 1.0) for i in range(2)]
+        fn = lambda i: ob.window_attn(a[i], tp, ctx)
+        keys = window * (window + 1) / 2 + (ctx - window) * window
+        return Case(fn, 2, float(B * H * 2 * (D + DV) * keys), "flop", "biased_attn_tc_kernel<windowed>", keep=(q, gate, out, kv, cu, hist))
+    if what == "attn":
+        rot = n_rot(B * window * KR * 2, 300e6)
+        ring = [torch.randn(B, window, KR, **bf) for _ in range(rot)]
+        q, gate, out = torch.randn(B, H, KR, **bf), torch.randn(B, H, **bf), torch.zeros(B, H, KR, **bf)
+        ws = torch.empty(ob.latent_attn_workspace(B, H, KR), device="cuda", dtype=torch.uint8)
+        a = [ob.LatentAttn(BF, H, KR, window, window, ring[i].data_ptr(), None, 0, None, None, 0, None, None, 0, 0, None, 1e-6, q.data_ptr(),
+                           KR ** -0.5, gate.data_ptr(), H, out.data_ptr(), 1.0) for i in range(rot)]
+        fn = lambda i: ob.latent_attn(a[i], tp, B, window, ws, plain)
+        return Case(fn, rot, B * window * KR * 2 + 2 * B * H * KR * 2, "B", "latent_attn_kernel", launches=2, keep=(ring, q, gate, out, ws, step, off))
+    if what == "rec":
+        rot = n_rot(2 * B * RH * RK * RV * 4, 300e6)
+        state = [torch.zeros(B, RH, RK, RV, **f32) for _ in range(rot)]
+        row, out = torch.randn(T, n_gla, **bf), torch.zeros(T, RH * RV, **bf)
+        A, zb, w = torch.randn(RH * RK, rank, **f32), torch.full((RH * RK,), 2.0, **f32), torch.ones(RV, **f32)
+        work = torch.empty(ob.gated_recurrence_workspace(T, RH, RK, RV, ob.GR_KEYED), device="cuda", dtype=torch.uint8)
+        p = row.data_ptr()
+        g = [ob.GatedRecurrence(BF, RH, RK, RV, q=p, v=p + 2 * RH * RK * 2, ld=n_gla, zb=zb.data_ptr(), w=w.data_ptr(), eps=1e-6, norm_width=RV,
+                                state=state[i].data_ptr(), out=out.data_ptr(), out_ld=RH * RV, out_scale=1.0, work=work.data_ptr(), kind=ob.GR_KEYED,
+                                k=p + RH * RK * 2, r=p + RH * (2 * RK + 2 * RV) * 2, rank=rank, A=A.data_ptr(), inv_tau=1 / 16, q_scale=RK ** -0.5,
+                                g=p + RH * (2 * RK + RV) * 2) for i in range(rot)]
+        fn = lambda i: ob.gated_recurrence(g[i], tp, T)
+        keep = (state, row, out, A, zb, w, work, cu, hist, off, step)
+        if prefill:  # decay, write and read of a state element and token, as counted for fv_rec
+            return Case(fn, rot, 5.0 * T * RH * RK * RV, "flop", "gated_recurrence_scan_kernel", launches=3, keep=keep)
+        return Case(fn, rot, 2 * B * RH * RK * RV * 4 + B * RH * (2 * RK + 3 * RV) * 2, "B", "gated_recurrence_step_kernel", keep=keep)
+    raise ValueError(f"unknown case {name}")
+
+
 def make_case(name, torch, model="7b", batch=8, ctx=2040, tp=1, plain=False) -> Case:
     m = MODELS[model] if isinstance(model, str) else model
+    if "fu_" in name:
+        return make_latent_case(name, torch, m, batch, ctx, plain)
     if "fv_" in name:
         return make_mechanism_case(name, torch, m, batch, ctx, plain)
     HID, D, V = m["hidden"], m["head_size"], m["vocab_size"]

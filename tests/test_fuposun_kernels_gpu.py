@@ -207,7 +207,7 @@ class Latents:
 
     def __init__(self, cuda, ob, kind, H, rank, window, lens, seed=0, R=None):
         self.ob, self.kind, self.d, self.torch = ob, kind, Dev(cuda, ob, kind), cuda
-        self.H, self.rank, self.rp, self.window, self.lens = H, rank, pad(rank), window, lens
+        self.H, self.rank, self.rp, self.window, self.lens = H, rank, pad(rank, 64), window, lens
         rng = self.rng = np.random.default_rng(seed)
         self.w = round_bf16(1 + 0.2 * rng.standard_normal(rank))
         self.qw = round_bf16(1 + 0.2 * rng.standard_normal(24))
@@ -267,7 +267,7 @@ class Latents:
         return ur.latent_attention(q, c, eye, eye, pos, np.arange(len(c)), self.scale, self.window)
 
 
-LATENT_SIZES = [(1, 16, 5), (8, 96, 33), (20, 72, 1), (16, 144, 64), (3, 272, 100), (17, 512, 40), (2, 1024, 31), (4, 128, 700)]  # H, rank, window
+LATENT_SIZES = [(1, 16, 5), (8, 96, 33), (20, 72, 1), (16, 144, 64), (3, 272, 100), (17, 512, 40), (2, 1024, 31), (4, 128, 700), (70, 64, 300)]  # H, rank, window
 
 
 @pytest.mark.parametrize("kind,plain", [("f32", True), ("bf16", True), ("bf16", False)])
@@ -278,7 +278,7 @@ def test_latent_attention(cuda, ob, kind, plain, H, rank, window):
     hist = [0, 0, 0, 0]
     for counts in ([10, 1, 40, 13], [2, 2, 3, 50]):
         q = rounded(t.rng.standard_normal((sum(counts), H, rank)), kind)
-        gate = rounded(t.rng.standard_normal((sum(counts), 24)), kind)
+        gate = rounded(t.rng.standard_normal((sum(counts), H + 3)), kind)
         t.store(hist, counts)
         got = t.attend(q, gate, plain, 0.7)
         t.keep()
@@ -343,7 +343,7 @@ def test_latent_attention_in_one_range_and_in_many(cuda, ob):
                                             (2, 64, 64, 1000)])
 def test_window_attention_of_a_context_pass(cuda, ob, H, dk, dv, window):
     """Keys and values formed from the joined latents; queries over several tiles, portions behind a history, both edges."""
-    rank, rp = 48, 48
+    rank, rp = 48, 64
     lens = [290, 61, 130, 2]
     hist = [0, 37, 126, 0]
     counts = [n - h for n, h in zip(lens, hist)]
@@ -355,7 +355,7 @@ def test_window_attention_of_a_context_pass(cuda, ob, H, dk, dv, window):
     uk, uv = (rounded(t.rng.standard_normal((H * n, rank)) / np.sqrt(rank), "bf16") for n in (dk, dv))
     ld, rows = H * (dk + dv), t.fresh.shape[0]
     kv = d.zeros(rows, ld)
-    ob.project(ob.BF16, t.fresh, d.up(np.concatenate([uk, uv]).T), None, kv, rows, ld, rp)
+    ob.project(ob.BF16, t.fresh, d.up(padded(np.concatenate([uk, uv]), rp).T), None, kv, rows, ld, rp)
     T = sum(counts)
     q = rounded(t.rng.standard_normal((T, H, dk)) * 2, "bf16")
     # one key that stands out at the last visible distance of the first sequence's last query, another just outside
