@@ -782,9 +782,10 @@ def run_design(args):
                      ("prefill_fv_mix", "prefill_qkv"), ("prefill_fv_gate", "prefill_gate"), ("prefill_fv_out", "prefill_down"),
                      ("prefill_fv_attn", "prefill_attn"), ("prefill_fv_rec", None)]
         else:
-            pairs = [("fu_in", "qkv"), ("fu_uq", "o_proj"), ("fu_absorb", "o_proj"), ("fu_uv", "o_proj"), ("fu_out", "o_proj"), ("fu_egate", "gate_up"),
-                     ("fu_edown", "down"), ("fu_route", None), ("fu_attn", "attn"), ("fu_rec", "fv_rec"), ("fu_norm", "fv_norm"),
-                     ("prefill_fu_in", "prefill_qkv"), ("prefill_fu_kv", "prefill_qkv"), ("prefill_fu_egate", "prefill_gate"),
+            # "/8": the shape of one of eight ranks, "@rows": that many cache rows (the like kernel at about as many bytes)
+            pairs = [("fu_in", "qkv"), ("fu_uq", "o_proj/2"), ("fu_absorb", "o_proj/8"), ("fu_uv", "o_proj/8"), ("fu_out", "o_proj"),
+                     ("fu_egate", "gate_up"), ("fu_edown", "down"), ("fu_route", None), ("fu_attn", "attn@64"), ("fu_rec", "fv_rec"),
+                     ("fu_norm", "fv_norm"), ("prefill_fu_in", "prefill_qkv"), ("prefill_fu_kv", "prefill_o/8"), ("prefill_fu_egate", "prefill_gate"),
                      ("prefill_fu_edown", "prefill_down"), ("prefill_fu_route", None), ("prefill_fu_attn", "prefill_attn"),
                      ("prefill_fu_rec", "prefill_fv_rec")]
         fp32_peak = 148 * 128 * 2 * 1.965e9 / 1e12  # nominal: the recurrences run on the fp32 pipes
@@ -794,10 +795,12 @@ def run_design(args):
                 if name is None or name in done:
                     continue
                 prefill = name.startswith("prefill_")
-                decode = ((8, 2040), (32, 2040)) if name in ("fv_attn", "attn", "fv_rec", "fu_rec") else \
-                    ((8, 1024), (32, 1024), (32, 4096)) if name == "fu_attn" else ((8, 2040),)
+                decode = ((8, 2040), (32, 2040)) if name in ("fv_attn", "attn", "attn@64", "fv_rec", "fu_rec") else \
+                    ((8, 1024), (32, 1024), (32, 4096)) if name == "fu_attn" else ((8, 2040), (32, 2040)) if "_e" in name else ((8, 2040),)
                 for b, ctx in ((1, 2048), (8, 512)) if prefill else decode:
-                    case = kc.make_case(name, torch, "7b", b, ctx, 1)
+                    base, _, tp = name.partition("/")
+                    base, _, rows = base.partition("@")
+                    case = kc.make_case(base, torch, "7b", b, int(rows or ctx), int(tp or 1))
                     t = kc.time_case(case, torch, iters=20, warm=5, graph=not prefill)
                     peak = fp32_peak * 1e12 if name in ("prefill_fv_rec", "prefill_fu_rec") else tf_peak * 1e12 if case.unit == "flop" else hbm_peak * 1e9
                     done[name] = True

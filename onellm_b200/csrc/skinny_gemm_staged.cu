@@ -549,7 +549,9 @@ static cudaError_t launch_staged(const T* x, const T* W0, const T* W1, T* y, int
     return cudaLaunchKernelEx(&cfg, kern, x, W0, W1, y, M, N, K, plan.per_block, plan.nst, fn, ep, GroupArgs{});
 }
 
-// Row groups: two blocks per SM, K split while that leaves whole waves of them to fill.
+bool plan_override_lookup(int N, int K, bool dual, int* ks, int* nst);
+
+// Row groups: K split while the blocks of all groups are resident at once.
 template <int MB, bool DUAL>
 static cudaError_t launch_grouped(const onellm_projection& p, const EpilogueArgs& ep, const GroupArgs& ga, cudaStream_t st)
 {
@@ -569,9 +571,12 @@ static cudaError_t launch_grouped(const onellm_projection& p, const EpilogueArgs
     const long blocks = (long)cols * ga.g.n;
     int ks = 1;
     while (ks < 8 && blocks * (ks + 1) <= 2L * num_sms() && (total + ks) / (ks + 1) >= 4) ks++;
+    // several waves of blocks: shallow rings, so that four of them share an SM and their ends overlap
+    int depth = blocks * ks <= 2L * num_sms() ? 12 : 6, oks = 0;
+    if (plan_override_lookup(p.N, p.K, DUAL, &oks, &depth)) ks = std::max(1, std::min({8, total, oks}));
     int per = (total + ks - 1) / ks;
     while (ks > 1 && per * (ks - 1) >= total) per = (total + --ks - 1) / ks;
-    const int nst = std::max(3, std::min({12, per + 1, (int)(cap / stage)}));
+    const int nst = std::max(3, std::min({12, depth, per + 1, (int)(cap / stage)}));
     cudaLaunchConfig_t cfg = {};
     cudaLaunchAttribute at[2];
     at[0].id = cudaLaunchAttributeClusterDimension;
