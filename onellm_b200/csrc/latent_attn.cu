@@ -244,7 +244,10 @@ __device__ __forceinline__ void ldsm_x2(uint32_t (&r)[2], uint32_t addr)
 }
 
 // bytes of the fixed part of the shared memory: queries, scores, weights, row factors
-static size_t la_fixed_bytes(int rank_p) { return (size_t)kLaHeads * (rank_p * 2 + 16) + 2 * kLaHeads * (kLaKeys + 1) * 4 + kLaHeads * (kLaKeys + 8) * 2 + 2 * kLaHeads * 4; }
+static size_t la_fixed_bytes(int rank_p)
+{
+    return (size_t)kLaHeads * (rank_p * 2 + 16) + 2 * kLaHeads * (kLaKeys + 1) * 4 + kLaHeads * (kLaKeys + 8) * 2 + 2 * kLaHeads * 4;
+}
 static size_t la_tile_bytes(int rank_p) { return (size_t)kLaKeys * (rank_p * 2 + 16); }
 
 // NP: 16-column groups of a warp, rank_p <= 128 NP

@@ -187,7 +187,9 @@ latent_attn_tc_kernel(const LtParams p, const __grid_constant__ CUtensorMap map_
         };
         bool ok = wait_all(q_full, 0) && issue_s(0);
         for (int j = 0; j < n_tiles && ok; j++) {
-            const bool more = j + 1 < n_tiles, ahead = more && __all_sync(0xffffffffu, mbar_test(full0 + 8 * ((j + 1) % p.n_buf), (uint32_t)((j + 1) / p.n_buf) & 1u));
+            const bool more = j + 1 < n_tiles;
+            const bool arrived = more && mbar_test(full0 + 8 * ((j + 1) % p.n_buf), (uint32_t)((j + 1) / p.n_buf) & 1u);
+            const bool ahead = __all_sync(0xffffffffu, arrived);
             if (ahead) ok = issue_s(j + 1);
             ok = ok && wait_all(p_full0 + 8 * (j & 1), (j >> 1) & 1);
             if (!ok) break;
